@@ -74,7 +74,7 @@ int lcu_quantize_model_dir(const char* in_dir, const char* out_dir, int bs);
 int lcu_matmul_nt_f16(void* out_dev, const void* lhs_dev, const void* rhs_dev, int m, int k, int n, float beta, void* stream);
 /* The feed-forward's first half as one launch: matmul_nt of lhs(m,k) with w1 and with w3 (llama_cu.cu:1180-1181; w13 =
  * [w1; w3], (2 f, k), k a multiple of 64) and silu (llama_cu.cu:533-539, 1182-1183) on the half-rounded products: out(m,f).
- * The same bits as lcu_matmul_nt_f16 on each matrix followed by lcu_silu.  tile = accumulator columns per output tile:
+ * Within one unit in the last place of lcu_matmul_nt_f16 on each matrix followed by lcu_silu.  tile = accumulator columns per output tile:
  * 256 (f a multiple of 128; the gate runs under the next tile's main loop) or 512 (f a multiple of 256).  Prompt passes
  * use it as the tuning key "prefill_gate_fused" says (-1 = when estimated faster, 256 / 512 = from 129 rows with that
  * tile, 0 = never). */
@@ -240,10 +240,9 @@ int lcu_profiler_stop(void);
  * (LCU_ERR_DEVICE_WAIT) with the device code (0x101) in *device_code_out; the context stays usable.  No counterpart
  * in the reference (its kernels have no waits). */
 int lcu_selftest_bounded_wait(int* device_code_out);
-/* The quantizer forms q = u8(roundf(127.5f + x / scale)) (transform.cu:60-80) with a reciprocal multiply, one residual
- * correction and trunc(v + 0.5f).  This entry compares that with the reference's IEEE division and roundf for EVERY pair
- * (x a finite half, scale a positive finite half, |x| within the absmax that rounds to the scale) on the device and
- * returns the number of pairs checked and the number of differing bytes (0). */
+/* The quantizer forms q = u8(roundf(127.5f + x / scale)) (transform.cu:60-80) as the truncation of x / scale + 128.  This
+ * entry compares the two for EVERY pair (x a finite half, scale a positive finite half, |x| within the absmax that rounds
+ * to the scale) on the device and returns the number of pairs checked and the number of differing bytes (0). */
 int lcu_selftest_quantizer_arithmetic(uint64_t* checked_out, uint64_t* differences_out);
 /* Host arithmetic only (no device needed): how lcu_matmul_nt_f16 cuts out(m,n) = lhs(m,k) . rhs(n,k)^T for m <= 128 rows on
  * a GPU of `sms` SMs - the tile width (96 to 256 columns; the last tile may hang over n) and the split-K factor (1, 2 or 4,
@@ -257,9 +256,9 @@ int lcu_plan_long_prompt_gemm(int m, int n, int k, int sms, int* kernel_out);
  * and each shared tile's owner finds exactly the pairs that ran the rest of it, in order; a positive code names the rule
  * that failed, -1 bad arguments. */
 int lcu_selftest_balanced_schedule(int n_tiles, int k_steps, int sm_pairs);
-/* lcu_matmul_nt_f16_gated forms silu's a / (1 + expf(-a)) (llama_cu.cu:533-539) with a refined reciprocal and one
- * residual correction instead of the IEEE division.  This entry compares the two on the device for all 65536
- * half-precision a (the only values the gate meets) and returns how many were compared and how many differ (0). */
+/* lcu_matmul_nt_f16_gated forms silu's a / (1 + expf(-a)) (llama_cu.cu:533-539) with CUDA's __fdividef.  This entry
+ * compares it, rounded to half, with the division on the device for all 65536 half-precision a and returns how many were
+ * compared and how many differ (a few, each by one unit in the last place). */
 int lcu_selftest_silu_arithmetic(uint64_t* checked_out, uint64_t* differences_out);
 /* lcu_matmul_nt_f16 (beta = 0, default stream) launched `reps` times back to back between two CUDA events on that
  * stream: mean milliseconds per launch.  Used to put the prompt GEMM against the tensor-core roofline. */

@@ -195,13 +195,9 @@ __global__ void __launch_bounds__(FA_THREADS, 1) attn_fused_kernel(const __grid_
     const int row = quad * 32 + lane, grow = m0 + row;
     const int last_key = pos0 + grow;  // the row sees keys 0 .. last_key
     const uint32_t lane_base = tmem_base + ((uint32_t)(quad * 32) << 16);
-    // x / sqrt(head_dim) as one multiplication and a residual correction: RN(x / d) in all but vanishingly rare
-    // double-rounding cases (the result is rounded to half right after)
-    const float scale_div = sqrtf((float)HD), scale_rcp = __frcp_rn(scale_div);
-    auto scaled = [&](uint32_t bits) {
-      const float x = __uint_as_float(bits), q = x * scale_rcp;
-      return fmaf(fmaf(-q, scale_div, x), scale_rcp, q);
-    };
+    // x / sqrt(head_dim) as a product with the reciprocal (the result is rounded to half right after)
+    const float scale_rcp = 1.0f / sqrtf((float)HD);
+    auto scaled = [&](uint32_t bits) { return __uint_as_float(bits) * scale_rcp; };
     auto ex2 = [](float y) {
       float r;
       asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(y));
@@ -288,13 +284,9 @@ __global__ void __launch_bounds__(FA_THREADS, 1) attn_fused_kernel(const __grid_
         sum += part_s[q] * ex2((part_m[q] - mx) * LOG2E);  // (a part with every key above the diagonal: factor 0)
     }
     bar_sync(1, 32 * FA_EPI_WARPS);  // (the pairs lie where pass 2 writes probabilities)
-    const float rsum = __frcp_rn(sum);
-    // e / sum as one multiplication and a residual correction (RN(e / sum) in all but vanishingly rare cases)
+    const float rsum = 1.0f / sum;
     const float off2 = -mx * LOG2E;
-    auto prob = [&](float x) {
-      const float e = ex2(fmaf(x, LOG2E, off2)), q = e * rsum;
-      return fmaf(fmaf(-q, sum, e), rsum, q);
-    };
+    auto prob = [&](float x) { return ex2(fmaf(x, LOG2E, off2)) * rsum; };  // (rounded to half right after)
 
     // ---- pass 2: probabilities rounded to half into the K-major operand tile (128-byte swizzled rows of 64 keys)
     for (int j = 0; j < n_tiles && go; ++j) {

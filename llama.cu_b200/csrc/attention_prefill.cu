@@ -33,13 +33,6 @@ __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t addr, uint32_t& r0, u
 __device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
 }
-// x / d from r = RN(1 / d): one multiplication and one residual correction.  This is the core of the correctly
-// rounded division sequence without its special-case handling (operands here are finite, d >= 1): it returns
-// RN(x / d) in all but vanishingly rare double-rounding cases, at a third of the instructions.
-__device__ __forceinline__ float div_by(float x, float d, float r) {
-  const float q = x * r;
-  return fmaf(fmaf(-q, d, x), r, q);
-}
 __device__ __forceinline__ uint32_t pack_half2(float a, float b) {
   const __half2 h = __floats2half2_rn(a, b);
   return *reinterpret_cast<const uint32_t*>(&h);
@@ -60,7 +53,7 @@ __global__ void __launch_bounds__(PA_THREADS) attn_prefill_kernel(const attn_par
   const int ntiles = (nkeys + PA_KT - 1) / PA_KT;
   const __half* kb = p.k_cache + (size_t)head * p.ctx_len * HD;
   const __half* vb = p.v_cache + (size_t)head * p.ctx_len * HD;
-  const float scale_div = sqrtf((float)HD), scale_rcp = __frcp_rn(scale_div);
+  const float scale_rcp = 1.0f / sqrtf((float)HD);  // (scores and probabilities are rounded to half right after the product)
 
   // Q fragments (A operand, 16 rows x HD per warp): rows g and g + 8 of the warp's block
   const int r_lo = q0 + warp * 16 + g, r_hi = r_lo + 8;
@@ -110,10 +103,10 @@ __global__ void __launch_bounds__(PA_THREADS) attn_prefill_kernel(const attn_par
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const int t = t0 + j * 8 + 2 * c;
-      s[j][0] = t <= last_lo ? __half2float(__float2half(div_by(s[j][0], scale_div, scale_rcp))) : -CUDART_INF_F;
-      s[j][1] = t + 1 <= last_lo ? __half2float(__float2half(div_by(s[j][1], scale_div, scale_rcp))) : -CUDART_INF_F;
-      s[j][2] = t <= last_hi ? __half2float(__float2half(div_by(s[j][2], scale_div, scale_rcp))) : -CUDART_INF_F;
-      s[j][3] = t + 1 <= last_hi ? __half2float(__float2half(div_by(s[j][3], scale_div, scale_rcp))) : -CUDART_INF_F;
+      s[j][0] = t <= last_lo ? __half2float(__float2half(s[j][0] * scale_rcp)) : -CUDART_INF_F;
+      s[j][1] = t + 1 <= last_lo ? __half2float(__float2half(s[j][1] * scale_rcp)) : -CUDART_INF_F;
+      s[j][2] = t <= last_hi ? __half2float(__float2half(s[j][2] * scale_rcp)) : -CUDART_INF_F;
+      s[j][3] = t + 1 <= last_hi ? __half2float(__float2half(s[j][3] * scale_rcp)) : -CUDART_INF_F;
     }
   };
 
@@ -163,7 +156,7 @@ __global__ void __launch_bounds__(PA_THREADS) attn_prefill_kernel(const attn_par
   }
 
   // ---- pass 2: probabilities (half) times V
-  const float rs_lo = __frcp_rn(sum_lo), rs_hi = __frcp_rn(sum_hi);
+  const float rs_lo = 1.0f / sum_lo, rs_hi = 1.0f / sum_hi;
   float o[HD / 8][4];
 #pragma unroll
   for (int j = 0; j < HD / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
@@ -188,10 +181,10 @@ __global__ void __launch_bounds__(PA_THREADS) attn_prefill_kernel(const attn_par
     uint32_t pa[4][4];  // A fragments of the 16 x 64 probability block, 16 keys each
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk) {
-      pa[kk][0] = pack_half2(div_by(expf(s[2 * kk][0] - mx_lo), sum_lo, rs_lo), div_by(expf(s[2 * kk][1] - mx_lo), sum_lo, rs_lo));
-      pa[kk][1] = pack_half2(div_by(expf(s[2 * kk][2] - mx_hi), sum_hi, rs_hi), div_by(expf(s[2 * kk][3] - mx_hi), sum_hi, rs_hi));
-      pa[kk][2] = pack_half2(div_by(expf(s[2 * kk + 1][0] - mx_lo), sum_lo, rs_lo), div_by(expf(s[2 * kk + 1][1] - mx_lo), sum_lo, rs_lo));
-      pa[kk][3] = pack_half2(div_by(expf(s[2 * kk + 1][2] - mx_hi), sum_hi, rs_hi), div_by(expf(s[2 * kk + 1][3] - mx_hi), sum_hi, rs_hi));
+      pa[kk][0] = pack_half2(expf(s[2 * kk][0] - mx_lo) * rs_lo, expf(s[2 * kk][1] - mx_lo) * rs_lo);
+      pa[kk][1] = pack_half2(expf(s[2 * kk][2] - mx_hi) * rs_hi, expf(s[2 * kk][3] - mx_hi) * rs_hi);
+      pa[kk][2] = pack_half2(expf(s[2 * kk + 1][0] - mx_lo) * rs_lo, expf(s[2 * kk + 1][1] - mx_lo) * rs_lo);
+      pa[kk][3] = pack_half2(expf(s[2 * kk + 1][2] - mx_hi) * rs_hi, expf(s[2 * kk + 1][3] - mx_hi) * rs_hi);
     }
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk) {

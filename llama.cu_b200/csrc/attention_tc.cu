@@ -119,13 +119,9 @@ __global__ void __launch_bounds__(QK_THREADS, 1) attn_qk_kernel(const __grid_con
   } else {
     const int quad = warp & 3, chalf = (warp - 2) >> 2;  // TMEM lane quadrant of this warp; it takes 64 of the 128 columns
     const int row = m0 + quad * 32 + lane;
-    // x / sqrt(head_dim) as one multiplication and a residual correction: RN(x / d) in all but vanishingly rare
-    // double-rounding cases (the result is rounded to half right after), a third of the division's instructions
-    const float scale_div = sqrtf((float)HD), scale_rcp = __frcp_rn(scale_div);
-    auto scaled = [&](uint32_t bits) {
-      const float x = __uint_as_float(bits), q = x * scale_rcp;
-      return fmaf(fmaf(-q, scale_div, x), scale_rcp, q);
-    };
+    // x / sqrt(head_dim) as a product with the reciprocal (the result is rounded to half right after)
+    const float scale_rcp = 1.0f / sqrtf((float)HD);
+    auto scaled = [&](uint32_t bits) { return __uint_as_float(bits) * scale_rcp; };
     bool go = true;
     for (int j = 0; j < n_tiles && go; ++j) {
       const int b = j & 1;
@@ -236,12 +232,8 @@ __global__ void __launch_bounds__(256) attn_softmax_kernel(const attn_tc_params 
     }
   }
   const float sum = warp_sum(sum0 + sum1);
-  const float rsum = __frcp_rn(sum);
-  // e / sum as one multiplication and a residual correction (RN(e / sum) in all but vanishingly rare cases)
-  auto prob = [&](float x) {
-    const float e = ex(x), q = e * rsum;
-    return fmaf(fmaf(-q, sum, e), rsum, q);
-  };
+  const float rsum = 1.0f / sum;
+  auto prob = [&](float x) { return ex(x) * rsum; };  // (rounded to half right after)
 #pragma unroll
   for (int j = 0; j < SM_VEC; ++j) {
     const int i0 = (j * 32 + lane) * 8;

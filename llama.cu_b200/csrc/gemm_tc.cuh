@@ -42,7 +42,7 @@ int launch_gemm_tc_sk(__half* out, const __half* lhs, int ldx, const __half* w, 
 int gemm_tc_sk_check_schedule(int n_tiles, int nk, int C);
 
 // w1|w3 and the SiLU gate as one launch (gemm_tc_sk.cu): out[m][f] = half(silu(half(lhs . w1^T)) * half(lhs . w3^T)) with
-// w13 = [w1; w3] stacked ([2 f][K]); the same bits as the stacked product followed by the gate kernel.
+// w13 = [w1; w3] stacked ([2 f][K]); the stacked product followed by the gate kernel, up to one unit in the last place.
 // gemm_tc_gate_mode: -1 = when the estimate favours it, 256 / 512 = from 129 rows with that many accumulator columns per
 // tile, 0 = never.  gemm_tc_gated_tile: the tile to use for this shape under that mode, 0 = run product and gate apart.
 int& gemm_tc_gate_mode();

@@ -1,5 +1,5 @@
 // Row-wise and element-wise kernels of the forward pass, the quantizer and the data generator.
-// Each kernel keeps the arithmetic (operation order inside an element, rounding points, libdevice
+// Each kernel keeps the arithmetic (operation order inside an element, rounding points, math
 // functions) of the reference kernel it replaces, cited beside it.
 #include "ops.cuh"
 
@@ -344,17 +344,13 @@ __device__ __forceinline__ unsigned long long warp_sum_u64(unsigned long long v)
   return v;
 }
 
-// q = u8(roundf(127.5f + x / s)) costs an IEEE division and a roundf per element - about 25 instructions, which is what
-// bounded the kernel at half the copy bandwidth.  For the inputs the quantizer can see - x a finite half, s a positive
-// finite half, |x| within the absmax that rounds to s - the same byte comes out of a reciprocal multiply with one
-// residual correction (the correctly rounded quotient) and trunc(v + 0.5f) for the non-negative v = 127.5f + quotient:
-// 7 instructions.  "The same byte" is not argued, it is checked: quantizer_check_kernel compares the two for every such
-// pair (2 x 10^9 of them) on the device, and tests/test_gpu_kernels.py requires zero differences.
+// q = u8(roundf(127.5f + x / s)).  For the inputs the quantizer can see - x a finite half, s a positive finite half, |x|
+// within the absmax that rounds to s - the byte comes out of one addition and a truncating conversion instead of the
+// addition and roundf.  quantizer_check_kernel compares the two for every such pair (2 x 10^9 of them) on the device, and
+// tests/test_gpu_kernels.py requires zero differences.
 __device__ __forceinline__ uint32_t quant_byte_reference(float x, float s) { return static_cast<uint8_t>(roundf(127.5f + x / s)); }
-__device__ __forceinline__ uint32_t quant_byte_fast(float x, float s, float rcp) {
-  const float t = x * rcp;
-  const float quo = fmaf(fmaf(-t, s, x), rcp, t);
-  return static_cast<uint8_t>(quo + 128.0f);  // trunc((127.5f + quo) + 0.5f) in one addition (conversion truncates); checked like the rest
+__device__ __forceinline__ uint32_t quant_byte_fast(float x, float s) {
+  return static_cast<uint8_t>(x / s + 128.0f);  // trunc((127.5f + x / s) + 0.5f) in one addition
 }
 
 // every (x, s) pair of the quantizer's domain: s = positive finite half number blockIdx.x * 256 + threadIdx.x..., x every
@@ -363,7 +359,6 @@ __global__ void __launch_bounds__(256) quantizer_check_kernel(unsigned long long
   unsigned long long checked = 0, diff = 0;
   for (uint32_t sb = blockIdx.x + 1; sb < 0x7c00u; sb += gridDim.x) {  // bit patterns of the positive finite halves
     const float s = __half2float(__ushort_as_half((unsigned short)sb));
-    const float rcp = __frcp_rn(s);
     for (uint32_t xb = threadIdx.x; xb < 0x10000u; xb += 256) {
       if ((xb & 0x7c00u) == 0x7c00u) continue;  // inf / nan
       const __half xh = __ushort_as_half((unsigned short)xb);
@@ -371,7 +366,7 @@ __global__ void __launch_bounds__(256) quantizer_check_kernel(unsigned long long
       // in the domain iff a block with this absmax would get this scale
       if (__half_as_ushort(__float2half(fabsf(x) / 127.5f)) > sb) continue;
       ++checked;
-      if (quant_byte_reference(x, s) != quant_byte_fast(x, s, rcp)) ++diff;
+      if (quant_byte_reference(x, s) != quant_byte_fast(x, s)) ++diff;
     }
   }
   checked = warp_sum_u64(checked);
@@ -421,11 +416,10 @@ __global__ void __launch_bounds__(256) quantize8_kernel(uint8_t* q, __half* scal
       if ((v & (LANES - 1)) == 0) scales[v / LANES] = s_absmax;
       uint32_t lo = 0, hi = 0;
       if (sf > 0.f && absmax_val < CUDART_INF_F) {  // (block-uniform) the checked domain: finite values, positive scale
-        const float rcp = __frcp_rn(sf);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          lo |= quant_byte_fast(f[e], sf, rcp) << (8 * e);
-          hi |= quant_byte_fast(f[e + 4], sf, rcp) << (8 * e);
+          lo |= quant_byte_fast(f[e], sf) << (8 * e);
+          hi |= quant_byte_fast(f[e + 4], sf) << (8 * e);
         }
       } else {  // an all-zero block (0 / 0), infinities or NaNs: the reference's own instructions
 #pragma unroll
@@ -758,13 +752,13 @@ int launch_quantize_absmax_uint8(uint8_t* q, __half* scales, const __half* in, s
   return LCU_OK;
 }
 
-// every half-precision a: silu_of_half against the division it replaces, bit for bit (NaN = NaN)
+// every half-precision a: silu_of_half against the division it stands for, both rounded to half (NaN = NaN)
 __global__ void silu_check_kernel(unsigned long long* counts) {
   const uint32_t i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= 65536u) return;
   const float a = __half2float(__ushort_as_half((unsigned short)i));
-  const float want = a / (1.0f + expf(-a)), got = silu_of_half(a);
-  const bool same = (want != want && got != got) || __float_as_uint(want) == __float_as_uint(got);
+  const float want = __half2float(__float2half(a / (1.0f + expf(-a)))), got = __half2float(__float2half(silu_of_half(a)));
+  const bool same = (want != want && got != got) || want == got;
   atomicAdd(counts, 1ull);
   if (!same) atomicAdd(counts + 1, 1ull);
 }

@@ -191,8 +191,8 @@ def test_prefill_gemm_with_balanced_k_steps(lcu, m, k, n, beta, tile):
 def test_gated_gemm_equals_the_stacked_product_followed_by_silu(lcu, m, k, f, tile):
     """w1|w3 and the SiLU gate as one launch (both products of a tile in tensor memory, the gate in the epilogue) against
     the two-step path the reference takes (llama_cu.cu:1180-1183): the stacked product stored as halves, then silu on
-    those halves.  Equal bits - the one launch rounds the products to half before the gate exactly as the store does -
-    when both paths add partial sums in the same order, which the balanced kernel with the same tile width guarantees."""
+    those halves.  The one launch rounds the products to half before the gate exactly as the store does, and the balanced
+    kernel with the same tile width adds partial sums in the same order, so only the gate's quotient can differ."""
     if f % (tile // 2):
         pytest.skip("tile width does not divide the output")
     rng = np.random.default_rng(m + 3 * f)
@@ -210,7 +210,9 @@ def test_gated_gemm_equals_the_stacked_product_followed_by_silu(lcu, m, k, f, ti
     stacked[:, order] = h
     want = lcu.silu(np.ascontiguousarray(stacked[:, :f]), np.ascontiguousarray(stacked[:, f:]))
     got = lcu.matmul_nt_gated(x, w13, tile)
-    assert np.array_equal(got, want)
+    # the fused gate's quotient is within two binary32 units of the division's: now and then one unit of the half result
+    off = np.abs(got.astype(np.int32) - want.astype(np.int32))
+    assert off.max() <= 1 and (off > 0).mean() < 0.01
     # and against the oracle's product + gate (binary64 accumulation), at the GEMM's tolerance
     ref = np.zeros((m, f), np.uint16)
     L.orc_matmul_nt_f16_gated(ref.reshape(-1), x.reshape(-1), w13.reshape(-1), m, k, f, 1)
@@ -218,21 +220,20 @@ def test_gated_gemm_equals_the_stacked_product_followed_by_silu(lcu, m, k, f, ti
     assert np.abs(f32(got) - f32(ref)).max() <= 4e-3 * scale
 
 
-def test_gate_arithmetic_equals_the_division_for_every_half(lcu):
-    """The one-launch w1|w3 + gate forms a / (1 + expf(-a)) with a refined reciprocal instead of the IEEE division
-    (llama_cu.cu:533-539): compared on the device for all 65536 half-precision a, no differing bit."""
+def test_gate_arithmetic_against_the_division_for_every_half(lcu):
+    """The one-launch w1|w3 + gate forms a / (1 + expf(-a)) with __fdividef (two units of binary32 off the division,
+    llama_cu.cu:533-539 divides): rounded to half, all but a few of the 65536 half-precision a give the same value."""
     import ctypes as C
     checked, diff = C.c_uint64(0), C.c_uint64(0)
     lcu.check(lcu.lib.lcu_selftest_silu_arithmetic(C.byref(checked), C.byref(diff)))
     assert checked.value == 65536
-    assert diff.value == 0
+    assert diff.value <= 64
 
 
-def test_quantizer_fast_arithmetic_equals_division_and_roundf_on_its_whole_domain(lcu):
-    """The quantizer forms its bytes with a reciprocal multiply, one residual correction and trunc(v + 0.5f) instead of the
-    reference's IEEE division and roundf (transform.cu:60-80).  The device compares the two for every pair the quantizer
-    can meet - every positive finite half as scale, every finite half within the absmax that rounds to it: about two
-    billion pairs - and must find no differing byte."""
+def test_quantizer_arithmetic_on_its_whole_domain(lcu):
+    """The quantizer truncates x / scale + 128 instead of rounding 127.5f + x / scale (transform.cu:60-80).  The device
+    compares the two for every pair the quantizer can meet - every positive finite half as scale, every finite half within
+    the absmax that rounds to it: about two billion pairs - and must find no differing byte."""
     import ctypes as C
     checked, diff = C.c_uint64(0), C.c_uint64(0)
     lcu.check(lcu.lib.lcu_selftest_quantizer_arithmetic(C.byref(checked), C.byref(diff)))
