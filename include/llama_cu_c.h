@@ -127,6 +127,23 @@ int lcu_synth_fill_f16(void* out_dev, uint64_t n, uint64_t seed, const char* nam
 int lcu_model_create(const void* params40, const int* layer_gpus, void** model_out);
 /* llama_model::load, llama_cu.cu:987-997: reads <dir>/params and the tensor files (llama_cu.cu:929-984) */
 int lcu_model_load(const char* dir, const int* layer_gpus, void** model_out);
+/* Block models (no counterpart in the reference): a directory with config.json, whose "architecture" names one of
+ * lcu_architectures(), and model.safetensors.  lcu_model_load takes such a directory as well (bfloat16); here dtype picks the
+ * number format: 0 bfloat16 weights, activations and caches with binary32 residual, norms, scores and recurrent state,
+ * 1 binary32 throughout.  Weight directories of the LLaMA family: dtype 0 only.  A block model lives on one GPU
+ * (layer_gpus[0], or the current device). */
+int lcu_model_load_as(const char* dir, const int* layer_gpus, int dtype, void** model_out);
+/* a block model with uninitialised (zero) weights from configuration text, for lcu_model_fill_synthetic; decay_rank: the
+ * low-rank size of the wkv decays, which a file gives by its tensor shapes */
+int lcu_model_create_from_config(const char* config_text, int dtype, int decay_rank, void** model_out);
+/* host only: reads configuration text; out8 = vocab, width, layers, layer runs, streams, bigram buckets, 0, 0 */
+int lcu_config_summary(const char* config_text, int32_t* out8);
+/* host only: the layer of every layer run in order (the first `capacity` of them); returns their number, or -status */
+int lcu_config_runs(const char* config_text, int32_t* runs_out, int capacity);
+/* names of the block architectures, separated by ", " */
+int lcu_architectures(char* out, int capacity);
+int lcu_model_shape(void* model, int32_t* vocab, int32_t* width, int32_t* layers);
+const char* lcu_model_family(void* model); /* "llama" or the architecture's name */
 /* seeded synthetic weights in place of a checkpoint (matrices scale*z, norm weights 1.0) */
 int lcu_model_fill_synthetic(void* model, uint64_t seed, float scale);
 /* writes the model as a weight directory in the reference's layout (extract.py:16-41, transform.cu:179-261) */
@@ -169,6 +186,10 @@ uint64_t lcu_context_memory_usage(void* ctx);
 int lcu_context_tokens_left(void* ctx);
 /* llama_context::next_token(new_tokens), llama_cu.cu:1073-1210: host token ids in, greedy token out */
 int lcu_context_next_token(void* ctx, const int16_t* tokens_host, int n_tokens, int* token_out);
+/* The same step for callers that want logits: binary32 logits of the tokens at want_host[0 .. n_want) (places among the
+ * n_tokens given), [n_want][n_vocab] in that order.  LLaMA contexts form the last token's logits only.  token_out may be
+ * NULL: no token is picked then after a step of several tokens. */
+int lcu_context_step(void* ctx, const int16_t* tokens_host, int n_tokens, const int32_t* want_host, int n_want, float* logits_host, int* token_out);
 /* n_steps greedy single-token steps chained on the device (the loop of main.cpp:80-100 without the
  * per-token host round trip); tokens_host_out[n_steps]; *ms_out = device time of the loop */
 int lcu_context_decode_chained(void* ctx, int16_t first_token, int n_steps, int16_t* tokens_host_out, float* ms_out);

@@ -6,6 +6,7 @@ fallback: importing works anywhere, but every compute call needs an sm_100a devi
 missing shared library raises at import time.
 """
 import ctypes as C
+import json
 import os
 import struct
 
@@ -63,6 +64,14 @@ _SIG = {
     "lcu_bench_matmul_f16": (C.c_int, [vp, vp, vp, C.c_int, C.c_int, C.c_int, C.c_int, C.POINTER(C.c_float)]),
     "lcu_synth_fill_f16": (C.c_int, [vp, C.c_uint64, C.c_uint64, C.c_char_p, C.c_float, C.c_uint64, vp]),
     "lcu_model_create": (C.c_int, [vp, vp, C.POINTER(vp)]),
+    "lcu_model_load_as": (C.c_int, [C.c_char_p, vp, C.c_int, C.POINTER(vp)]),
+    "lcu_model_create_from_config": (C.c_int, [C.c_char_p, C.c_int, C.c_int, C.POINTER(vp)]),
+    "lcu_config_summary": (C.c_int, [C.c_char_p, vp]),
+    "lcu_config_runs": (C.c_int, [C.c_char_p, vp, C.c_int]),
+    "lcu_architectures": (C.c_int, [C.c_char_p, C.c_int]),
+    "lcu_model_shape": (C.c_int, [vp, vp, vp, vp]),
+    "lcu_model_family": (C.c_char_p, [vp]),
+    "lcu_context_step": (C.c_int, [vp, vp, C.c_int, vp, C.c_int, vp, C.POINTER(C.c_int)]),
     "lcu_model_load": (C.c_int, [C.c_char_p, vp, C.POINTER(vp)]),
     "lcu_model_fill_synthetic": (C.c_int, [vp, C.c_uint64, C.c_float]),
     "lcu_model_save": (C.c_int, [vp, C.c_char_p]),
@@ -121,6 +130,25 @@ class LcuError(RuntimeError):
 def check(rc):
     if rc != 0:
         raise LcuError(f"status {rc}: {lib.lcu_last_error().decode(errors='replace')}")
+
+
+DTYPES = {"bfloat16": 0, "float32": 1}  # number formats of the block models
+
+
+def architectures():
+    """Names of the block architectures config.json may give."""
+    buf = C.create_string_buffer(4096)
+    check(lib.lcu_architectures(buf, len(buf)))
+    return buf.value.decode().split(", ")
+
+
+def config_runs(config):
+    """Layer of every layer run, in order, as the library reads the configuration (host only)."""
+    out = np.empty(1 << 16, np.int32)
+    n = lib.lcu_config_runs(json.dumps(config).encode(), _ptr(out), out.size)
+    if n < 0:
+        check(-n)
+    return out[:n].tolist()
 
 
 PARAMS_FMT = "<QIIIIIIfBBH"  # the 40-byte params record
@@ -298,14 +326,31 @@ class Model:
         return m
 
     @classmethod
-    def load(cls, path, layer_gpus=None):
+    def load(cls, path, layer_gpus=None, dtype="bfloat16"):
+        """A weight directory of the LLaMA family, or a block model's (config.json + model.safetensors; dtype "bfloat16" or
+        "float32")."""
         h = vp()
         lg = None if layer_gpus is None else _ptr(np.ascontiguousarray(layer_gpus, np.int32))
-        check(lib.lcu_model_load(path.encode(), lg, C.byref(h)))
-        raw = C.create_string_buffer(40)
-        lib.lcu_model_params(h, raw)
-        f = struct.unpack(PARAMS_FMT, raw.raw)
-        return cls(h, f[6], f[2])
+        check(lib.lcu_model_load_as(path.encode(), lg, DTYPES[dtype], C.byref(h)))
+        return cls._of(h)
+
+    @classmethod
+    def from_config(cls, config, dtype="bfloat16", seed=1234, scale=0.02, decay_rank=64):
+        """A block model with seeded synthetic weights; config is the dictionary a config.json holds."""
+        h = vp()
+        check(lib.lcu_model_create_from_config(json.dumps(config).encode(), DTYPES[dtype], decay_rank, C.byref(h)))
+        m = cls._of(h)
+        check(lib.lcu_model_fill_synthetic(h, seed, scale))
+        return m
+
+    @classmethod
+    def _of(cls, h):
+        v, w = C.c_int32(0), C.c_int32(0)
+        check(lib.lcu_model_shape(h, C.byref(v), C.byref(w), None))
+        return cls(h, v.value, w.value)
+
+    def family(self):
+        return lib.lcu_model_family(self.handle).decode()
 
     def params(self):
         raw = C.create_string_buffer(40)
@@ -353,6 +398,16 @@ class Context:
         out = C.c_int(0)
         check(lib.lcu_context_next_token(self.handle, _ptr(t), len(t), C.byref(out)))
         return out.value
+
+    def step(self, tokens, want=(), token=False):
+        """Feeds tokens; returns the binary32 logits at the places `want` among them [len(want), n_vocab] (and the greedy
+        or sampled next token when asked for)."""
+        t = np.ascontiguousarray(np.asarray(tokens, np.int16))
+        w = np.ascontiguousarray(np.asarray(want, np.int32))
+        out = np.empty((len(w), self.model.n_vocab), np.float32)
+        nxt = C.c_int(0)
+        check(lib.lcu_context_step(self.handle, _ptr(t), len(t), _ptr(w), len(w), _ptr(out), C.byref(nxt) if token else None))
+        return (out, nxt.value) if token else out
 
     def decode_chained(self, first_token, n_steps):
         toks = np.empty(n_steps, np.int16)

@@ -1,0 +1,574 @@
+// Mixers of the block models: attention over a sliding window and pooled blocks, linear recurrences, and the fused
+// one-token launch of all branches of a mixer.
+#include <algorithm>
+
+#include <math_constants.h>
+
+#include "block_ops.cuh"
+#include "elem.cuh"
+
+namespace lcu {
+namespace {
+
+constexpr int MX_THREADS = 256;
+constexpr int PART_FLOATS = 4096;  // partial sums of the value pass (groups x value columns)
+
+__host__ __device__ __forceinline__ int pow2_at_least(int n) {
+  int p = 1;
+  while (p < n) p *= 2;
+  return p;
+}
+
+// what position i sees: blocks 0 .. blocks-1 and tokens lo .. i
+__host__ __device__ __forceinline__ void window_of(int i, int window, int pool, int& lo, int& blocks) {
+  lo = i + 1 > window ? i + 1 - window : 0;
+  const int past = i + 1 - window;  // positions that have left the window
+  blocks = pool > 0 && past > 0 ? past / pool : 0;
+}
+
+__device__ __forceinline__ float block_max(float v, float* red) {
+  v = warp_max(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float m = red[0];
+#pragma unroll
+  for (int w = 1; w < MX_THREADS / 32; ++w) m = fmaxf(m, red[w]);
+  return m;
+}
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float s = 0.f;
+#pragma unroll
+  for (int w = 0; w < MX_THREADS / 32; ++w) s += red[w];
+  return s;
+}
+
+// ------------------------------------------------------------------ attention of one query row and head
+// `rank` of `C` CTAs takes a slice of the visible keys.  The row's own key and value come from `cur_k` / `cur_v` (shared
+// memory copies) when given, else from the cache.  Leaves max, sum and the unnormalised value row in res[0], res[1],
+// res[2 ..].  Shared memory: q [ldk], scores [slice], part [PART_FLOATS].
+template <typename T>
+__device__ void attend_slice(const attn_rows<T>& p, const T* q_row, int head, int pos, int rank, int C, const T* cur_k, const T* cur_v, float* q,
+                             float* sc, float* part, float* red, float* res) {
+  constexpr int VEC = 16 / sizeof(T);
+  const int tid = threadIdx.x;
+  const int kvh = head / (p.heads / p.kv_heads);
+  const int ldk = p.cache.ldk, ldv = p.cache.ldv;
+  const T* kc = p.cache.k + (size_t)kvh * p.cache.ctx_len * ldk;
+  const T* vc = p.cache.v + (size_t)kvh * p.cache.ctx_len * ldv;
+  const T* kp = p.cache.kp + (size_t)kvh * p.cache.n_blocks * ldk;
+  const T* vp = p.cache.vp + (size_t)kvh * p.cache.n_blocks * ldv;
+  int lo, blocks;
+  window_of(pos, p.window, p.pool, lo, blocks);
+  const int total = blocks + pos + 1 - lo;
+  const int t0 = (int)((long long)total * rank / C), n = (int)((long long)total * (rank + 1) / C) - t0;
+  for (int d = tid; d < ldk; d += MX_THREADS) q[d] = d < p.dim ? to_f(q_row[head * p.dim + d]) : 0.f;
+  __syncthreads();
+  auto key_at = [&](int t) -> const T* {
+    if (t < blocks) return kp + (size_t)t * ldk;
+    const int j = lo + t - blocks;
+    return cur_k && j == pos ? cur_k : kc + (size_t)j * ldk;
+  };
+  auto value_at = [&](int t) -> const T* {
+    if (t < blocks) return vp + (size_t)t * ldv;
+    const int j = lo + t - blocks;
+    return cur_v && j == pos ? cur_v : vc + (size_t)j * ldv;
+  };
+  // scores: lpk lanes per key
+  {
+    const int lpk = min(32, pow2_at_least((ldk + VEC - 1) / VEC)), groups = MX_THREADS / lpk, grp = tid / lpk, sub = tid % lpk;
+    constexpr int U = 4;
+    const int rounds = (n + groups * U - 1) / (groups * U);  // (the same for every lane: the shuffles below are warp-wide)
+    for (int rd = 0; rd < rounds; ++rd) {
+      float s[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        s[u] = 0.f;
+        const int t = (rd * U + u) * groups + grp;
+        if (t < n) {
+          const T* k = key_at(t0 + t);
+          for (int d = sub * VEC; d < ldk; d += lpk * VEC) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(k + d);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) s[u] = fmaf(q[d + e], to_f(reinterpret_cast<const T*>(&raw)[e]), s[u]);
+          }
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        for (int o = lpk >> 1; o > 0; o >>= 1) s[u] += __shfl_xor_sync(0xffffffffu, s[u], o);
+        const int t = (rd * U + u) * groups + grp;
+        if (sub == 0 && t < n) sc[t] = s[u] * p.scale;
+      }
+    }
+  }
+  __syncthreads();
+  float mx = -CUDART_INF_F;
+  for (int t = tid; t < n; t += MX_THREADS) mx = fmaxf(mx, sc[t]);
+  mx = block_max(mx, red);
+  float sum = 0.f;
+  for (int t = tid; t < n; t += MX_THREADS) {
+    const float e = expf(sc[t] - mx);
+    sc[t] = e;
+    sum += e;
+  }
+  sum = block_sum(sum, red);  // (its barriers also publish the exponentials)
+  // values: lpv lanes per row of values, groups of them walk the keys
+  const int lpv = min(32, pow2_at_least((ldv + VEC - 1) / VEC)), groups = MX_THREADS / lpv, grp = tid / lpv, sub = tid % lpv;
+  for (int d0 = 0; d0 < ldv; d0 += lpv * VEC) {
+    const int d = d0 + sub * VEC;
+    float acc[VEC] = {};
+    if (d < ldv) {
+#pragma unroll 4
+      for (int t = grp; t < n; t += groups) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(value_at(t0 + t) + d);
+        const float w = sc[t];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) acc[e] = fmaf(w, to_f(reinterpret_cast<const T*>(&raw)[e]), acc[e]);
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) part[(grp * lpv + sub) * VEC + e] = acc[e];
+    __syncthreads();
+    for (int j = tid; j < lpv * VEC && d0 + j < p.vdim; j += MX_THREADS) {
+      float v = 0.f;
+      for (int g = 0; g < groups; ++g) v += part[g * lpv * VEC + j];
+      res[2 + d0 + j] = v;
+    }
+  }
+  if (tid == 0) {
+    res[0] = n > 0 ? mx : -CUDART_INF_F;
+    res[1] = n > 0 ? sum : 0.f;
+  }
+  __syncthreads();
+}
+
+// rows of a pass, one CTA per (row, head); keys and blocks are in the cache already
+template <typename T>
+__global__ void __launch_bounds__(MX_THREADS) window_rows_kernel(const attn_rows<T> p, int pos0, int max_keys) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float red[MX_THREADS / 32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int head = blockIdx.x, r = blockIdx.y;
+  float* q = sm;
+  float* part = q + p.cache.ldk;
+  float* res = part + PART_FLOATS;
+  float* sc = res + 2 + round_up_dev(p.vdim + 2, 4);
+  attend_slice(p, p.q + (size_t)r * p.ld, head, pos0 + r, 0, 1, (const T*)nullptr, (const T*)nullptr, q, sc, part, red, res);
+  const float inv = p.out_scale / res[1];
+  for (int d = threadIdx.x; d < p.vdim; d += MX_THREADS) p.out[(size_t)r * p.ldo + head * p.vdim + d] = from_f<T>(res[2 + d] * inv);
+}
+
+// new rows of k and v into the cache
+template <typename T>
+__global__ void __launch_bounds__(256) window_append_kernel(const attn_rows<T> p, int m, int pos0) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.x;
+  for (int i = threadIdx.x; i < p.kv_heads * p.dim; i += 256) {
+    const int g = i / p.dim, d = i - g * p.dim;
+    p.cache.k[((size_t)g * p.cache.ctx_len + pos0 + r) * p.cache.ldk + d] = p.k[(size_t)r * p.ld + i];
+  }
+  for (int i = threadIdx.x; i < p.kv_heads * p.vdim; i += 256) {
+    const int g = i / p.vdim, d = i - g * p.vdim;
+    p.cache.v[((size_t)g * p.cache.ctx_len + pos0 + r) * p.cache.ldv + d] = p.v[(size_t)r * p.ld + i];
+  }
+}
+
+// mean of the cached rows of one block
+template <typename T>
+__device__ __forceinline__ void pool_block(const T* rows, int ld, int pool, const T* last, T* out, int dim) {
+  for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+    float s = 0.f;
+    for (int j = 0; j < pool; ++j) s += to_f(last && j == pool - 1 ? last[d] : rows[(size_t)j * ld + d]);
+    out[d] = from_f<T>(s / (float)pool);
+  }
+}
+template <typename T>
+__global__ void __launch_bounds__(128) window_pool_kernel(const attn_rows<T> p, int first_block) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int b = first_block + blockIdx.x, g = blockIdx.y;
+  const size_t row = (size_t)g * p.cache.ctx_len + (size_t)b * p.pool, dst = (size_t)g * p.cache.n_blocks + b;
+  pool_block(p.cache.k + row * p.cache.ldk, p.cache.ldk, p.pool, (const T*)nullptr, p.cache.kp + dst * p.cache.ldk, p.dim);
+  pool_block(p.cache.v + row * p.cache.ldv, p.cache.ldv, p.pool, (const T*)nullptr, p.cache.vp + dst * p.cache.ldv, p.vdim);
+}
+
+// ------------------------------------------------------------------ recurrences over rows
+// One CTA owns COLS = 128 / G value columns of one head; G neighbouring lanes share a column, each holding KC of its state
+// entries in registers for the whole pass.  Rows come through shared memory SC_ROWS at a time.  Lane `sub` of a column holds
+// channels (c / 4) * 4 G + 4 sub + c % 4, so that a warp reads its row vectors as contiguous 16-byte pieces.
+constexpr int SC_THREADS = 128;
+constexpr int SC_ROWS = 16;
+
+template <typename T, int KC, bool WKV>
+__global__ void __launch_bounds__(SC_THREADS) scan_kernel(const scan_rows<T> p, int m, int pos0, int G) {
+  extern __shared__ __align__(16) float sm[];
+  const int dimp = G * KC, cols = SC_THREADS / G;
+  float* qs = sm;                       // [SC_ROWS][dimp]
+  float* ks = qs + SC_ROWS * dimp;      // [SC_ROWS][dimp]
+  float* ws = ks + SC_ROWS * dimp;      // [SC_ROWS][dimp], wkv
+  float* vs = ws + (WKV ? SC_ROWS * dimp : 0);  // [SC_ROWS][cols]
+  float* os = vs + SC_ROWS * cols;      // [SC_ROWS][cols]
+  const int tid = threadIdx.x, sub = tid % G, col = tid / G;
+  const int head = blockIdx.x, v0 = blockIdx.y * cols, D = p.dim, DV = p.vdim;
+  pdl_launch_dependents();
+  pdl_wait();
+  float S[KC], u[KC];
+  float* st = p.state + (size_t)head * D * DV;
+  const bool live = v0 + col < DV;
+#pragma unroll
+  for (int c = 0; c < KC; ++c) {
+    const int i = (c >> 2) * 4 * G + 4 * sub + (c & 3);
+    S[c] = pos0 > 0 && live && i < D ? st[(size_t)i * DV + v0 + col] : 0.f;
+    u[c] = WKV && i < D ? p.u[head * D + i] : 0.f;
+  }
+  const float dec = WKV ? 0.f : p.decay[head];
+  for (int i = tid; i < SC_ROWS * dimp; i += SC_THREADS) {  // (channels past the head's size stay zero)
+    qs[i] = 0.f;
+    ks[i] = 0.f;
+    if (WKV) ws[i] = 0.f;
+  }
+  const int half = p.rot_dims >> 1;
+  for (int r0 = 0; r0 < m; r0 += SC_ROWS) {
+    const int nr = min(SC_ROWS, m - r0);
+    __syncthreads();
+    for (int i = tid; i < nr * D; i += SC_THREADS) {
+      const int r = i / D, d = i - r * D, row = r0 + r;
+      const T* qr = p.q + (size_t)row * p.ldq + head * D;
+      const T* kr = p.k + (size_t)row * p.ldk + head * D;
+      float qv = to_f(qr[d]), kv = to_f(kr[d]);
+      if (!WKV) {
+        if (d < p.rot_dims) {
+          const bool low = d < half;
+          const float2 cs = p.rope[(size_t)(pos0 + row) * half + (low ? d : d - half)];
+          const int pd = low ? d + half : d - half;
+          const float qo = to_f(qr[pd]), ko = to_f(kr[pd]);
+          qv = low ? qv * cs.x - qo * cs.y : qv * cs.x + qo * cs.y;
+          kv = low ? kv * cs.x - ko * cs.y : kv * cs.x + ko * cs.y;
+        }
+        kv *= p.kscale;
+      } else {
+        ws[r * dimp + d] = p.w[(size_t)row * p.heads * D + head * D + d];
+      }
+      qs[r * dimp + d] = qv;
+      ks[r * dimp + d] = kv;
+    }
+    for (int i = tid; i < nr * cols; i += SC_THREADS) {
+      const int r = i / cols, j = i - r * cols;
+      vs[i] = v0 + j < DV ? to_f(p.v[(size_t)(r0 + r) * p.ldv + head * DV + v0 + j]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 4
+    for (int r = 0; r < nr; ++r) {
+      const float v = vs[r * cols + col];
+      float o = 0.f;
+#pragma unroll
+      for (int c4 = 0; c4 < KC / 4; ++c4) {
+        const int at = r * dimp + c4 * 4 * G + 4 * sub;
+        const float4 q4 = *reinterpret_cast<const float4*>(qs + at), k4 = *reinterpret_cast<const float4*>(ks + at);
+        float4 w4 = make_float4(dec, dec, dec, dec);
+        if (WKV) w4 = *reinterpret_cast<const float4*>(ws + at);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int c = c4 * 4 + e;
+          const float q = reinterpret_cast<const float*>(&q4)[e], k = reinterpret_cast<const float*>(&k4)[e], w = reinterpret_cast<const float*>(&w4)[e];
+          const float kv = k * v;
+          if (WKV) {
+            o = fmaf(q, fmaf(u[c], kv, S[c]), o);
+            S[c] = fmaf(w, S[c], kv);
+          } else {
+            S[c] = fmaf(w, S[c], kv);
+            o = fmaf(q, S[c], o);
+          }
+        }
+      }
+      for (int s = G >> 1; s > 0; s >>= 1) o += __shfl_xor_sync(0xffffffffu, o, s);
+      if (sub == 0) os[r * cols + col] = o;
+    }
+    __syncthreads();
+    for (int i = tid; i < nr * cols; i += SC_THREADS) {
+      const int r = i / cols, j = i - r * cols;
+      if (v0 + j < DV) p.out[(size_t)(r0 + r) * p.ldo + head * DV + v0 + j] = os[i];
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < KC; ++c) {
+    const int i = (c >> 2) * 4 * G + 4 * sub + (c & 3);
+    if (live && i < D) st[(size_t)i * DV + v0 + col] = S[c];
+  }
+}
+
+template <typename T, int KC, bool WKV>
+int launch_scan_one(const scan_rows<T>& p, int m, int pos0, cudaStream_t stream) {
+  const int G = pow2_at_least((p.dim + KC - 1) / KC);
+  LCU_REQUIRE(G <= 32, "scan: head size %d", p.dim);
+  const int cols = SC_THREADS / G;
+  const size_t smem = (size_t)SC_ROWS * ((WKV ? 3 : 2) * G * KC + 2 * cols) * sizeof(float);
+  static bool attr_done[16] = {};
+  int dev = 0;
+  LCU_CUDA(cudaGetDevice(&dev));
+  if (dev < 16 && !attr_done[dev]) {
+    LCU_CUDA(cudaFuncSetAttribute((scan_kernel<T, KC, WKV>), cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+    attr_done[dev] = true;
+  }
+  LCU_CUDA(launch_after(scan_kernel<T, KC, WKV>, dim3(p.heads, (p.vdim + cols - 1) / cols), dim3(SC_THREADS), smem, stream, p, m, pos0, G));
+  return LCU_OK;
+}
+
+// ------------------------------------------------------------------ one token, all branches
+constexpr int ST_CLUSTER = 8;
+
+// sum over the cluster of a value every thread of a CTA holds; `slot` is a shared float that stays valid until the next
+// cluster barrier
+__device__ __forceinline__ float cluster_total(float v, float* slot) {
+  if (threadIdx.x == 0) *slot = v;
+  cluster_sync();
+  float t = 0.f;
+#pragma unroll
+  for (int r = 0; r < ST_CLUSTER; ++r) t += ld_dsmem_f32(mapa(smem_u32(slot), r));
+  return t;
+}
+
+template <typename T>
+__device__ void step_attention(const step_branch<T>& b, int head, int rank, int pos, float* sm, float* red) {
+  const attn_rows<T>& p = b.attn;
+  const int tid = threadIdx.x, per = p.heads / p.kv_heads, kvh = head / per;
+  const int ldk = p.cache.ldk, ldv = p.cache.ldv;
+  T* cur_k = reinterpret_cast<T*>(sm);  // [ldk], [ldv]: the token's key and value as the cache will hold them
+  T* cur_v = cur_k + ldk;
+  float* q = sm + ldk + ldv;
+  float* part = q + ldk;
+  float* res = part + PART_FLOATS;
+  float* sc = res + 2 + round_up_dev(p.vdim + 2, 4);
+  for (int d = tid; d < ldk; d += MX_THREADS) cur_k[d] = d < p.dim ? p.k[kvh * p.dim + d] : from_f<T>(0.f);
+  for (int d = tid; d < ldv; d += MX_THREADS) cur_v[d] = d < p.vdim ? p.v[kvh * p.vdim + d] : from_f<T>(0.f);
+  __syncthreads();
+  attend_slice(p, p.q, head, pos, rank, ST_CLUSTER, cur_k, cur_v, q, sc, part, red, res);
+  // the first query head of a group keeps the token: its cache rows, and the means of the block it completes (which no
+  // position sees before the next step)
+  if (head % per == 0 && rank == 0) {
+    const size_t row = (size_t)kvh * p.cache.ctx_len + pos;
+    for (int d = tid; d < p.dim; d += MX_THREADS) p.cache.k[row * ldk + d] = cur_k[d];
+    for (int d = tid; d < p.vdim; d += MX_THREADS) p.cache.v[row * ldv + d] = cur_v[d];
+    if (p.pool > 0 && (pos + 1) % p.pool == 0) {
+      const size_t first = row - (p.pool - 1), dst = (size_t)kvh * p.cache.n_blocks + pos / p.pool;
+      pool_block(p.cache.k + first * ldk, ldk, p.pool, cur_k, p.cache.kp + dst * ldk, p.dim);
+      pool_block(p.cache.v + first * ldv, ldv, p.pool, cur_v, p.cache.vp + dst * ldv, p.vdim);
+    }
+  }
+  cluster_sync();
+  float mx = -CUDART_INF_F, sum = 0.f, f[ST_CLUSTER];
+#pragma unroll
+  for (int r = 0; r < ST_CLUSTER; ++r) mx = fmaxf(mx, ld_dsmem_f32(mapa(smem_u32(res), r)));
+#pragma unroll
+  for (int r = 0; r < ST_CLUSTER; ++r) {
+    const float m = ld_dsmem_f32(mapa(smem_u32(res), r));
+    f[r] = m > -CUDART_INF_F ? expf(m - mx) : 0.f;
+    if (f[r] > 0.f) sum += f[r] * ld_dsmem_f32(mapa(smem_u32(res + 1), r));
+  }
+  const float inv = p.out_scale / sum;
+  const int d1 = p.vdim * (rank + 1) / ST_CLUSTER;
+  for (int d = p.vdim * rank / ST_CLUSTER + tid; d < d1; d += MX_THREADS) {
+    float v = 0.f;
+#pragma unroll
+    for (int r = 0; r < ST_CLUSTER; ++r)
+      if (f[r] > 0.f) v += f[r] * ld_dsmem_f32(mapa(smem_u32(res + 2 + d), r));
+    b.out[head * p.vdim + d] = from_f<T>(v * inv);
+  }
+  cluster_sync();
+}
+
+template <typename T, bool WKV>
+__device__ void step_recurrence(const step_branch<T>& b, int head, int rank, int pos, float* sm, float* red) {
+  const scan_rows<T>& p = b.scan;
+  const int tid = threadIdx.x, D = p.dim, DV = p.vdim;
+  float* q = sm;
+  float* k = q + D;
+  float* w = k + D;        // wkv: decays
+  float* part = w + D;     // [MX_THREADS]
+  float* lows = part + MX_THREADS;
+  __shared__ float s_slot;
+  const int half = p.rot_dims >> 1;
+  for (int d = tid; d < D; d += MX_THREADS) {
+    const T *qr = p.q + head * D, *kr = p.k + head * D;
+    float qv = to_f(qr[d]), kv = to_f(kr[d]);
+    if (!WKV) {
+      if (d < p.rot_dims) {
+        const bool low = d < half;
+        const float2 cs = p.rope[(size_t)pos * half + (low ? d : d - half)];
+        const int pd = low ? d + half : d - half;
+        const float qo = to_f(qr[pd]), ko = to_f(kr[pd]);
+        qv = low ? qv * cs.x - qo * cs.y : qv * cs.x + qo * cs.y;
+        kv = low ? kv * cs.x - ko * cs.y : kv * cs.x + ko * cs.y;
+      }
+      kv *= p.kscale;
+    }
+    q[d] = qv;
+    k[d] = kv;
+  }
+  if (WKV) {
+    for (int j = tid; j < b.rank; j += MX_THREADS) lows[j] = tanhf(b.low[j]);
+    __syncthreads();
+    const int ch_all = p.heads * D;
+    const int ng = max(1, MX_THREADS / D), grp = tid / D, c0 = tid - grp * D;
+    if (ng > 1) {  // groups of threads share the rank
+      float a = 0.f;
+      if (grp < ng)
+        for (int j = grp; j < b.rank; j += ng) a = fmaf(b.w2t[(size_t)j * ch_all + head * D + c0], lows[j], a);
+      part[tid] = a;
+      __syncthreads();
+      if (tid < D) {
+        float z = b.w0[head * D + tid];
+        for (int g = 0; g < ng; ++g) z += part[g * D + tid];
+        w[tid] = expf(-expf(z));
+      }
+    } else {
+      for (int c = tid; c < D; c += MX_THREADS) {
+        float z = b.w0[head * D + c];
+        for (int j = 0; j < b.rank; ++j) z = fmaf(b.w2t[(size_t)j * ch_all + head * D + c], lows[j], z);
+        w[c] = expf(-expf(z));
+      }
+    }
+  }
+  __syncthreads();
+  const int v0 = DV * rank / ST_CLUSTER, nv = DV * (rank + 1) / ST_CLUSTER - v0;  // (at most 64 columns)
+  float* st = p.state + (size_t)head * D * DV;
+  const float dec = WKV ? 0.f : p.decay[head];
+  const float* u = WKV ? p.u + head * D : nullptr;
+  float o = 0.f;
+  if (nv > 0) {
+    const int ng = MX_THREADS / nv, grp = tid / nv, j = tid - grp * nv;
+    float acc = 0.f;
+    if (grp < ng) {
+      const float v = to_f(p.v[head * DV + v0 + j]);
+#pragma unroll 4
+      for (int i = grp; i < D; i += ng) {
+        float* s = st + (size_t)i * DV + v0 + j;
+        float S = pos > 0 ? *s : 0.f;
+        const float kv = k[i] * v;
+        if (WKV) {
+          acc = fmaf(q[i], fmaf(u[i], kv, S), acc);
+          S = fmaf(w[i], S, kv);
+        } else {
+          S = fmaf(dec, S, kv);
+          acc = fmaf(q[i], S, acc);
+        }
+        *s = S;
+      }
+    }
+    part[tid] = acc;
+    __syncthreads();
+    if (tid < nv)
+      for (int g = 0; g < ng; ++g) o += part[g * nv + tid];
+  }
+  const float ss = cluster_total(block_sum(o * o, red), &s_slot);
+  const float inv = 1.0f / sqrtf(ss / (float)DV + b.eps);
+  if (tid < nv) {
+    const int c = head * DV + v0 + tid;
+    float v = o * inv;
+    if (b.norm) v *= b.norm[c];
+    b.out[c] = from_f<T>(v * silu_f(to_f(b.g[c])) * b.out_scale);
+  }
+  cluster_sync();
+}
+
+template <typename T>
+__global__ void __launch_bounds__(MX_THREADS) mixer_step_kernel(const __grid_constant__ mixer_step<T> p) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float red[MX_THREADS / 32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int cl = blockIdx.x / ST_CLUSTER, rank = blockIdx.x % ST_CLUSTER;
+  const int bi = p.n_branches > 1 && cl >= p.b[1].first ? 1 : 0;
+  const step_branch<T>& b = p.b[bi];
+  const int head = cl - b.first, pos = *p.pos;
+  if (b.kind == BRANCH_WINDOW_ATTN) step_attention(b, head, rank, pos, sm, red);
+  else if (b.kind == BRANCH_RETENTION) step_recurrence<T, false>(b, head, rank, pos, sm, red);
+  else step_recurrence<T, true>(b, head, rank, pos, sm, red);
+}
+
+template <typename T>
+size_t attention_smem(const attn_rows<T>& p, int keys, bool step) {
+  return ((step ? p.cache.ldk + p.cache.ldv : 0) + p.cache.ldk + PART_FLOATS + 2 + round_up(p.vdim + 2, 4) + keys + 8) * sizeof(float);
+}
+template <typename T>
+int most_keys(const attn_rows<T>& p, int last_pos) {
+  int lo, blocks;
+  window_of(last_pos, p.window, p.pool, lo, blocks);
+  return blocks + std::min(p.window, last_pos + 1);
+}
+
+}  // namespace
+
+template <typename T>
+int launch_window_append(const attn_rows<T>& p, int m, int pos0, cudaStream_t stream) {
+  LCU_REQUIRE(pos0 >= 0 && pos0 + m <= p.cache.ctx_len, "window attention: rows %d..%d outside the cache of %d", pos0, pos0 + m, p.cache.ctx_len);
+  LCU_CUDA(launch_after(window_append_kernel<T>, dim3(m), dim3(256), 0, stream, p, m, pos0));
+  if (p.pool > 0) {
+    const int b0 = pos0 / p.pool, b1 = (pos0 + m) / p.pool;
+    if (b1 > b0) LCU_CUDA(launch_after(window_pool_kernel<T>, dim3(b1 - b0, p.kv_heads), dim3(128), 0, stream, p, b0));
+  }
+  return LCU_OK;
+}
+
+template <typename T>
+int launch_window_attention(const attn_rows<T>& p, int m, int pos0, int* err, cudaStream_t stream) {
+  (void)err;
+  const int keys = most_keys(p, pos0 + m - 1);
+  const size_t smem = attention_smem(p, keys, false);
+  LCU_REQUIRE(smem <= 220 * 1024, "window attention: %d visible keys", keys);
+  static bool attr_done[16] = {};
+  int dev = 0;
+  LCU_CUDA(cudaGetDevice(&dev));
+  if (dev < 16 && !attr_done[dev]) {
+    LCU_CUDA(cudaFuncSetAttribute(window_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    attr_done[dev] = true;
+  }
+  LCU_CUDA(launch_after(window_rows_kernel<T>, dim3(p.heads, m), dim3(MX_THREADS), smem, stream, p, pos0, keys));
+  return LCU_OK;
+}
+
+template <typename T>
+int launch_scan(const scan_rows<T>& p, bool wkv, int m, int pos0, cudaStream_t stream) {
+#define LCU_SCAN(KC) return wkv ? launch_scan_one<T, KC, true>(p, m, pos0, stream) : launch_scan_one<T, KC, false>(p, m, pos0, stream)
+  if (p.dim <= 32) LCU_SCAN(4);
+  if (p.dim <= 64) LCU_SCAN(8);
+  LCU_SCAN(16);
+#undef LCU_SCAN
+}
+
+template <typename T>
+int launch_mixer_step(const mixer_step<T>& p, int ctx_len, cudaStream_t stream) {
+  size_t smem = 0;
+  for (int i = 0; i < p.n_branches; ++i) {
+    const step_branch<T>& b = p.b[i];
+    if (b.kind == BRANCH_WINDOW_ATTN) smem = std::max(smem, attention_smem(b.attn, most_keys(b.attn, ctx_len - 1) / ST_CLUSTER + 2, true));
+    else smem = std::max(smem, (3 * (size_t)b.scan.dim + MX_THREADS + b.rank + 8) * sizeof(float));
+  }
+  LCU_REQUIRE(smem <= 220 * 1024, "mixer step: %zu bytes of shared memory", smem);
+  static bool attr_done[16] = {};
+  int dev = 0;
+  LCU_CUDA(cudaGetDevice(&dev));
+  if (dev < 16 && !attr_done[dev]) {
+    LCU_CUDA(cudaFuncSetAttribute(mixer_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    attr_done[dev] = true;
+  }
+  return launch_clustered(mixer_step_kernel<T>, p.n_clusters * ST_CLUSTER, ST_CLUSTER, MX_THREADS, smem, stream, p);
+}
+
+#define LCU_BLOCK_MIXERS(T)                                                                    \
+  template int launch_window_append<T>(const attn_rows<T>&, int, int, cudaStream_t);           \
+  template int launch_window_attention<T>(const attn_rows<T>&, int, int, int*, cudaStream_t);  \
+  template int launch_scan<T>(const scan_rows<T>&, bool, int, int, cudaStream_t);              \
+  template int launch_mixer_step<T>(const mixer_step<T>&, int, cudaStream_t);
+LCU_BLOCK_MIXERS(__nv_bfloat16)
+LCU_BLOCK_MIXERS(float)
+
+}  // namespace lcu

@@ -1,0 +1,416 @@
+// Row-wise kernels of the block models: embedding, hyper-connected residual, token shift, decays, head gates, weight
+// placement, and the binary32 products.
+#include <algorithm>
+
+#include "block_ops.cuh"
+#include "elem.cuh"
+
+namespace lcu {
+namespace {
+
+// ------------------------------------------------------------------ embedding
+template <typename T>
+__global__ void __launch_bounds__(256) block_embed_kernel(const embed_params<T> p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.x;
+  __shared__ long long s_row;
+  const int tok = p.ids[r];
+  if (threadIdx.x == 0) {
+    const int pos = (p.pos ? *p.pos : p.pos_value) + r;
+    long long row = p.buckets;
+    const int prev = r > 0 ? (int)p.ids[r - 1] : *p.prev_token;
+    if (pos > 0 && p.buckets > 0) row = ((long long)prev * p.mul_prev + (long long)tok * p.mul_cur) % p.buckets;
+    s_row = row;
+    if (r == 0) *p.prev_token = p.ids[p.m - 1];  // (only row 0 reads it, just above)
+  }
+  __syncthreads();
+  const T* e = p.table + (size_t)tok * p.width;
+  const T* b = p.buckets > 0 ? p.bigram + (size_t)s_row * p.width : nullptr;
+  float* x = p.xs + (size_t)r * p.streams * p.width;
+  for (int c = threadIdx.x; c < p.width; c += 256) {
+    float v = to_f(e[c]) * p.scale;
+    if (b) v += to_f(b[c]);
+    for (int s = 0; s < p.streams; ++s) x[(size_t)s * p.width + c] = v;
+  }
+}
+
+// ------------------------------------------------------------------ hyper-connected residual + norm
+constexpr int HY_THREADS = 256;
+constexpr int HY_CLUSTER = 8;  // CTAs that share one row when there is only one
+
+// SM: room for the streams (p.streams <= SM); CL: CTAs per row
+template <typename T, int SM, int CL>
+__global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_params<T> p, const int per) {
+  extern __shared__ float u_row[];  // this CTA's columns of u
+  __shared__ float s_red[HY_THREADS / 32], s_part;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int i_row = blockIdx.x / CL, rank = blockIdx.x % CL;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = p.rows ? p.rows[i_row] : i_row;
+  const int S = p.streams, W = p.width;
+  const int c0 = min(W, rank * per), c1 = min(W, c0 + per);
+  float in[SM], up[SM], mix[SM][SM];
+#pragma unroll
+  for (int s = 0; s < SM; ++s) {
+    in[s] = s < S ? p.in[s] : 0.f;
+    up[s] = p.y && s < S ? p.up_out[s] : 0.f;
+#pragma unroll
+    for (int t = 0; t < SM; ++t) mix[s][t] = p.y && s < S && t < S ? p.up_mix[s * S + t] : 0.f;
+  }
+  float* x = p.xs + (size_t)row * S * W;
+  const float* y = p.y ? p.y + (size_t)row * p.ldy : nullptr;
+  float ss = 0.f;
+  auto column = [&](float (&v)[SM], float yv) {  // new streams in v, returns u
+    if (y) {
+      float n[SM];
+#pragma unroll
+      for (int t = 0; t < SM; ++t) {
+        float a = up[t] * yv;
+#pragma unroll
+        for (int s = 0; s < SM; ++s) a = fmaf(mix[s][t], v[s], a);
+        n[t] = a;
+      }
+#pragma unroll
+      for (int t = 0; t < SM; ++t) v[t] = n[t];
+    }
+    float u = 0.f;
+#pragma unroll
+    for (int s = 0; s < SM; ++s) u = fmaf(in[s], v[s], u);
+    return u;
+  };
+  if ((W & 3) == 0) {  // (per is a multiple of 4: rows and slices start 16-byte aligned)
+    for (int c = c0 + 4 * tid; c < c1; c += 4 * HY_THREADS) {
+      float4 xv[SM];
+#pragma unroll
+      for (int s = 0; s < SM; ++s) xv[s] = s < S ? *reinterpret_cast<const float4*>(x + (size_t)s * W + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      const float4 yv = y ? *reinterpret_cast<const float4*>(y + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      float4 u;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        float v[SM];
+#pragma unroll
+        for (int s = 0; s < SM; ++s) v[s] = reinterpret_cast<const float*>(&xv[s])[e];
+        const float ue = column(v, reinterpret_cast<const float*>(&yv)[e]);
+        reinterpret_cast<float*>(&u)[e] = ue;
+        ss = fmaf(ue, ue, ss);
+#pragma unroll
+        for (int s = 0; s < SM; ++s) reinterpret_cast<float*>(&xv[s])[e] = v[s];
+      }
+      *reinterpret_cast<float4*>(u_row + c - c0) = u;
+      if (y && p.store) {
+#pragma unroll
+        for (int s = 0; s < SM; ++s)
+          if (s < S) *reinterpret_cast<float4*>(x + (size_t)s * W + c) = xv[s];
+      }
+    }
+  } else {
+    for (int c = c0 + tid; c < c1; c += HY_THREADS) {
+      float v[SM];
+#pragma unroll
+      for (int s = 0; s < SM; ++s) v[s] = s < S ? x[(size_t)s * W + c] : 0.f;
+      const float u = column(v, y ? y[c] : 0.f);
+      u_row[c - c0] = u;
+      ss = fmaf(u, u, ss);
+      if (y && p.store) {
+#pragma unroll
+        for (int s = 0; s < SM; ++s)
+          if (s < S) x[(size_t)s * W + c] = v[s];
+      }
+    }
+  }
+  ss = warp_sum(ss);
+  if (lane == 0) s_red[warp] = ss;
+  __syncthreads();
+  float total = 0.f;
+#pragma unroll
+  for (int w = 0; w < HY_THREADS / 32; ++w) total += s_red[w];
+  if (CL > 1) {
+    if (tid == 0) s_part = total;
+    cluster_sync();
+    total = 0.f;
+#pragma unroll
+    for (int r = 0; r < CL; ++r) total += ld_dsmem_f32(mapa(smem_u32(&s_part), r));
+  }
+  const float inv = 1.0f / sqrtf(total / (float)W + p.eps);
+  T* h = p.h + (size_t)i_row * p.ldh;
+  const bool start = p.mix && *p.pos == 0;
+  for (int c = c0 + tid; c < c1; c += HY_THREADS) {
+    const float u = u_row[c - c0];
+    if (p.u_out) p.u_out[(size_t)i_row * W + c] = u;
+    const T hv = from_f<T>(u * inv * (1.0f + p.norm_w[c]));
+    h[c] = hv;
+    if (p.mix) {
+      const float hf = to_f(hv), d = (start ? 0.f : to_f(p.prev[c])) - hf;
+      for (int i = 0; i < p.n_mix; ++i) p.mix[i * p.mix_stride + c] = from_f<T>(fmaf(d, p.mu[(size_t)i * W + c], hf));
+      p.prev[c] = hv;
+    }
+  }
+  if (CL > 1) cluster_sync();  // nobody leaves while its partial sum may still be read
+}
+
+template <typename T, int SM, int CL>
+int launch_hyper_one(const hyper_params<T>& p, int n_rows, cudaStream_t stream) {
+  const int per = (int)round_up(ceil_div(p.width, CL), 4);
+  const size_t smem = (size_t)per * sizeof(float);
+  LCU_REQUIRE(smem <= 200 * 1024, "hyper_rows: a row of %d does not fit in shared memory", p.width);
+  static bool attr_done[16] = {};
+  int dev = 0;
+  LCU_CUDA(cudaGetDevice(&dev));
+  if (dev < 16 && !attr_done[dev]) {
+    LCU_CUDA(cudaFuncSetAttribute((hyper_rows_kernel<T, SM, CL>), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    attr_done[dev] = true;
+  }
+  return launch_clustered(hyper_rows_kernel<T, SM, CL>, n_rows * CL, CL, HY_THREADS, smem, stream, p, per);
+}
+
+// ------------------------------------------------------------------ token shift
+template <typename T>
+__global__ void __launch_bounds__(256) token_shift_kernel(const T* h, int ldh, T* prev, const float* mu, T* mix, size_t mix_stride, int n_mix, int m,
+                                                          int width, int pos0) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.x;
+  for (int c = threadIdx.x; c < width; c += 256) {
+    const float hf = to_f(h[(size_t)r * ldh + c]);
+    float hp;
+    if (r > 0) {
+      hp = to_f(h[(size_t)(r - 1) * ldh + c]);
+    } else {
+      hp = pos0 == 0 ? 0.f : to_f(prev[c]);
+      prev[c] = h[(size_t)(m - 1) * ldh + c];  // (only row 0 touches prev)
+    }
+    const float d = hp - hf;
+    for (int i = 0; i < n_mix; ++i) mix[i * mix_stride + (size_t)r * ldh + c] = from_f<T>(fmaf(d, mu[(size_t)i * width + c], hf));
+  }
+}
+
+__global__ void rotation_table_kernel(float2* table, int n_pos, int half, double base) {
+  const int idx = blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= n_pos * half) return;
+  const int pos = idx / half, i = idx - pos * half;
+  const double a = (double)pos * pow(base, -(double)i / half);
+  table[idx] = make_float2((float)cos(a), (float)sin(a));
+}
+
+// ------------------------------------------------------------------ wkv decays
+constexpr int WD_ROWS = 8;
+__global__ void __launch_bounds__(256) wkv_decay_kernel(float* w, const float* low, int ld_low, const float* w2t, const float* w0, int rank,
+                                                        int channels, int m) {
+  extern __shared__ float th[];  // [WD_ROWS][rank]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r0 = blockIdx.y * WD_ROWS, nr = min(WD_ROWS, m - r0);
+  for (int i = threadIdx.x; i < WD_ROWS * rank; i += 256) {
+    const int r = i / rank, j = i - r * rank;
+    th[i] = r < nr ? tanhf(low[(size_t)(r0 + r) * ld_low + j]) : 0.f;
+  }
+  __syncthreads();
+  const int ch = blockIdx.x * 256 + threadIdx.x;
+  if (ch >= channels) return;
+  float acc[WD_ROWS];
+#pragma unroll
+  for (int r = 0; r < WD_ROWS; ++r) acc[r] = w0[ch];
+  for (int j = 0; j < rank; ++j) {
+    const float a = w2t[(size_t)j * channels + ch];
+#pragma unroll
+    for (int r = 0; r < WD_ROWS; ++r) acc[r] = fmaf(a, th[r * rank + j], acc[r]);
+  }
+  for (int r = 0; r < nr; ++r) w[(size_t)(r0 + r) * channels + ch] = expf(-expf(acc[r]));
+}
+
+// ------------------------------------------------------------------ normalised, gated heads (one warp per row and head)
+template <typename T>
+__global__ void __launch_bounds__(256) head_gate_kernel(T* out, int ldo, const float* o, int ld_raw, const T* g, int ldg, const float* norm, int heads,
+                                                        int vdim, float eps, float out_scale, int m) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int idx = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (idx >= m * heads) return;
+  const int r = idx / heads, hd = idx - r * heads;
+  const float* x = o + (size_t)r * ld_raw + hd * vdim;
+  float ss = 0.f;
+  for (int j = lane; j < vdim; j += 32) ss = fmaf(x[j], x[j], ss);
+  ss = warp_sum(ss);
+  const float inv = 1.0f / sqrtf(ss / (float)vdim + eps);
+  for (int j = lane; j < vdim; j += 32) {
+    const int c = hd * vdim + j;
+    float v = x[j] * inv;
+    if (norm) v *= norm[c];
+    out[(size_t)r * ldo + c] = from_f<T>(v * silu_f(to_f(g[(size_t)r * ldg + c])) * out_scale);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) gate_rows_kernel(T* out, const T* ab, int m, int f) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int V = 16 / sizeof(T);
+  const size_t i = (size_t)blockIdx.x * 256 + threadIdx.x;
+  const int fv = f / V;
+  if (i >= (size_t)m * fv) return;
+  const size_t r = i / fv, jv = i - r * fv;
+  const uint4 av = reinterpret_cast<const uint4*>(ab + r * 2 * f)[jv], bv = reinterpret_cast<const uint4*>(ab + r * 2 * f + f)[jv];
+  __align__(16) T o[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) o[e] = from_f<T>(silu_f(to_f(reinterpret_cast<const T*>(&av)[e])) * to_f(reinterpret_cast<const T*>(&bv)[e]));
+  reinterpret_cast<uint4*>(out + r * f)[jv] = *reinterpret_cast<const uint4*>(o);
+}
+
+template <typename T>
+__global__ void place_kernel(T* dst, int ld, const void* src, int f32, int rows, int cols, int transpose) {
+  const size_t n = (size_t)rows * cols;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = i / cols, c = i - r * cols;
+    const float v = f32 ? reinterpret_cast<const float*>(src)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(src)[i]);
+    dst[transpose ? c * ld + r : r * ld + c] = from_f<T>(v);
+  }
+}
+
+// ------------------------------------------------------------------ binary32 products
+// few rows: one warp per output column, all rows of x at once
+constexpr int MF_ROWS = 8;
+__global__ void __launch_bounds__(256) matmul_f32_few_kernel(float* out, const float* x, int ldx, const float* w, int m, int N, int K) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int n = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, r0 = blockIdx.y * MF_ROWS;
+  if (n >= N) return;
+  const int nr = min(MF_ROWS, m - r0);
+  float acc[MF_ROWS] = {};
+  for (int k = lane * 4; k < K; k += 128) {
+    const float4 a = *reinterpret_cast<const float4*>(w + (size_t)n * K + k);
+#pragma unroll
+    for (int r = 0; r < MF_ROWS; ++r)
+      if (r < nr) {
+        const float4 b = *reinterpret_cast<const float4*>(x + (size_t)(r0 + r) * ldx + k);
+        acc[r] = fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, acc[r]))));
+      }
+  }
+#pragma unroll
+  for (int r = 0; r < MF_ROWS; ++r) {
+    const float v = warp_sum(acc[r]);
+    if (lane == 0 && r < nr) out[(size_t)(r0 + r) * N + n] = v;
+  }
+}
+// 64 x 64 tiles, 4 x 4 results per thread
+__global__ void __launch_bounds__(256) matmul_f32_tile_kernel(float* out, const float* x, int ldx, const float* w, int m, int N, int K) {
+  __shared__ float xs[16][68], ws[16][68];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  float acc[4][4] = {};
+  const int lr = tid >> 2, lk = (tid & 3) * 4;  // loader: row of the tile, four k
+  for (int k0 = 0; k0 < K; k0 += 16) {
+    const float4 a = m0 + lr < m ? *reinterpret_cast<const float4*>(x + (size_t)(m0 + lr) * ldx + k0 + lk) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 b = n0 + lr < N ? *reinterpret_cast<const float4*>(w + (size_t)(n0 + lr) * K + k0 + lk) : make_float4(0.f, 0.f, 0.f, 0.f);
+    __syncthreads();
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      xs[lk + e][lr] = reinterpret_cast<const float*>(&a)[e];
+      ws[lk + e][lr] = reinterpret_cast<const float*>(&b)[e];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      const float4 av = *reinterpret_cast<const float4*>(&xs[k][ty * 4]), bv = *reinterpret_cast<const float4*>(&ws[k][tx * 4]);
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(reinterpret_cast<const float*>(&av)[i], reinterpret_cast<const float*>(&bv)[j], acc[i][j]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    if (m0 + ty * 4 + i < m)
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (n0 + tx * 4 + j < N) out[(size_t)(m0 + ty * 4 + i) * N + n0 + tx * 4 + j] = acc[i][j];
+}
+
+}  // namespace
+
+template <typename T>
+int launch_block_embed(const embed_params<T>& p, cudaStream_t stream) {
+  LCU_CUDA(launch_after(block_embed_kernel<T>, dim3(p.m), dim3(256), 0, stream, p));
+  return LCU_OK;
+}
+
+template <typename T>
+int launch_hyper_rows(const hyper_params<T>& p, int n_rows, cudaStream_t stream) {
+  if (n_rows < 1) return LCU_OK;
+  LCU_REQUIRE(p.streams >= 1 && p.streams <= 8, "hyper_rows: %d streams", p.streams);
+  LCU_REQUIRE(p.mix == nullptr || n_rows == 1, "hyper_rows: the token shift is fused for a single row only");
+#define LCU_HYPER(SM) \
+  return n_rows == 1 ? launch_hyper_one<T, SM, HY_CLUSTER>(p, n_rows, stream) : launch_hyper_one<T, SM, 1>(p, n_rows, stream)
+  if (p.streams == 1) LCU_HYPER(1);
+  if (p.streams == 2) LCU_HYPER(2);
+  if (p.streams <= 4) LCU_HYPER(4);
+  LCU_HYPER(8);
+#undef LCU_HYPER
+}
+
+template <typename T>
+int launch_token_shift(const T* h, int ldh, T* prev, const float* mu, T* mix, size_t mix_stride, int n_mix, int m, int width, int pos0,
+                       cudaStream_t stream) {
+  LCU_CUDA(launch_after(token_shift_kernel<T>, dim3(m), dim3(256), 0, stream, h, ldh, prev, mu, mix, mix_stride, n_mix, m, width, pos0));
+  return LCU_OK;
+}
+
+int launch_rotation_table(float2* table, int n_pos, int dims, double base, cudaStream_t stream) {
+  const int half = dims / 2;
+  rotation_table_kernel<<<(unsigned)ceil_div((size_t)n_pos * half, 256), 256, 0, stream>>>(table, n_pos, half, base);
+  LCU_CUDA(cudaGetLastError());
+  return LCU_OK;
+}
+
+int launch_wkv_decay(float* w, const float* low, int ld_low, const float* w2t, const float* w0, int rank, int channels, int m, cudaStream_t stream) {
+  LCU_REQUIRE((size_t)WD_ROWS * rank * 4 <= 48 * 1024, "wkv_decay: rank %d", rank);
+  LCU_CUDA(launch_after(wkv_decay_kernel, dim3((channels + 255) / 256, (m + WD_ROWS - 1) / WD_ROWS), dim3(256), (size_t)WD_ROWS * rank * 4, stream, w, low,
+                        ld_low, w2t, w0, rank, channels, m));
+  return LCU_OK;
+}
+
+template <typename T>
+int launch_head_gate(T* out, int ldo, const float* o, int ld_raw, const T* g, int ldg, const float* norm, int heads, int vdim, float eps,
+                     float out_scale, int m, cudaStream_t stream) {
+  LCU_CUDA(launch_after(head_gate_kernel<T>, dim3((unsigned)ceil_div((size_t)m * heads, 8)), dim3(256), 0, stream, out, ldo, o, ld_raw, g, ldg, norm, heads,
+                        vdim, eps, out_scale, m));
+  return LCU_OK;
+}
+
+template <typename T>
+int launch_gate_rows(T* out, const T* ab, int m, int f, cudaStream_t stream) {
+  LCU_REQUIRE(f % 8 == 0, "gate_rows: rows of %d elements are not 16-byte vectors", f);
+  LCU_CUDA(launch_after(gate_rows_kernel<T>, dim3((unsigned)ceil_div((size_t)m * f * sizeof(T) / 16, 256)), dim3(256), 0, stream, out, ab, m, f));
+  return LCU_OK;
+}
+
+template <typename T>
+int launch_place(T* dst, int ld, const void* src, place_source type, int rows, int cols, bool transpose, cudaStream_t stream) {
+  const size_t n = (size_t)rows * cols;
+  if (n == 0) return LCU_OK;
+  place_kernel<T><<<(unsigned)std::min<size_t>(ceil_div(n, 256), 148 * 16), 256, 0, stream>>>(dst, ld, src, type == PLACE_F32, rows, cols, transpose);
+  LCU_CUDA(cudaGetLastError());
+  return LCU_OK;
+}
+
+int launch_matmul_f32(float* out, const float* x, int ldx, const float* w, int m, int N, int K, cudaStream_t stream) {
+  LCU_REQUIRE(m >= 1 && K % 16 == 0 && ldx % 4 == 0, "matmul_f32: unsupported shape m=%d K=%d", m, K);
+  if (m <= MF_ROWS) LCU_CUDA(launch_after(matmul_f32_few_kernel, dim3((N + 7) / 8, 1), dim3(256), 0, stream, out, x, ldx, w, m, N, K));
+  else LCU_CUDA(launch_after(matmul_f32_tile_kernel, dim3((N + 63) / 64, (m + 63) / 64), dim3(256), 0, stream, out, x, ldx, w, m, N, K));
+  return LCU_OK;
+}
+
+#define LCU_BLOCK_OPS(T)                                                                                                             \
+  template int launch_block_embed<T>(const embed_params<T>&, cudaStream_t);                                                          \
+  template int launch_hyper_rows<T>(const hyper_params<T>&, int, cudaStream_t);                                                      \
+  template int launch_token_shift<T>(const T*, int, T*, const float*, T*, size_t, int, int, int, int, cudaStream_t);                 \
+  template int launch_head_gate<T>(T*, int, const float*, int, const T*, int, const float*, int, int, float, float, int, cudaStream_t); \
+  template int launch_gate_rows<T>(T*, const T*, int, int, cudaStream_t);                                                            \
+  template int launch_place<T>(T*, int, const void*, place_source, int, int, bool, cudaStream_t);
+LCU_BLOCK_OPS(__nv_bfloat16)
+LCU_BLOCK_OPS(float)
+
+}  // namespace lcu

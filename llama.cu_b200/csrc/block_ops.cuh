@@ -1,0 +1,159 @@
+// Kernels of the block models beside the matrix products: embedding with bigrams, hyper-connected residual rows with the
+// following norm, window-and-blocks attention, linear recurrences (retention, wkv), token shift, head normalisation and
+// gates.  T is the activation / cache / weight type of the model: __nv_bfloat16 or float.  Norms, residual streams,
+// positions, scores, softmax, decays, recurrent state and everything that enters a recurrence beside the projections are
+// binary32 in both.
+#pragma once
+#include <cuda_bf16.h>
+
+#include "block_spec.cuh"
+#include "common.cuh"
+
+namespace lcu {
+
+// rows of the residual: xs[row][stream][width] = (table[token] * scale + bigram row), the same in every stream.  The first
+// token of a sequence (position 0) takes bigram row `buckets`.  *prev_token is the token before the first row and becomes
+// the last row's token.
+template <typename T>
+struct embed_params {
+  float* xs;
+  const T *table, *bigram;
+  const short* ids;
+  int* prev_token;
+  const int* pos;  // device position of row 0, or null: pos_value
+  int pos_value;
+  int m, width, streams, buckets;
+  long long mul_prev, mul_cur;
+  float scale;
+};
+template <typename T>
+int launch_block_embed(const embed_params<T>& p, cudaStream_t stream);
+
+// One pass over residual rows between two sublayers:
+//   x_t <- sum_s up_mix[s][t] x_s + up_out[t] y      (the sublayer just computed; skipped when y is null)
+//   u = sum_s in[s] x_s;  h = u / sqrt(mean(u^2) + eps) * (1 + norm_w)    (the norm of the next one)
+// and, for a single row of a token-shifted mixer, its inputs mix_i = h + (h_prev - h) * mu_i with h_prev replaced by h.
+template <typename T>
+struct hyper_params {
+  float* xs;             // [rows][streams][width]
+  int width, streams;
+  const float* y;        // [rows][ldy]
+  int ldy;
+  const float *up_mix, *up_out;
+  int store;             // write the new streams back
+  const float* in;
+  const float* norm_w;
+  float eps;
+  const int* rows;       // row numbers to work on, or null: 0 .. n-1; results are dense
+  T* h;                  // [n][ldh]
+  int ldh;
+  float* u_out;          // optional: u of every row [n][width]
+  // token shift of a single row
+  T* prev;               // [width]
+  const float* mu;       // [n_mix][width]
+  T* mix;                // n_mix rows, mix_stride apart
+  size_t mix_stride;
+  int n_mix;
+  const int* pos;
+};
+template <typename T>
+int launch_hyper_rows(const hyper_params<T>& p, int n_rows, cudaStream_t stream);
+
+// mix_i[row] = h[row] + (h[row-1] - h[row]) * mu_i; row -1 is `prev` (zeros at position 0), which becomes the last row
+template <typename T>
+int launch_token_shift(const T* h, int ldh, T* prev, const float* mu, T* mix, size_t mix_stride, int n_mix, int m, int width, int pos0,
+                       cudaStream_t stream);
+
+// cos / sin of position * base^(-2 i / dims), angles in binary64: table[pos][dims / 2]
+int launch_rotation_table(float2* table, int n_pos, int dims, double base, cudaStream_t stream);
+
+// ---- attention over a sliding window and one mean key / value per block of `pool` tokens that lies wholly before it.
+// Caches are [kv_head][position][ld] and [kv_head][block][ld], ld = dim rounded up to 8.
+template <typename T>
+struct window_cache {
+  T *k, *v, *kp, *vp;
+  int ctx_len, n_blocks, ldk, ldv;
+};
+template <typename T>
+struct attn_rows {
+  const T *q, *k, *v;  // new rows; row stride ld
+  int ld;
+  window_cache<T> cache;
+  int heads, kv_heads, dim, vdim, window, pool;
+  float scale, out_scale;
+  T* out;
+  int ldo;
+};
+// cache rows pos0 .. pos0+m-1, then the blocks they complete, then attention of the rows
+template <typename T>
+int launch_window_append(const attn_rows<T>& p, int m, int pos0, cudaStream_t stream);
+template <typename T>
+int launch_window_attention(const attn_rows<T>& p, int m, int pos0, int* err, cudaStream_t stream);
+
+// ---- linear recurrences over rows, per head:
+//   retention: S <- decay S + k v^T, o = S^T q          (k and q rotated, k times kscale)
+//   wkv:       o = (S + diag(u) k v^T)^T q, S <- diag(w) S + k v^T
+template <typename T>
+struct scan_rows {
+  const T *q, *k, *v;     // row stride ld (of the recurrences' projections)
+  int ldq, ldk, ldv;
+  int heads, dim, vdim;
+  float* state;           // [heads][dim][vdim]
+  const float2* rope;     // retention: rotation table, or null
+  int rot_dims;
+  float kscale;
+  const float* decay;     // retention: per head
+  const float* w;         // wkv: [rows][heads * dim]
+  const float* u;         // wkv: [heads][dim]
+  float* out;             // [rows][ldo] binary32
+  int ldo;
+};
+template <typename T>
+int launch_scan(const scan_rows<T>& p, bool wkv, int m, int pos0, cudaStream_t stream);
+
+// w[row][ch] = exp(-exp(w0[ch] + sum_r w2t[r][ch] tanh(low[row][r])))
+int launch_wkv_decay(float* w, const float* low, int ld_low, const float* w2t, const float* w0, int rank, int channels, int m, cudaStream_t stream);
+
+// out[row][head * vdim + j] = o / rms(o of the head) * norm * silu(g) * out_scale
+template <typename T>
+int launch_head_gate(T* out, int ldo, const float* o, int ld_raw, const T* g, int ldg, const float* norm, int heads, int vdim, float eps,
+                     float out_scale, int m, cudaStream_t stream);
+
+// ---- one token through all branches of a mixer in one launch: a cluster of CTAs per head
+template <typename T>
+struct step_branch {
+  int kind;               // branch_kind
+  int first;              // first cluster of the launch
+  attn_rows<T> attn;      // attention (row pointers: the token's row)
+  scan_rows<T> scan;      // recurrences; w unused
+  const T* g;             // gate projection of the token
+  const float* low;       // wkv: input of the decay's second product
+  const float *w2t, *w0;
+  int rank;
+  const float* norm;      // wkv: weight of the normalised heads, or null
+  float eps, out_scale;
+  T* out;                 // the branch's columns
+};
+constexpr int STEP_MAX_BRANCHES = 2;
+template <typename T>
+struct mixer_step {
+  step_branch<T> b[STEP_MAX_BRANCHES];
+  int n_branches, n_clusters;
+  const int* pos;
+};
+template <typename T>
+int launch_mixer_step(const mixer_step<T>& p, int ctx_len, cudaStream_t stream);
+
+// out[row][j] = silu(ab[row][j]) * ab[row][f + j]
+template <typename T>
+int launch_gate_rows(T* out, const T* ab, int m, int f, cudaStream_t stream);
+
+// ---- weights: bfloat16 (or binary32) source rows into a matrix of the model
+enum place_source { PLACE_BF16 = 0, PLACE_F32 = 1 };
+template <typename T>
+int launch_place(T* dst, int ld, const void* src, place_source type, int rows, int cols, bool transpose, cudaStream_t stream);
+
+// ---- binary32 products: out[m][N] = x[m][ldx] . w[N][K]^T
+int launch_matmul_f32(float* out, const float* x, int ldx, const float* w, int m, int N, int K, cudaStream_t stream);
+
+}  // namespace lcu

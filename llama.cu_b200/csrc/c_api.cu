@@ -9,6 +9,7 @@
 #include <vector>
 
 #include "attention.cuh"
+#include "block_model.cuh"
 #include "gemm_tc.cuh"
 #include "gemv.cuh"
 #include "ops.cuh"
@@ -42,6 +43,13 @@ partition make_partition(const model_params& p, const int* layer_gpus) {
   cudaGetDevice(&cur);  // no partition given: everything on the calling thread's current device
   for (uint32_t i = 0; i < p.n_layers; ++i) part.layer_gpus.push_back(layer_gpus ? layer_gpus[i] : cur);
   return part;
+}
+
+// the LLaMA model behind a handle, for the entry points that exist for that family only
+int llama_model(void* mdl, model** out) {
+  *out = dynamic_cast<model*>((model_base*)mdl);
+  LCU_REQUIRE(*out != nullptr, "this call is for models of the LLaMA family; the model is a %s", mdl ? ((model_base*)mdl)->family() : "null pointer");
+  return LCU_OK;
 }
 
 int* scratch_err() { return device_scratch_words(); }
@@ -332,11 +340,79 @@ int lcu_model_create(const void* params40, const int* layer_gpus, void** model_o
   std::unique_ptr<model> m;
   int rc = model::create(m, p, make_partition(p, layer_gpus));
   if (rc) return rc;
-  *model_out = m.release();
+  *model_out = static_cast<model_base*>(m.release());
   return LCU_OK;
 }
+static int load_block_model(const char* dir, const int* layer_gpus, int dtype, void** model_out) {
+  LCU_REQUIRE(dtype == BLOCK_BF16 || dtype == BLOCK_F32, "model_load: number format %d is not 0 (bfloat16) or 1 (binary32)", dtype);
+  int dev = 0;
+  LCU_CUDA(cudaGetDevice(&dev));
+  device_guard g(layer_gpus ? layer_gpus[0] : dev);  // (a block model lives on one GPU)
+  std::unique_ptr<block_model> m;
+  int rc = block_model::load(m, dir, (block_dtype)dtype);
+  if (rc) return rc;
+  *model_out = static_cast<model_base*>(m.release());
+  return LCU_OK;
+}
+static bool has_config(const char* dir) {
+  FILE* f = fopen((std::string(dir) + "/config.json").c_str(), "rb");
+  if (f) fclose(f);
+  return f != nullptr;
+}
+int lcu_model_load_as(const char* dir, const int* layer_gpus, int dtype, void** model_out) {
+  NEED_DEVICE();
+  LCU_REQUIRE(dir && model_out, "model_load: bad arguments");
+  if (has_config(dir)) return load_block_model(dir, layer_gpus, dtype, model_out);
+  LCU_REQUIRE(dtype == 0, "model_load: weight directories of the LLaMA family hold halves or u8; there is no binary32 path for them");
+  return lcu_model_load(dir, layer_gpus, model_out);
+}
+int lcu_model_create_from_config(const char* config_text, int dtype, int decay_rank, void** model_out) {
+  NEED_DEVICE();
+  LCU_REQUIRE(config_text && model_out && (dtype == BLOCK_BF16 || dtype == BLOCK_F32) && decay_rank >= 1, "model_create_from_config: bad arguments");
+  block_spec spec;
+  int rc = read_block_config(config_text, spec);
+  if (rc) return rc;
+  std::unique_ptr<block_model> m;
+  rc = block_model::create(m, spec, (block_dtype)dtype, std::vector<int>(spec.layers.size(), decay_rank));
+  if (rc) return rc;
+  *model_out = static_cast<model_base*>(m.release());
+  return LCU_OK;
+}
+int lcu_config_summary(const char* config_text, int32_t* out8) {
+  LCU_REQUIRE(config_text && out8, "config_summary: bad arguments");
+  block_spec s;
+  int rc = read_block_config(config_text, s);
+  if (rc) return rc;
+  const int v[8] = {s.vocab, s.width, (int)s.layers.size(), (int)s.runs.size(), s.streams, s.buckets, 0, 0};
+  memcpy(out8, v, sizeof v);
+  return LCU_OK;
+}
+int lcu_config_runs(const char* config_text, int32_t* runs_out, int capacity) {
+  block_spec s;
+  LCU_REQUIRE(config_text && runs_out, "config_runs: bad arguments");
+  int rc = read_block_config(config_text, s);
+  if (rc) return -rc;
+  for (size_t i = 0; i < s.runs.size() && (int)i < capacity; ++i) runs_out[i] = s.runs[i];
+  return (int)s.runs.size();
+}
+int lcu_architectures(char* out, int capacity) {
+  const std::string s = architecture_names();
+  LCU_REQUIRE(out && capacity > (int)s.size(), "architectures: buffer of %d bytes is too small", capacity);
+  memcpy(out, s.c_str(), s.size() + 1);
+  return LCU_OK;
+}
+int lcu_model_shape(void* mdl, int32_t* vocab, int32_t* width, int32_t* layers) {
+  model_base* m = (model_base*)mdl;
+  LCU_REQUIRE(m, "model_shape: null model");
+  if (vocab) *vocab = m->vocab();
+  if (width) *width = m->width();
+  if (layers) *layers = m->n_layers();
+  return LCU_OK;
+}
+const char* lcu_model_family(void* mdl) { return mdl ? ((model_base*)mdl)->family() : ""; }
 int lcu_model_load(const char* dir, const int* layer_gpus, void** model_out) {
   NEED_DEVICE();
+  if (has_config(dir)) return load_block_model(dir, layer_gpus, BLOCK_BF16, model_out);
   model_params p;
   FILE* f = fopen((std::string(dir) + "/params").c_str(), "rb");
   if (!f || fread(&p, 1, sizeof(p), f) != sizeof(p) || fgetc(f) != EOF) {
@@ -350,29 +426,39 @@ int lcu_model_load(const char* dir, const int* layer_gpus, void** model_out) {
   if (rc) return rc;
   rc = m->load_dir(dir);
   if (rc) return rc;
-  *model_out = m.release();
+  *model_out = static_cast<model_base*>(m.release());
   return LCU_OK;
 }
-int lcu_model_fill_synthetic(void* mdl, uint64_t seed, float scale) { return ((model*)mdl)->fill_synthetic(seed, scale); }
-int lcu_model_save(void* mdl, const char* dir) { return ((model*)mdl)->save_dir(dir); }
+int lcu_model_fill_synthetic(void* mdl, uint64_t seed, float scale) { return ((model_base*)mdl)->fill_synthetic(seed, scale); }
+int lcu_model_save(void* mdl, const char* dir) {
+  model* m = nullptr;
+  int rc = llama_model(mdl, &m);
+  return rc ? rc : m->save_dir(dir);
+}
 int lcu_model_tensor(void* mdl, const char* name, int which, void** dev_out, uint64_t* bytes_out, int* device_out) {
   size_t bytes = 0;
-  int rc = ((model*)mdl)->find_tensor(name, which, dev_out, &bytes, device_out);
+  model* m = nullptr;
+  int rc = llama_model(mdl, &m);
+  if (rc) return rc;
+  rc = m->find_tensor(name, which, dev_out, &bytes, device_out);
   if (bytes_out) *bytes_out = bytes;
   return rc;
 }
 int lcu_model_params(void* mdl, void* params40_out) {
-  memcpy(params40_out, &((model*)mdl)->params, sizeof(model_params));
+  model* m = nullptr;
+  int rc = llama_model(mdl, &m);
+  if (rc) return rc;
+  memcpy(params40_out, &m->params, sizeof(model_params));
   return LCU_OK;
 }
 uint64_t lcu_model_shadow_bytes(void* mdl) {
-  model* m = (model*)mdl;
+  model* m = dynamic_cast<model*>((model_base*)mdl);
   if (!m) return 0;
   std::lock_guard<std::mutex> lock(m->shadow_mu);
   return m->shadow_state > 0 ? m->shadow_bytes : 0;
 }
-uint64_t lcu_model_weight_bytes(void* mdl) { return ((model*)mdl)->weight_bytes_total; }
-void lcu_model_free(void* mdl) { delete (model*)mdl; }
+uint64_t lcu_model_weight_bytes(void* mdl) { return ((model_base*)mdl)->weight_bytes_total; }
+void lcu_model_free(void* mdl) { delete (model_base*)mdl; }
 uint32_t lcu_ffn_dim(uint32_t dim, uint32_t multiple_of) {
   model_params p{};
   p.dim = dim;
@@ -417,7 +503,7 @@ int lcu_context_create(void* mdl, int context_len, float temperature, void** ctx
   opt.context_len = context_len;
   opt.temperature = temperature;
   std::unique_ptr<context> c;
-  int rc = context::create(c, (model*)mdl, opt);
+  int rc = context::create(c, (model_base*)mdl, opt);
   if (rc) return rc;
   *ctx_out = c.release();
   return LCU_OK;
@@ -428,6 +514,9 @@ uint64_t lcu_context_memory_usage(void* ctx) { return ((context*)ctx)->memory_us
 int lcu_context_tokens_left(void* ctx) { return ((context*)ctx)->tokens_left(); }
 int lcu_context_next_token(void* ctx, const int16_t* tokens_host, int n_tokens, int* token_out) {
   return ((context*)ctx)->next_token(tokens_host, n_tokens, token_out);
+}
+int lcu_context_step(void* ctx, const int16_t* tokens_host, int n_tokens, const int32_t* want_host, int n_want, float* logits_host, int* token_out) {
+  return ((context*)ctx)->step(tokens_host, n_tokens, want_host, n_want, logits_host, token_out);
 }
 int lcu_context_decode_chained(void* ctx, int16_t first_token, int n_steps, int16_t* tokens_host_out, float* ms_out) {
   return ((context*)ctx)->decode_chained(first_token, n_steps, tokens_host_out, ms_out);

@@ -1,0 +1,50 @@
+// Element conversions, the gate function and the clustered launch shared by the block-model kernels.
+#pragma once
+#include <cuda_bf16.h>
+
+#include "common.cuh"
+
+namespace lcu {
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T>
+__device__ __forceinline__ T from_f(float v);
+template <>
+__device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+__host__ __device__ __forceinline__ int round_up_dev(int a, int b) { return (a + b - 1) / b * b; }
+
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+
+// launch of a kernel whose CTAs work in clusters of `cluster` (1: plain), as a programmatic dependent of the kernel before it
+template <typename... KP, typename... Args>
+int launch_clustered(void (*kernel)(KP...), int grid, int cluster, int threads, size_t smem, cudaStream_t stream, Args&&... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(grid);
+  cfg.blockDim = dim3(threads);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  int n = 0;
+  if (cluster > 1) {
+    attr[n].id = cudaLaunchAttributeClusterDimension;
+    attr[n].val.clusterDim.x = cluster;
+    attr[n].val.clusterDim.y = 1;
+    attr[n].val.clusterDim.z = 1;
+    ++n;
+  }
+  if (prompt_pdl()) {
+    attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[n].val.programmaticStreamSerializationAllowed = 1;
+    ++n;
+  }
+  cfg.attrs = attr;
+  cfg.numAttrs = n;
+  LCU_CUDA(cudaLaunchKernelEx(&cfg, kernel, static_cast<KP>(args)...));
+  return LCU_OK;
+}
+
+}  // namespace lcu

@@ -34,28 +34,46 @@ namespace {
 constexpr int BM = 128;      // output rows (tokens) per tile = TMEM lanes
 constexpr int BK = 64;       // K per stage: 64 halves = one 128-byte swizzled row
 constexpr int TC_THREADS = 192;
+template <typename T>
+constexpr tc_type tc_type_of() {
+  return sizeof(T) == 2 && tc_elem<T>::IDESC_FORMAT == 0 ? TC_F16 : TC_BF16;
+}
 constexpr int TC_MAX_STAGES = 12;  // one-SM kernel: barrier slots for the ring
 
-// half(acc + beta * previous) for 32 consecutive outputs of one row (64 bytes, 16-byte aligned)
-__device__ __forceinline__ void store_row_piece(__half* o, const float (&acc)[32], float beta) {
+// acc + beta * previous, rounded to the output type, for 32 consecutive outputs of one row (16-byte aligned)
+template <typename TO>
+__device__ __forceinline__ void store_row_piece(TO* o, const float (&acc)[32], float beta) {
+  using E = tc_elem<TO>;
   uint4 v[4];
   if (beta != 0.f) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) v[i] = reinterpret_cast<const uint4*>(o)[i];
   }
-  __half2* h = reinterpret_cast<__half2*>(v);
+  uint32_t* h = reinterpret_cast<uint32_t*>(v);
 #pragma unroll
   for (int i = 0; i < 16; ++i) {
     float a0 = acc[2 * i], a1 = acc[2 * i + 1];
     if (beta != 0.f) {
-      const float2 prev = __half22float2(h[i]);
+      const float2 prev = E::unpack(h[i]);
       a0 = fmaf(beta, prev.x, a0);
       a1 = fmaf(beta, prev.y, a1);
     }
-    h[i] = __floats2half2_rn(a0, a1);
+    h[i] = E::pack(a0, a1);
   }
 #pragma unroll
   for (int i = 0; i < 4; ++i) reinterpret_cast<uint4*>(o)[i] = v[i];
+}
+template <>
+__device__ __forceinline__ void store_row_piece<float>(float* o, const float (&acc)[32], float beta) {
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    float4 v = make_float4(acc[4 * i], acc[4 * i + 1], acc[4 * i + 2], acc[4 * i + 3]);
+    if (beta != 0.f) {
+      const float4 p = reinterpret_cast<const float4*>(o)[i];
+      v = make_float4(fmaf(beta, p.x, v.x), fmaf(beta, p.y, v.y), fmaf(beta, p.z, v.z), fmaf(beta, p.w, v.w));
+    }
+    reinterpret_cast<float4*>(o)[i] = v;
+  }
 }
 __device__ __forceinline__ void st_dsmem_f4(uint32_t addr, float a, float b, float c, float d) {
   asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "f"(a), "f"(b), "f"(c), "f"(d) : "memory");
@@ -66,9 +84,10 @@ __device__ __forceinline__ void st_dsmem_f4(uint32_t addr, float a, float b, flo
 // CTA r accumulates k-blocks [r nk / S, (r+1) nk / S), then owns the BN / S output columns starting at
 // r BN / S: every CTA pushes its fp32 partials of the columns it does not own into the owner's shared
 // memory (distributed shared memory), one cluster barrier, and the owner adds them in rank order.
-template <int BN, int S>
+// T: operand type (__half or __nv_bfloat16); TO: output type (T, or float for results that feed a 32-bit sum).
+template <typename T, typename TO, int BN, int S>
 __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
-                                                                __half* out, int m, int N, int K, float beta, int nstages, int a_box_rows,
+                                                                TO* out, int m, int N, int K, float beta, int nstages, int a_box_rows,
                                                                 int kbs, int* err) {
   // A stage holds the activation box (a_box_rows rows, 2 to 16 KB) and the BN weight rows.  The MMA reads 128 operand rows
   // from the box's address: with a short box the rest comes from whatever follows in the ring, reaches output rows >= m
@@ -81,8 +100,8 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const __grid_con
   const uint32_t A_BYTES = (uint32_t)a_box_rows * (BK * 2), STAGE = (uint32_t)kbs * (A_BYTES + B_BYTES);
   constexpr int MAXS = TC_MAX_STAGES;
   constexpr uint32_t TM_COLS = BN <= 32 ? 32 : BN <= 64 ? 64 : BN <= 128 ? 128 : 256;  // tensor memory comes in powers of two
-  // instruction descriptor: fp32 accumulate, fp16 x fp16, both K-major, N = BN, M = 128
-  constexpr uint32_t IDESC = (1u << 4) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
+  // instruction descriptor: fp32 accumulate, operand format, both K-major, N = BN, M = 128
+  constexpr uint32_t IDESC = (1u << 4) | tc_elem<T>::IDESC_FORMAT | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
   constexpr int CW = BN / S;        // columns owned by each CTA of the cluster
   constexpr int CPR = CW / 32;      // 32-column pieces per owner
   constexpr uint32_t RED_BYTES = S > 1 ? (S - 1) * BM * CW * 4 : 0;
@@ -235,11 +254,6 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const __grid_con
 //   empty[s]      one per CTA; the leader's MMA thread commits to both (commit with a CTA mask)
 //   acc_full[b]   one per CTA; committed to both when a tile's last MMA has been issued
 //   acc_empty[b]  leader only, 8 arrivals: the four epilogue warps of both CTAs
-__device__ __forceinline__ void tma_load_2d_pair(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar_cluster_addr) {
-  asm volatile("cp.async.bulk.tensor.2d.cta_group::2.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst),
-               "l"(map), "r"(x), "r"(y), "r"(bar_cluster_addr)
-               : "memory");
-}
 __device__ __forceinline__ void tma_load_3d_pair(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar_cluster_addr) {
   asm volatile("cp.async.bulk.tensor.3d.cta_group::2.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];" ::"r"(dst),
                "l"(map), "r"(x), "r"(y), "r"(z), "r"(bar_cluster_addr)
@@ -261,14 +275,14 @@ __device__ __forceinline__ void mbar_arrive_cluster(uint32_t bar_cluster_addr) {
   asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(bar_cluster_addr) : "memory");
 }
 
-template <int BN>  // weight rows per pair tile: 128 or 256
+template <typename T, typename TO, int BN>  // weight rows per pair tile: 128 or 256
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TC_THREADS, 1)
-    gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, __half* out, int m, int N, int K,
+    gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, TO* out, int m, int N, int K,
                         float beta, int nstages, int tiles_m, int n_tiles, int kbs, int* err) {
   // (a stage is kbs k-blocks, one three-dimensional tensor copy per operand, as in the one-SM kernel)
   constexpr uint32_t A_BYTES = BM * BK * 2, B_BYTES = (BN / 2) * BK * 2;
   const uint32_t STAGE = (uint32_t)kbs * (A_BYTES + B_BYTES);
-  constexpr uint32_t IDESC = (1u << 4) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)((2 * BM) >> 4) << 24);
+  constexpr uint32_t IDESC = (1u << 4) | tc_elem<T>::IDESC_FORMAT | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)((2 * BM) >> 4) << 24);
   constexpr uint32_t TMEM_COLS = 2 * BN;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -412,53 +426,8 @@ int get_encoder(encode_fn* out) {
   return LCU_OK;
 }
 
-// [rows][K] halves, row-major; box = box_rows x 64 halves with 128-byte swizzle; rows past the end read as zero.
-// Encoded maps are kept (a map depends on address and shape only), so that a prompt's 7 products per layer
-// do not pay for two driver calls each.
-struct map_key {
-  const void* ptr;
-  uint64_t rows, K, ld;
-  uint32_t box_rows;
-  bool operator==(const map_key& o) const { return ptr == o.ptr && rows == o.rows && K == o.K && ld == o.ld && box_rows == o.box_rows; }
-};
-struct map_key_hash {
-  size_t operator()(const map_key& k) const {
-    uint64_t h = (uint64_t)(uintptr_t)k.ptr * 0x9e3779b97f4a7c15ull;
-    h ^= (k.rows + 0x632be59bd9b4e019ull) * 0xff51afd7ed558ccdull;
-    h ^= (k.K * 31 + k.ld * 17 + k.box_rows) * 0xc4ceb9fe1a85ec53ull;
-    return (size_t)(h ^ (h >> 29));
-  }
-};
-
-int make_map(CUtensorMap* map, const void* ptr, uint64_t rows, uint64_t K, uint64_t ld, uint32_t box_rows, bool streamed) {
-  static std::mutex mu;
-  static std::unordered_map<map_key, CUtensorMap, map_key_hash> cache;
-  const map_key key{ptr, rows, K, ld, box_rows};
-  std::lock_guard<std::mutex> lock(mu);
-  auto it = cache.find(key);
-  if (it != cache.end()) {
-    *map = it->second;
-    return LCU_OK;
-  }
-  encode_fn enc;
-  int rc = get_encoder(&enc);
-  if (rc) return rc;
-  const cuuint64_t dims[2] = {K, rows};
-  const cuuint64_t strides[1] = {ld * 2};
-  const cuuint32_t box[2] = {(cuuint32_t)BK, box_rows};
-  const cuuint32_t estr[2] = {1, 1};
-  const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                         CU_TENSOR_MAP_SWIZZLE_128B, streamed ? CU_TENSOR_MAP_L2_PROMOTION_L2_256B : CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-                         CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  LCU_REQUIRE(r == CUDA_SUCCESS, "cuTensorMapEncodeTiled failed with code %d (ptr %p rows %llu K %llu ld %llu)", (int)r, ptr,
-              (unsigned long long)rows, (unsigned long long)K, (unsigned long long)ld);
-  if (cache.size() >= 8192) cache.clear();
-  cache.emplace(key, *map);
-  return LCU_OK;
-}
-
-template <int BN, int S>
-int launch_bn(__half* out, const __half* lhs, int ldx, const __half* w, int m, int N, int K, float beta, int* err, cudaStream_t stream) {
+template <typename T, typename TO, int BN, int S>
+int launch_bn(void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream) {
   CUtensorMap map_a, map_b;
   const int a_box_rows = m > 64 ? BM : m > 32 ? 64 : m > 16 ? 32 : 16;
   constexpr size_t RED = S > 1 ? (size_t)(S - 1) * BM * (BN / S) * 4 : 0;
@@ -490,7 +459,7 @@ int launch_bn(__half* out, const __half* lhs, int ldx, const __half* w, int m, i
   int dev = 0;
   LCU_CUDA(cudaGetDevice(&dev));
   if (dev < 16 && !attr_done[dev]) {
-    LCU_CUDA(cudaFuncSetAttribute(gemm_tc_kernel<BN, S>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    LCU_CUDA(cudaFuncSetAttribute((gemm_tc_kernel<T, TO, BN, S>), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     attr_done[dev] = true;
   }
   cudaLaunchConfig_t cfg = {};
@@ -514,12 +483,12 @@ int launch_bn(__half* out, const __half* lhs, int ldx, const __half* w, int m, i
   }
   cfg.attrs = attr;
   cfg.numAttrs = n_attr;
-  LCU_CUDA(cudaLaunchKernelEx(&cfg, gemm_tc_kernel<BN, S>, map_a, map_b, out, m, N, K, beta, nstages, a_box_rows, kbs, err));
+  LCU_CUDA(cudaLaunchKernelEx(&cfg, gemm_tc_kernel<T, TO, BN, S>, map_a, map_b, (TO*)out, m, N, K, beta, nstages, a_box_rows, kbs, err));
   return LCU_OK;
 }
 
-template <int BN>
-int launch_pair(__half* out, const __half* lhs, int ldx, const __half* w, int m, int N, int K, float beta, int* err, cudaStream_t stream) {
+template <typename T, typename TO, int BN>
+int launch_pair(void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream) {
   CUtensorMap map_a, map_b;
   int kbs = sk_kb_per_stage();  // k-blocks per stage and tensor copy
   if (kbs <= 0) kbs = 2;
@@ -542,13 +511,13 @@ int launch_pair(__half* out, const __half* lhs, int ldx, const __half* w, int m,
   int dev = 0;
   LCU_CUDA(cudaGetDevice(&dev));
   if (dev < 16 && !attr_done[dev]) {
-    LCU_CUDA(cudaFuncSetAttribute(gemm_tc_pair_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    LCU_CUDA(cudaFuncSetAttribute((gemm_tc_pair_kernel<T, TO, BN>), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     attr_done[dev] = true;
   }
   const int tiles_m = (m + 2 * BM - 1) / (2 * BM), n_tiles = tiles_m * (N / BN);
   int clusters = gemv_sm_count() / 2;
   if (clusters > n_tiles) clusters = n_tiles;
-  LCU_CUDA(launch_after(gemm_tc_pair_kernel<BN>, dim3(2 * clusters), dim3(TC_THREADS), smem, stream, map_a, map_b, out, m, N, K, beta, nstages, tiles_m,
+  LCU_CUDA(launch_after(gemm_tc_pair_kernel<T, TO, BN>, dim3(2 * clusters), dim3(TC_THREADS), smem, stream, map_a, map_b, (TO*)out, m, N, K, beta, nstages, tiles_m,
                         n_tiles, kbs, err));
   return LCU_OK;
 }
@@ -704,8 +673,10 @@ bool gemm_tc_supported(int m, int N, int K, int ldx, const void* lhs, const void
          ((uintptr_t)out & 15) == 0;
 }
 
-int launch_gemm_tc(__half* out, const __half* lhs, int ldx, const __half* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
-                   int force_bn, int force_pair, int force_split) {
+namespace {
+template <typename T, typename TO>
+int launch_gemm_shape(void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
+                      int force_bn, int force_pair, int force_split) {
   LCU_REQUIRE(gemm_tc_supported(m, N, K, ldx, lhs, w, out), "gemm_tc: unsupported shape m=%d N=%d K=%d ldx=%d or unaligned pointers", m, N, K, ldx);
   const int sms = gemv_sm_count();
   // More than 128 rows: three kernels can run the product - whole tiles per SM pair (below), the kernel that deals the
@@ -713,11 +684,12 @@ int launch_gemm_tc(__half* out, const __half* lhs, int ldx, const __half* w, int
   // 512-wide tiles (a third less operand traffic per multiply-add, no overlap of epilogue and main loop).  Which one is
   // fastest depends on how the tile count meets the 74 pairs (gemm_tc_estimates).  Mode -1 = that rule; 256 / 512 force
   // the balanced kernel with that tile width; 0 = never.
-  if (force_pair < 0 && !force_bn && (m > BM || gemm_tc_sk_mode() > 0)) {
+  // (the balanced kernel stores 16-bit results only)
+  if (sizeof(TO) == 2 && force_pair < 0 && !force_bn && (m > BM || gemm_tc_sk_mode() > 0)) {
     const int mode = gemm_tc_sk_mode();
     int tile = mode > 0 ? mode : 0;
     if (mode < 0) tile = gemm_tc_plan_long(m, N, K, sms);
-    if (tile && gemm_tc_sk_supported(m, N, K, ldx, lhs, w, out, tile)) return launch_gemm_tc_sk(out, lhs, ldx, w, m, N, K, beta, err, stream, tile);
+    if (tile && gemm_tc_sk_supported(m, N, K, ldx, lhs, w, out, tile)) return launch_gemm_tc_sk(tc_type_of<T>(), out, lhs, ldx, w, m, N, K, beta, err, stream, tile);
   }
   // Large products: the two-SM kernel, with its 256-wide tile when that still gives (nearly) every SM pair a tile.
   // Up to 256 rows of a matrix with few tiles stay on the one-SM kernel, which can split K to fill the SMs.
@@ -731,7 +703,7 @@ int launch_gemm_tc(__half* out, const __half* lhs, int ldx, const __half* w, int
   }
   if (pair) {
     LCU_REQUIRE((pair == 128 || pair == 256) && N % pair == 0, "gemm_tc: pair tile width %d does not divide N=%d", pair, N);
-    return pair == 256 ? launch_pair<256>(out, lhs, ldx, w, m, N, K, beta, err, stream) : launch_pair<128>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+    return pair == 256 ? launch_pair<T, TO, 256>(out, lhs, ldx, w, m, N, K, beta, err, stream) : launch_pair<T, TO, 128>(out, lhs, ldx, w, m, N, K, beta, err, stream);
   }
   int bn = force_bn, split = force_split;
   if (!bn) bn = N % 128 == 0 ? 128 : N % 64 == 0 ? 64 : 32;  // measured: the widest tile wins even when it leaves SMs idle
@@ -745,19 +717,31 @@ int launch_gemm_tc(__half* out, const __half* lhs, int ldx, const __half* w, int
     }
     if (K / BK < 8 * split) split = 1;  // every CTA of the cluster needs k-blocks of its own
     LCU_REQUIRE(split == 1 || split == 2 || split == 4, "gemm_tc: split-K factor %d is not 1, 2 or 4", split);
-    if (split == 4) return launch_bn<128, 4>(out, lhs, ldx, w, m, N, K, beta, err, stream);
-    if (split == 2) return launch_bn<128, 2>(out, lhs, ldx, w, m, N, K, beta, err, stream);
-    return launch_bn<128, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+    if (split == 4) return launch_bn<T, TO, 128, 4>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+    if (split == 2) return launch_bn<T, TO, 128, 2>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+    return launch_bn<T, TO, 128, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
   }
   switch (bn) {
-    case 32: return launch_bn<32, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
-    case 64: return launch_bn<64, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
-    case 96: return launch_bn<96, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
-    case 160: return launch_bn<160, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
-    case 192: return launch_bn<192, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
-    case 224: return launch_bn<224, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
-    default: return launch_bn<256, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+    case 32: return launch_bn<T, TO, 32, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+    case 64: return launch_bn<T, TO, 64, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+    case 96: return launch_bn<T, TO, 96, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+    case 160: return launch_bn<T, TO, 160, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+    case 192: return launch_bn<T, TO, 192, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+    case 224: return launch_bn<T, TO, 224, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+    default: return launch_bn<T, TO, 256, 1>(out, lhs, ldx, w, m, N, K, beta, err, stream);
   }
+}
+
+}  // namespace
+
+int launch_gemm_tc(tc_type type, void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
+                   int force_bn, int force_pair, int force_split) {
+  switch (type) {
+    case TC_F16: return launch_gemm_shape<__half, __half>(out, lhs, ldx, w, m, N, K, beta, err, stream, force_bn, force_pair, force_split);
+    case TC_BF16: return launch_gemm_shape<__nv_bfloat16, __nv_bfloat16>(out, lhs, ldx, w, m, N, K, beta, err, stream, force_bn, force_pair, force_split);
+    case TC_BF16_F32: return launch_gemm_shape<__nv_bfloat16, float>(out, lhs, ldx, w, m, N, K, beta, err, stream, force_bn, force_pair, force_split);
+  }
+  LCU_REQUIRE(false, "gemm_tc: unknown operand type %d", (int)type);
 }
 
 }  // namespace lcu

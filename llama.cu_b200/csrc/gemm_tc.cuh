@@ -5,6 +5,10 @@
 
 namespace lcu {
 
+// operand and output types of the tensor-core products: halves in and out, bfloat16 in and out, bfloat16 in and binary32
+// out (results that are added to a 32-bit residual)
+enum tc_type : int { TC_F16 = 0, TC_BF16 = 1, TC_BF16_F32 = 2 };
+
 // shapes the kernel takes: N a multiple of 32, K a multiple of 64, 16-byte aligned rows
 bool gemm_tc_supported(int m, int N, int K, int ldx, const void* lhs, const void* w, const void* out);
 
@@ -14,8 +18,12 @@ bool gemm_tc_supported(int m, int N, int K, int ldx, const void* lhs, const void
 //             0 = never, 128 / 256 = always with that tile width.
 // force_split: -1 = the one-SM kernel splits K over a cluster of 2 or 4 CTAs when its tiles would fill
 //             less than half / a quarter of the SMs; 1 / 2 / 4 forces the factor (128-wide tiles only).
-int launch_gemm_tc(__half* out, const __half* lhs, int ldx, const __half* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
+int launch_gemm_tc(tc_type type, void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
                    int force_bn = 0, int force_pair = -1, int force_split = -1);
+inline int launch_gemm_tc(__half* out, const __half* lhs, int ldx, const __half* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
+                          int force_bn = 0, int force_pair = -1, int force_split = -1) {
+  return launch_gemm_tc(TC_F16, out, lhs, ldx, w, m, N, K, beta, err, stream, force_bn, force_pair, force_split);
+}
 
 // Wide-tile variant with the K loop balanced over the SM pairs (gemm_tc_sk.cu): 256 x tile_n output tiles (tile_n 256 or
 // 512, dividing N), any number of rows.  Partial sums of tiles shared between pairs go through a workspace kept per
@@ -34,7 +42,7 @@ int& tc_kb_per_stage();
 // balanced pair kernel: k-blocks per stage and tensor copy (0 = 2)
 int& sk_kb_per_stage();
 bool gemm_tc_sk_supported(int m, int N, int K, int ldx, const void* lhs, const void* w, const void* out, int tile_n);
-int launch_gemm_tc_sk(__half* out, const __half* lhs, int ldx, const __half* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
+int launch_gemm_tc_sk(tc_type type, void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
                       int tile_n);
 
 // host walk of the balanced kernel's schedule for n_tiles tiles of nk K steps on C SM pairs: 0 = every K step of every tile
@@ -49,7 +57,11 @@ int& gemm_tc_gate_mode();
 int gemm_tc_gated_tile(int m, int f, int K);
 bool gemm_tc_gated_supported(int m, int f, int K, int ldx, const void* lhs, const void* w13, const void* out);
 // tile_n: accumulator columns per tile (256: 128 output columns, the gate hidden under the next tile; 512: 256 output columns)
-int launch_gemm_tc_gated(__half* out, const __half* lhs, int ldx, const __half* w13, int m, int f, int K, int* err, cudaStream_t stream,
+int launch_gemm_tc_gated(tc_type type, void* out, const void* lhs, int ldx, const void* w13, int m, int f, int K, int* err, cudaStream_t stream,
                          int tile_n = 256);
+inline int launch_gemm_tc_gated(__half* out, const __half* lhs, int ldx, const __half* w13, int m, int f, int K, int* err, cudaStream_t stream,
+                                int tile_n = 256) {
+  return launch_gemm_tc_gated(TC_F16, out, lhs, ldx, w13, m, f, K, err, stream, tile_n);
+}
 
 }  // namespace lcu

@@ -35,11 +35,6 @@ constexpr int SK_BK = 64;
 constexpr int SK_THREADS = 192;
 constexpr int DEV_ERR_PARTIAL_WAIT = 0x107;  // a tile's owner timed out waiting for another pair's partial sums
 
-__device__ __forceinline__ void sk_tma_load_pair(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar_cluster_addr) {
-  asm volatile("cp.async.bulk.tensor.2d.cta_group::2.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst),
-               "l"(map), "r"(x), "r"(y), "r"(bar_cluster_addr)
-               : "memory");
-}
 __device__ __forceinline__ void sk_tma_load_pair_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar_cluster_addr) {
   asm volatile("cp.async.bulk.tensor.3d.cta_group::2.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];" ::"r"(dst),
                "l"(map), "r"(x), "r"(y), "r"(z), "r"(bar_cluster_addr)
@@ -159,7 +154,7 @@ struct sk_schedule {
 // and the SiLU gate as one launch, without the [rows][2 f] intermediate.  With NB = 1 each CTA of the pair loads one
 // matrix's 128 rows, and the gate's arithmetic (a division and an exponential per element on four warps) runs under the
 // next tile's main loop.
-template <int NB, bool GATE>
+template <typename T, int NB, bool GATE>  // T: __half or __nv_bfloat16 ("half" above stands for either)
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(SK_THREADS, 1)
     gemm_tc_sk_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                       const __grid_constant__ CUtensorMap map_out, int m, int N, int K,
@@ -171,7 +166,8 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(SK_THREADS, 1)
   // three-dimensional tensor copy (64 halves x 128 rows x kbs k-blocks)
   constexpr uint32_t A_BYTES = SK_BM * SK_BK * 2, B_BYTES = 128 * SK_BK * 2;
   const uint32_t STAGE = (uint32_t)kbs * (A_BYTES + NB * B_BYTES);
-  constexpr uint32_t IDESC = (1u << 4) | ((uint32_t)(256 >> 3) << 17) | ((uint32_t)(256 >> 4) << 24);  // fp32 acc, fp16 x fp16, K-major, N = 256, M = 256
+  using E = tc_elem<T>;
+  constexpr uint32_t IDESC = (1u << 4) | E::IDESC_FORMAT | ((uint32_t)(256 >> 3) << 17) | ((uint32_t)(256 >> 4) << 24);  // fp32 acc, K-major, N = 256, M = 256
   constexpr int NBUF = NB == 1 ? 2 : 1;  // accumulator buffers: the epilogue of one segment runs under the main loop of the next
   constexpr uint32_t TMEM_COLS = BN * NBUF;
   extern __shared__ uint8_t smem_raw[];
@@ -399,27 +395,20 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(SK_THREADS, 1)
           }
           if (GATE && (idx & 1) == 0) {
 #pragma unroll
-            for (int i = 0; i < 16; ++i) {
-              const __half2 h = __floats2half2_rn(sum[2 * i], sum[2 * i + 1]);
-              first[i] = *reinterpret_cast<const uint32_t*>(&h);
-            }
+            for (int i = 0; i < 16; ++i) first[i] = E::pack(sum[2 * i], sum[2 * i + 1]);
             continue;
           }
           uint32_t outw[16];  // the piece's 32 output halves (beta = 0 paths)
           if (GATE) {
 #pragma unroll
             for (int i = 0; i < 16; ++i) {
-              const float2 a = __half22float2(*reinterpret_cast<const __half2*>(&first[i]));
-              const float2 bq = __half22float2(__floats2half2_rn(sum[2 * i], sum[2 * i + 1]));
-              const __half2 gt = __halves2half2(__float2half(silu_of_half(a.x) * bq.x), __float2half(silu_of_half(a.y) * bq.y));
-              outw[i] = *reinterpret_cast<const uint32_t*>(&gt);
+              const float2 a = E::unpack(first[i]);
+              const float2 bq = E::unpack(E::pack(sum[2 * i], sum[2 * i + 1]));
+              outw[i] = E::pack(silu_of_half(a.x) * bq.x, silu_of_half(a.y) * bq.y);
             }
           } else {
 #pragma unroll
-            for (int i = 0; i < 16; ++i) {
-              const __half2 h = __floats2half2_rn(sum[2 * i], sum[2 * i + 1]);
-              outw[i] = *reinterpret_cast<const uint32_t*>(&h);
-            }
+            for (int i = 0; i < 16; ++i) outw[i] = E::pack(sum[2 * i], sum[2 * i + 1]);
           }
           // results go out through shared memory: the warp's 32 rows x 64 columns are stored by one bulk tensor copy
           // (rows are 44 KB apart in memory; stores of 64 bytes per thread kept the load/store unit busy for longer
@@ -450,12 +439,12 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(SK_THREADS, 1)
             const uint32_t at = rowb + ((uint32_t)((((c & 32) >> 3) + i) ^ (lane & 7)) << 4);
             uint4 v = make_uint4(outw[4 * i], outw[4 * i + 1], outw[4 * i + 2], outw[4 * i + 3]);
             if (!GATE && beta != 0.f) {
-              __half2* h = reinterpret_cast<__half2*>(&v);
+              uint32_t* h = reinterpret_cast<uint32_t*>(&v);
               asm volatile("ld.shared.v4.b32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "r"(at) : "memory");
 #pragma unroll
               for (int e = 0; e < 4; ++e) {
-                const float2 prev = __half22float2(h[e]);
-                h[e] = __floats2half2_rn(fmaf(beta, prev.x, sum[8 * i + 2 * e]), fmaf(beta, prev.y, sum[8 * i + 2 * e + 1]));
+                const float2 prev = E::unpack(h[e]);
+                h[e] = E::pack(fmaf(beta, prev.x, sum[8 * i + 2 * e]), fmaf(beta, prev.y, sum[8 * i + 2 * e + 1]));
               }
             }
             asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(at), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
@@ -535,8 +524,8 @@ int& sk_kb_per_stage() {
 namespace {
 
 // GATE: w is the stack [w1; w3] of two [N][K] matrices and out is [m][N]
-template <int NB, bool GATE>
-int launch_sk(__half* out, const __half* lhs, int ldx, const __half* w, int m, int N, int K, float beta, int* err, cudaStream_t stream) {
+template <typename T, int NB, bool GATE>
+int launch_sk(void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream) {
   constexpr int BN = 256 * NB;
   constexpr int BN_OUT = GATE ? BN / 2 : BN;
   CUtensorMap map_a, map_b;
@@ -570,7 +559,7 @@ int launch_sk(__half* out, const __half* lhs, int ldx, const __half* w, int m, i
   int dev = 0;
   LCU_CUDA(cudaGetDevice(&dev));
   if (dev < 16 && !attr_done[dev]) {
-    LCU_CUDA(cudaFuncSetAttribute(gemm_tc_sk_kernel<NB, GATE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    LCU_CUDA(cudaFuncSetAttribute((gemm_tc_sk_kernel<T, NB, GATE>), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     attr_done[dev] = true;
   }
   const int tiles_m = (m + 2 * SK_BM - 1) / (2 * SK_BM), n_tiles = tiles_m * (N / BN_OUT);
@@ -580,7 +569,7 @@ int launch_sk(__half* out, const __half* lhs, int ldx, const __half* w, int m, i
   int rc = sk_get_workspace(dev, stream, (size_t)clusters * 256 * BN, clusters, &ws);
   if (rc) return rc;
   const int seq = ++ws->seq;
-  LCU_CUDA(launch_after(gemm_tc_sk_kernel<NB, GATE>, dim3(2 * clusters), dim3(SK_THREADS), smem, stream, map_a, map_b, map_out, m, N, K, beta, nstages,
+  LCU_CUDA(launch_after(gemm_tc_sk_kernel<T, NB, GATE>, dim3(2 * clusters), dim3(SK_THREADS), smem, stream, map_a, map_b, map_out, m, N, K, beta, nstages,
                         tiles_m, n_tiles, ws->partials, ws->flags, seq, err, GATE ? N : 0, kbs));
   return LCU_OK;
 }
@@ -592,21 +581,31 @@ bool gemm_tc_sk_supported(int m, int N, int K, int ldx, const void* lhs, const v
          ((uintptr_t)w & 15) == 0 && ((uintptr_t)out & 15) == 0;
 }
 
-int launch_gemm_tc_sk(__half* out, const __half* lhs, int ldx, const __half* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
+int launch_gemm_tc_sk(tc_type type, void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
                       int tile_n) {
   LCU_REQUIRE(gemm_tc_sk_supported(m, N, K, ldx, lhs, w, out, tile_n), "gemm_tc_sk: unsupported shape m=%d N=%d K=%d ldx=%d tile %d", m, N, K, ldx,
               tile_n);
-  return tile_n == 512 ? launch_sk<2, false>(out, lhs, ldx, w, m, N, K, beta, err, stream) : launch_sk<1, false>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+  LCU_REQUIRE(type == TC_F16 || type == TC_BF16, "gemm_tc_sk: output type %d is not a 16-bit one", (int)type);
+  if (type == TC_BF16)
+    return tile_n == 512 ? launch_sk<__nv_bfloat16, 2, false>(out, lhs, ldx, w, m, N, K, beta, err, stream)
+                         : launch_sk<__nv_bfloat16, 1, false>(out, lhs, ldx, w, m, N, K, beta, err, stream);
+  return tile_n == 512 ? launch_sk<__half, 2, false>(out, lhs, ldx, w, m, N, K, beta, err, stream)
+                       : launch_sk<__half, 1, false>(out, lhs, ldx, w, m, N, K, beta, err, stream);
 }
 
 bool gemm_tc_gated_supported(int m, int f, int K, int ldx, const void* lhs, const void* w, const void* out) {
   return m >= 1 && f % 128 == 0 && K % SK_BK == 0 && ldx % 8 == 0 && ((uintptr_t)lhs & 15) == 0 && ((uintptr_t)w & 15) == 0 && ((uintptr_t)out & 15) == 0;
 }
 
-int launch_gemm_tc_gated(__half* out, const __half* lhs, int ldx, const __half* w13, int m, int f, int K, int* err, cudaStream_t stream, int tile_n) {
+int launch_gemm_tc_gated(tc_type type, void* out, const void* lhs, int ldx, const void* w13, int m, int f, int K, int* err, cudaStream_t stream, int tile_n) {
   LCU_REQUIRE(gemm_tc_gated_supported(m, f, K, ldx, lhs, w13, out) && (tile_n == 256 || (tile_n == 512 && f % 256 == 0)),
               "gemm_tc_gated: unsupported shape m=%d f=%d K=%d ldx=%d tile=%d", m, f, K, ldx, tile_n);
-  return tile_n == 512 ? launch_sk<2, true>(out, lhs, ldx, w13, m, f, K, 0.f, err, stream) : launch_sk<1, true>(out, lhs, ldx, w13, m, f, K, 0.f, err, stream);
+  LCU_REQUIRE(type == TC_F16 || type == TC_BF16, "gemm_tc_gated: output type %d is not a 16-bit one", (int)type);
+  if (type == TC_BF16)
+    return tile_n == 512 ? launch_sk<__nv_bfloat16, 2, true>(out, lhs, ldx, w13, m, f, K, 0.f, err, stream)
+                         : launch_sk<__nv_bfloat16, 1, true>(out, lhs, ldx, w13, m, f, K, 0.f, err, stream);
+  return tile_n == 512 ? launch_sk<__half, 2, true>(out, lhs, ldx, w13, m, f, K, 0.f, err, stream)
+                       : launch_sk<__half, 1, true>(out, lhs, ldx, w13, m, f, K, 0.f, err, stream);
 }
 
 // The schedule, walked on the host for every pair of a launch: 0 when every K step of every tile is run exactly once,

@@ -10,6 +10,8 @@ enum gemv_epilogue : int {
   EPI_SILU = 2      // two matrices w1|w3 interleaved row by row: out[i] = half(silu(half(a_i)) * half(b_i))
 };
 
+constexpr int GEMV_MAX_BATCH = 6;
+
 struct gemv_params {
   // weights: up to three [rows_per_mat][K] matrices that share K; fp16, or u8 with fp16 scales [rows][K/bs]
   const void* w[3];
@@ -52,6 +54,22 @@ struct gemv_params {
   int exchange_id;         // the value published is *seq * 1024 + exchange_id
   const int* seq;          // device scalar: number of the decode step in flight (monotonic over the context's life)
 };
+
+// bfloat16 weights and activations (gemv_params::bf16): one row, no fused norm; the gate epilogue works on the binary32 sums.
+// EPI_PLAIN may run several matrices with an input vector each in one launch (a recurrent layer's projections); n_batch
+// entries, every one with rows_b[i] rows of K, written to out_b[i].
+struct gemv_batch {
+  int n = 0;
+  const void* w[GEMV_MAX_BATCH];
+  const void* x[GEMV_MAX_BATCH];
+  void* out[GEMV_MAX_BATCH];
+  int rows[GEMV_MAX_BATCH];
+  int f32[GEMV_MAX_BATCH];              // output type: 0 bfloat16, 1 binary32
+  int first_cta[GEMV_MAX_BATCH + 1];    // filled in by the launch
+};
+int launch_gemv_bf16(const gemv_batch& b, int K, int* err, cudaStream_t stream, int pdl);
+// out[f] = bfloat16(silu(w1 . x) * (w3 . x)), w13 = [w1; w3] stacked ([2 f][K])
+int launch_gemv_bf16_gated(void* out, const void* x, const void* w13, int f, int K, int* err, cudaStream_t stream, int pdl);
 
 constexpr int TP_EXCHANGES_PER_STEP = 1024;  // bound of the exchange ids of one decode step
 

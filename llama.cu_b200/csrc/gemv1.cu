@@ -22,10 +22,15 @@
 // dependent launch the rings of kernel n+1 fill while kernel n drains; every wait is bounded; int8
 // weights are de-quantised in registers bit-identically to half((q - 127.5f) * scale)
 // (reference llama_cu.cu:287-289); the RMSNorm prologue keeps the reference's summation order.
+#include <cuda_bf16.h>
+
 #include "gemv.cuh"
 
 namespace lcu {
 namespace {
+
+template <int WT>
+constexpr bool is16 = WT == 0 || WT == 3;  // two-byte weights: halves (0) or bfloat16 (3)
 
 // Consumer warps per CTA (template parameter of the kernel): 4, or 5 for u8 kernels whose activation row leaves room
 // for two CTAs per SM only - ten consumer warps per SM instead of eight, the u8 kernels being latency-bound.
@@ -74,7 +79,7 @@ template <int WT, bool FULL>
 __device__ __forceinline__ void step(float (&accs)[NACC][4], const int s, const int flip, const int c, const int g, const int vb,
                                      const uint8_t* seg0, const uint8_t* xseg, const uint8_t* st, const float* xs64, const int ci,
                                      const int bs) {
-  constexpr int ESZ = WT == 0 ? 2 : 1;
+  constexpr int ESZ = is16<WT> ? 2 : 1;
   constexpr int ROWB = geom<WT>::ROWB, SEG = geom<WT>::SEG, NSTEPS = geom<WT>::NSTEPS;
   constexpr int CHUNK_K = ROWB / ESZ;
   float* acc = accs[(2 * s) % NACC];
@@ -86,11 +91,16 @@ __device__ __forceinline__ void step(float (&accs)[NACC][4], const int s, const 
     lo = *reinterpret_cast<const uint4*>(seg0 + off);
     hi = *reinterpret_cast<const uint4*>(seg0 + ROWB + off);
   }
-  if (WT == 0) {
+  if (is16<WT>) {
     uint4 xb = make_uint4(0, 0, 0, 0);
     if (ok) xb = *reinterpret_cast<const uint4*>(xseg + off);
-    mma_16816(acc, lo.x, hi.x, lo.y, hi.y, xb.x, xb.y);
-    mma_16816(acc_b, lo.z, hi.z, lo.w, hi.w, xb.z, xb.w);
+    if (WT == 3) {
+      mma_16816_bf16(acc, lo.x, hi.x, lo.y, hi.y, xb.x, xb.y);
+      mma_16816_bf16(acc_b, lo.z, hi.z, lo.w, hi.w, xb.z, xb.w);
+    } else {
+      mma_16816(acc, lo.x, hi.x, lo.y, hi.y, xb.x, xb.y);
+      mma_16816(acc_b, lo.z, hi.z, lo.w, hi.w, xb.z, xb.w);
+    }
   } else {
     uint4 x0 = make_uint4(0, 0, 0, 0), x1 = x0;
     __half sc_lo = __ushort_as_half(0), sc_hi = sc_lo;
@@ -186,15 +196,17 @@ __device__ __forceinline__ void step_pair_factored(float (&accs)[NACC][4], const
 // with the scale factored out of each 64-weight group: sum_k x_k (q_k - 127.5) s = s * (sum_k x_k
 // (1024 + q_k) - 1151.5 * sum_k x_k), the bytes going to the tensor core as the exact halves
 // 1024 + q (one PRMT per two weights) and the group sums of x coming from the prologue.  Mode 2 has
-// no per-weight rounding: it is closer to the exact product but is not the reference's rounding.
+// no per-weight rounding: it is closer to the exact product but is not the reference's rounding.  3 = bfloat16 weights and
+// activations: no fused norm or cache write; EPI_PLAIN runs the matrices of `bt`, each with its own vector, on runs of CTAs.
 template <int WT, int EPI, int NW>
-__global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(const gemv_params p, const int sw, const int pf_bytes) {
+__global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(const gemv_params p, const int sw, const int pf_bytes,
+                                                                                        const __grid_constant__ gemv_batch bt) {
   constexpr int NCONS = NW * 32;
   static_assert(NW >= 4 && NW <= NW_MAX, "the RMSNorm reduction uses the first four consumer warps");
-  constexpr int ESZ = WT == 0 ? 2 : 1;
+  constexpr int ESZ = is16<WT> ? 2 : 1;
   constexpr int ROWB = geom<WT>::ROWB, SEG = geom<WT>::SEG, NSTEPS = geom<WT>::NSTEPS;
   constexpr int CHUNK_K = ROWB / ESZ;        // weights of one row per stage
-  constexpr int STAGE_BYTES = 2 * ROWB + (WT ? 2 * geom<WT>::SC_ROW : 0);
+  constexpr int STAGE_BYTES = 2 * ROWB + (is16<WT> ? 0 : 2 * geom<WT>::SC_ROW);
 
   extern __shared__ __align__(128) uint8_t smem[];
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem);  // full: [w * MAX_SW + s], empty: [EMPTY_BASE + w * MAX_SW + s]
@@ -205,8 +217,8 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
   // u8 kernels read 32 activation bytes per 16 weight bytes; with the row stored flat, the two segments of a
   // quarter warp would meet on the same banks.  The activations of every segment are therefore shifted by 16 more
   // bytes than those of the one before (vector i of eight halves lives at byte 16 * (i + i / (SEG / 8))).
-  auto xoff = [](int vec_index) { return WT == 0 ? vec_index * 16 : (vec_index + (vec_index >> (geom<WT>::SEG_SHIFT - 3))) * 16; };
-  const int xbytes = WT == 0 ? p.K * 2 : p.K * 2 + (p.K >> geom<WT>::SEG_SHIFT) * 16 + 16;
+  auto xoff = [](int vec_index) { return is16<WT> ? vec_index * 16 : (vec_index + (vec_index >> (geom<WT>::SEG_SHIFT - 3))) * 16; };
+  const int xbytes = is16<WT> ? p.K * 2 : p.K * 2 + (p.K >> geom<WT>::SEG_SHIFT) * 16 + 16;
   float* xs64 = reinterpret_cast<float*>(xs + ((xbytes + 127) & ~127));  // sums of x over aligned groups of 64
   // norm weights beyond what the consumers hold in registers (rows longer than NVEC * 8 * consumer threads) are staged here
   uint8_t* nws = reinterpret_cast<uint8_t*>(xs64) + ((p.K / 64 * 4 + 127) & ~127);
@@ -215,18 +227,26 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   pdl_launch_dependents();
 
-  const int pairs = (p.n_mats * p.rows_per_mat) >> 1;
-  const int pr0 = (int)(((long long)pairs * blockIdx.x) / gridDim.x);
-  const int npairs = (int)(((long long)pairs * (blockIdx.x + 1)) / gridDim.x) - pr0;
+  int pairs = (p.n_mats * p.rows_per_mat) >> 1, cta = blockIdx.x, n_ctas = gridDim.x, bi = 0;
+  if (WT == 3 && EPI == EPI_PLAIN) {  // which of the batch's matrices this CTA works on
+    while (bi + 1 < bt.n && (int)blockIdx.x >= bt.first_cta[bi + 1]) ++bi;
+    cta = blockIdx.x - bt.first_cta[bi];
+    n_ctas = bt.first_cta[bi + 1] - bt.first_cta[bi];
+    pairs = bt.rows[bi] >> 1;
+  }
+  auto weights_of = [&](int mat) { return reinterpret_cast<const uint8_t*>(WT == 3 && EPI == EPI_PLAIN ? bt.w[bi] : p.w[mat]); };
+  const __half* x_row = WT == 3 && EPI == EPI_PLAIN ? reinterpret_cast<const __half*>(bt.x[bi]) : p.x;
+  const int pr0 = (int)(((long long)pairs * cta) / n_ctas);
+  const int npairs = (int)(((long long)pairs * (cta + 1)) / n_ctas) - pr0;
   const int rowbytes = p.K * ESZ;
   const int nchunks = (rowbytes + ROWB - 1) / ROWB;
 
   // Scales of a row chunk are one contiguous run; when rows start 16-byte aligned they travel as one more bulk copy
   // per row on the same barrier, otherwise as 4-byte cp.async pieces issued by all lanes (32 more barrier arrivals).
-  const bool sc_bulk = WT != 0 && ((p.K / p.bs) & 7) == 0 && ((ROWB / p.bs) & 7) == 0;
+  const bool sc_bulk = !is16<WT> && ((p.K / p.bs) & 7) == 0 && ((ROWB / p.bs) & 7) == 0;
   if (tid == 0) {
     for (int i = 0; i < NW * MAX_SW; ++i) {
-      mbar_init(smem_u32(&bars[i]), (WT == 0 || sc_bulk) ? 1 : 33);
+      mbar_init(smem_u32(&bars[i]), (is16<WT> || sc_bulk) ? 1 : 33);
       mbar_init(smem_u32(&bars[EMPTY_BASE + i]), 1);
     }
     mbar_init(xbar, 1);
@@ -245,7 +265,7 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
       for (int r = lane; r < rows_pf; r += 32) {
         int mat, row;
         map_row<EPI>(p, 2 * pr0 + r, mat, row);
-        l2_prefetch(reinterpret_cast<const uint8_t*>(p.w[mat]) + (size_t)row * rowbytes, (uint32_t)rowbytes);
+        l2_prefetch(weights_of(mat) + (size_t)row * rowbytes, (uint32_t)rowbytes);
       }
     }
     int slot[NW];
@@ -263,17 +283,17 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
     const uint32_t bars_u32 = smem_u32(bars), stages_u32 = smem_u32(stages);
     const bool lane_sc = lane >= 2;
     const bool lane_copies = lane < 2 || (sc_bulk && (lane == 2 || lane == 16));
-    const uint32_t lane_dst = lane_sc ? 2 * ROWB + (lane >> 4) * (WT ? geom<WT>::SC_ROW : 0) : lane * ROWB;
+    const uint32_t lane_dst = lane_sc ? 2 * ROWB + (lane >> 4) * (is16<WT> ? 0 : geom<WT>::SC_ROW) : lane * ROWB;
     auto issue = [&](const int w, const uint8_t* row_src, const __half* sc_src, const int cbytes) {
       const uint32_t full = bars_u32 + (uint32_t)(w * MAX_SW + slot[w]) * 8;
       mbar_wait(full + EMPTY_BASE * 8, par[w] ^ 1, p.err, DEV_ERR_EMPTY_WAIT);
       const uint32_t st = stages_u32 + (uint32_t)(w * sw + slot[w]) * STAGE_BYTES;
-      const uint32_t scbytes = WT != 0 ? (uint32_t)(cbytes >> bs_shift) * 2 : 0;  // scale bytes per row of this chunk
+      const uint32_t scbytes = !is16<WT> ? (uint32_t)(cbytes >> bs_shift) * 2 : 0;  // scale bytes per row of this chunk
       if (lane == 0) mbar_arrive_expect_tx(full, (uint32_t)(2 * cbytes) + (sc_bulk ? 2 * scbytes : 0));
       __syncwarp();
       if (lane_copies)
         bulk_g2s_hint(st + lane_dst, lane_sc ? (const void*)sc_src : (const void*)row_src, lane_sc ? scbytes : (uint32_t)cbytes, full, pol);
-      if (WT != 0 && !sc_bulk) {
+      if (!is16<WT> && !sc_bulk) {
         const int ppr = (cbytes >> bs_shift) >> 1;  // 4-byte pieces per row
         for (int j = lane & 15; j < ppr; j += 16) cp_async4(st + 2 * ROWB + (lane >> 4) * geom<WT>::SC_ROW + j * 4, sc_src + 2 * j);
         cp_async_mbar_arrive_noinc(full);
@@ -286,9 +306,9 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
     auto pair_sources = [&](const int pr, const uint8_t*& row_src, const __half*& sc_src) {
       int mat, row;
       map_row<EPI>(p, 2 * pr + (lane & 1), mat, row);
-      row_src = reinterpret_cast<const uint8_t*>(p.w[mat]) + (size_t)row * rowbytes;
+      row_src = weights_of(mat) + (size_t)row * rowbytes;
       sc_src = nullptr;
-      if (WT) {
+      if (!is16<WT>) {
         int m2, r2;
         map_row<EPI>(p, 2 * pr + (lane >> 4), m2, r2);
         sc_src = p.sc[m2] + (size_t)r2 * (p.K >> bs_shift);
@@ -303,7 +323,7 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
       for (int ci = 0; ci < nchunks; ++ci) {
         const int cbytes = min(ROWB, rowbytes - ci * ROWB);
 #pragma unroll
-        for (int w = 0; w < NW; ++w) issue(w, src_row[w] + (size_t)ci * ROWB, WT ? src_sc[w] + ((ci * CHUNK_K) >> bs_shift) : nullptr, cbytes);
+        for (int w = 0; w < NW; ++w) issue(w, src_row[w] + (size_t)ci * ROWB, !is16<WT> ? src_sc[w] + ((ci * CHUNK_K) >> bs_shift) : nullptr, cbytes);
       }
     }
     // tail round: the pairs left over go to warps 0 .. r_tail-1
@@ -317,10 +337,10 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
         const int cbytes = min(ROWB, rowbytes - ci * ROWB);
 #pragma unroll
         for (int w = 0; w < NW; ++w)
-          if (w < r_tail) issue(w, src_row[w] + (size_t)ci * ROWB, WT ? src_sc[w] + ((ci * CHUNK_K) >> bs_shift) : nullptr, cbytes);
+          if (w < r_tail) issue(w, src_row[w] + (size_t)ci * ROWB, !is16<WT> ? src_sc[w] + ((ci * CHUNK_K) >> bs_shift) : nullptr, cbytes);
       }
     }
-    if (WT != 0) cp_async_wait<0>();
+    if (!is16<WT>) cp_async_wait<0>();
     return;
   }
 
@@ -329,7 +349,7 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
   constexpr int NVEC = 4;  // 16-byte vectors of norm weights per thread kept in registers (covers K <= 4096 with four warps)
   const int vec = p.K >> 3;
   uint4 nw[NVEC];
-  if (p.norm_w != nullptr && npairs > 0) {
+  if (WT != 3 && p.norm_w != nullptr && npairs > 0) {
 #pragma unroll
     for (int j = 0; j < NVEC; ++j) {
       const int i = tid + j * NCONS;
@@ -358,7 +378,7 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
       for (int j = 0; j < NVEC; ++j) {
         const int i = tid + j * NCONS;
         if (i < vec) {
-          xv[j] = __ldcg(reinterpret_cast<const uint4*>(p.x + i * 8));
+          xv[j] = __ldcg(reinterpret_cast<const uint4*>(x_row + i * 8));
           *reinterpret_cast<uint4*>(xs + xoff(i)) = xv[j];
         }
       }
@@ -373,11 +393,11 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
         __syncwarp();
         const int nseg = (p.K + 511) >> 9;
         for (int sg = lane; sg < nseg; sg += 32)
-          bulk_g2s(smem_u32(xs + xoff(sg * 64)), p.x + sg * 512, (uint32_t)min(1024, (p.K - sg * 512) * 2), xbar);
+          bulk_g2s(smem_u32(xs + xoff(sg * 64)), x_row + sg * 512, (uint32_t)min(1024, (p.K - sg * 512) * 2), xbar);
       }
       mbar_wait(xbar, 0, p.err, DEV_ERR_FULL_WAIT);
     }
-    if (p.norm_w != nullptr) {
+    if (WT != 3 && p.norm_w != nullptr) {
       // RMSNorm with the reference's summation order (llama_cu.cu:72-106): 256 strided partial sums,
       // xor trees inside 8 warps, xor tree over the 8 warp sums.  Each of the 128 threads here plays
       // two of the reference's threads (t and t + 128), each warp two of its warps (w and w + 4).
@@ -460,7 +480,7 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
     // u8 kernels (latency-bound): what the epilogue reads from global memory is requested now, one address for the
     // whole warp, so that its latency passes under the row's products instead of after them.  The fp16 kernels run at
     // the memory roofline, where the early loads measured no difference; they fetch in the epilogue.
-    constexpr bool EARLY = WT != 0;
+    constexpr bool EARLY = !is16<WT>;
     const int vrow = 2 * (pr0 + i);
     __half2 prev = __half2half2(__ushort_as_half(0));
     float2 cs = make_float2(1.f, 0.f);
@@ -518,6 +538,15 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
     v1 = warp_sum(v1);
     if (lane == 0) {
       const int pr = pr0 + i;
+      if (WT == 3) {
+        if (EPI == EPI_PLAIN) {
+          if (bt.f32[bi]) *reinterpret_cast<float2*>(reinterpret_cast<float*>(bt.out[bi]) + vrow) = make_float2(v0, v1);
+          else *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(bt.out[bi]) + vrow) = __floats2bfloat162_rn(v0, v1);
+        } else {  // the gate on the binary32 sums
+          reinterpret_cast<__nv_bfloat16*>(p.out)[pr] = __float2bfloat16(v0 / (1.0f + expf(-v0)) * v1);
+        }
+        continue;
+      }
       if (!EARLY) fetch_epilogue_operands();
       if (EPI == EPI_PLAIN) {
         float a0 = v0, a1 = v1;
@@ -577,7 +606,7 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
 }
 
 template <int WT, int EPI, int NW>
-int launch_one(const gemv_params& p, cudaStream_t stream, int pdl, size_t smem, int grid, int sw, int pf_bytes) {
+int launch_one(const gemv_params& p, cudaStream_t stream, int pdl, size_t smem, int grid, int sw, int pf_bytes, const gemv_batch& bt = gemv_batch{}) {
   static bool attr_done[16] = {};
   int dev = 0;
   LCU_CUDA(cudaGetDevice(&dev));
@@ -595,7 +624,7 @@ int launch_one(const gemv_params& p, cudaStream_t stream, int pdl, size_t smem, 
   attr[0].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = pdl ? 1 : 0;
-  LCU_CUDA(cudaLaunchKernelEx(&cfg, gemv1_kernel<WT, EPI, NW>, p, sw, pf_bytes));
+  LCU_CUDA(cudaLaunchKernelEx(&cfg, gemv1_kernel<WT, EPI, NW>, p, sw, pf_bytes, bt));
   return LCU_OK;
 }
 
@@ -686,6 +715,55 @@ int launch_gemv_single_row(const gemv_params& p, int epilogue, cudaStream_t stre
   }
 #undef LCU_GEMV1_CASE
   LCU_REQUIRE(false, "gemv: unknown epilogue %d", epilogue);
+}
+
+int launch_gemv_bf16(const gemv_batch& b, int K, int* err, cudaStream_t stream, int pdl) {
+  LCU_REQUIRE(b.n >= 1 && b.n <= GEMV_MAX_BATCH, "gemv: %d matrices outside 1..%d", b.n, GEMV_MAX_BATCH);
+  LCU_REQUIRE(K > 0 && K % 256 == 0, "gemv: K=%d must be a positive multiple of 256", K);
+  long long total = 0;
+  for (int i = 0; i < b.n; ++i) {
+    LCU_REQUIRE(b.rows[i] > 0 && b.rows[i] % 2 == 0, "gemv: row count %d must be even", b.rows[i]);
+    LCU_REQUIRE((((uintptr_t)b.w[i] | (uintptr_t)b.x[i]) & 15) == 0 && ((uintptr_t)b.out[i] & 7) == 0, "gemv: unaligned operand of matrix %d", i);
+    total += b.rows[i] / 2;
+  }
+  gemv_params p{};
+  p.n_mats = 1;
+  p.rows_per_mat = (int)(2 * total);
+  p.K = K;
+  p.m = 1;
+  p.err = err;
+  gemv1_config c;
+  int rc = configure(p, gemv_sm_count(), c);
+  if (rc) return rc;
+  // CTAs are dealt to the matrices in proportion to their rows, at least one each
+  gemv_batch bt = b;
+  const int spare = c.grid > b.n ? c.grid - b.n : 0;
+  long long seen = 0;
+  for (int i = 0; i < b.n; ++i) {
+    bt.first_cta[i] = i + (int)(spare * seen / total);
+    seen += b.rows[i] / 2;
+  }
+  bt.first_cta[b.n] = b.n + spare;
+  return launch_one<3, EPI_PLAIN, 4>(p, stream, pdl, c.smem, b.n + spare, c.sw, c.pf, bt);
+}
+
+int launch_gemv_bf16_gated(void* out, const void* x, const void* w13, int f, int K, int* err, cudaStream_t stream, int pdl) {
+  LCU_REQUIRE(K > 0 && K % 256 == 0 && f > 0, "gemv: K=%d must be a positive multiple of 256", K);
+  LCU_REQUIRE((((uintptr_t)w13 | (uintptr_t)x) & 15) == 0, "gemv: unaligned operand");
+  gemv_params p{};
+  p.w[0] = w13;
+  p.w[1] = reinterpret_cast<const uint8_t*>(w13) + (size_t)f * K * 2;
+  p.n_mats = 2;
+  p.rows_per_mat = f;
+  p.K = K;
+  p.m = 1;
+  p.x = reinterpret_cast<const __half*>(x);
+  p.out = reinterpret_cast<__half*>(out);
+  p.err = err;
+  gemv1_config c;
+  int rc = configure(p, gemv_sm_count(), c);
+  if (rc) return rc;
+  return launch_one<3, EPI_SILU, 4>(p, stream, pdl, c.smem, c.grid, c.sw, c.pf);
 }
 
 }  // namespace lcu

@@ -51,7 +51,7 @@ __global__ void __cluster_dims__(HC_CLUSTER, 1, 1) __launch_bounds__(HC_THREADS)
   for (int e = tid; e < n_local; e += HC_THREADS) {
     const int i = 256 * (e >> 5) + 32 * (int)rank + (e & 31);
     float v = -CUDART_INF_F;
-    if (i < V) v = __half2float(p.logits[i]) / temp;
+    if (i < V) v = head_logit(p, i) / temp;
     e_buf[e] = v;
     mx = fmaxf(mx, v);
   }
@@ -98,9 +98,10 @@ __global__ void __cluster_dims__(HC_CLUSTER, 1, 1) __launch_bounds__(HC_THREADS)
   for (int e = tid; e < n_local; e += HC_THREADS) {
     const int i = 256 * (e >> 5) + 32 * (int)rank + (e & 31);
     if (i < V) {
-      const __half ph = __float2half(e_buf[e] / sum);
+      const float pr = e_buf[e] / sum;
+      const __half ph = __float2half(pr);
       p.probs[i] = ph;
-      const float pf = __half2float(ph);
+      const float pf = p.logits_f32 ? pr : __half2float(ph);
       if (pf > best || (pf == best && i < best_i)) {
         best = pf;
         best_i = i;

@@ -229,7 +229,7 @@ __global__ void __launch_bounds__(HEAD_THREADS) logits_head_kernel(const head_pa
   pdl_wait();
 
   float mx = -CUDART_INF_F;
-  for (int i = tid; i < V; i += HEAD_THREADS) mx = fmaxf(mx, __half2float(p.logits[i]) / temp);
+  for (int i = tid; i < V; i += HEAD_THREADS) mx = fmaxf(mx, head_logit(p, i) / temp);
   mx = warp_max(mx);
   if (lane == 0) s_red[warp] = mx;
   __syncthreads();
@@ -242,14 +242,14 @@ __global__ void __launch_bounds__(HEAD_THREADS) logits_head_kernel(const head_pa
   mx = s_bcast[0];
 
   if (cache_exp)
-    for (int i = tid; i < V; i += HEAD_THREADS) e_cache[i] = expf(__half2float(p.logits[i]) / temp - mx);
+    for (int i = tid; i < V; i += HEAD_THREADS) e_cache[i] = expf(head_logit(p, i) / temp - mx);
   __syncthreads();
   float sum = 0.f;
   if (tid < 256) {
     if (cache_exp)
       for (int i = tid; i < V; i += 256) sum += e_cache[i];
     else
-      for (int i = tid; i < V; i += 256) sum += expf(__half2float(p.logits[i]) / temp - mx);
+      for (int i = tid; i < V; i += 256) sum += expf(head_logit(p, i) / temp - mx);
     sum = warp_sum(sum);
     if (lane == 0) s_red[warp] = sum;
   }
@@ -266,10 +266,11 @@ __global__ void __launch_bounds__(HEAD_THREADS) logits_head_kernel(const head_pa
   float best = -1.f;
   int best_i = 0x7fffffff;
   for (int i = tid; i < V; i += HEAD_THREADS) {
-    const float e = cache_exp ? e_cache[i] : expf(__half2float(p.logits[i]) / temp - mx);
-    const __half ph = __float2half(e / sum);
+    const float e = cache_exp ? e_cache[i] : expf(head_logit(p, i) / temp - mx);
+    const float pr = e / sum;
+    const __half ph = __float2half(pr);
     p.probs[i] = ph;
-    const float pf = __half2float(ph);
+    const float pf = p.logits_f32 ? pr : __half2float(ph);
     if (pf > best) {  // strided ascending i: keeps the first index of this thread's maximum
       best = pf;
       best_i = i;
@@ -966,6 +967,16 @@ int launch_bump_pos(int* pos, int inc, cudaStream_t stream) {
 }
 int launch_token_to_ids(short* ids, const int* token, cudaStream_t stream) {
   token_to_ids_kernel<<<1, 1, 0, stream>>>(ids, token);
+  LCU_CUDA(cudaGetLastError());
+  return LCU_OK;
+}
+
+__global__ void half_to_f32_kernel(float* out, const __half* in, size_t n) {
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) out[i] = __half2float(in[i]);
+}
+int launch_half_to_f32(float* out, const __half* in, size_t n, cudaStream_t stream) {
+  if (n == 0) return LCU_OK;
+  half_to_f32_kernel<<<(unsigned)std::min<size_t>((n + 255) / 256, 148 * 8), 256, 0, stream>>>(out, in, n);
   LCU_CUDA(cudaGetLastError());
   return LCU_OK;
 }

@@ -40,6 +40,7 @@ int launch_silu_rows(__half* out, const __half* ab, int m, int f, cudaStream_t s
 // *pos += advance; next_ids[0] = token; if log != nullptr, log[*step] = token and ++*step.
 struct head_params {
   const __half* logits;
+  const float* logits_f32;  // instead of `logits`: binary32 logits; the token is then the maximum before the rounding to half
   __half* probs;  // may alias logits
   int n_vocab;
   float temperature;
@@ -51,6 +52,9 @@ struct head_params {
   int* step;
   int log_capacity;
 };
+#ifdef __CUDACC__
+__device__ __forceinline__ float head_logit(const head_params& p, int i) { return p.logits_f32 ? p.logits_f32[i] : __half2float(p.logits[i]); }
+#endif
 int launch_logits_head(const head_params& p, cudaStream_t stream, int pdl);
 // one-block version of the same computation (any vocabulary size; used when the clustered kernel does not fit)
 int launch_logits_head_single(const head_params& p, cudaStream_t stream, int pdl);
@@ -75,6 +79,7 @@ int launch_error_stats(float* stats, float* partial, const __half* a, const __ha
 
 // seeded synthetic data: out[i] = half(scale * z(seed, fnv1a(name), first + i)), z ~ approx N(0,1)
 int launch_synth_fill(__half* out, size_t n, uint64_t seed, uint64_t stream_id, float scale, uint64_t first, cudaStream_t stream);
+int launch_half_to_f32(float* out, const __half* in, size_t n, cudaStream_t stream);
 int launch_fill_half(__half* out, size_t n, float value, cudaStream_t stream);
 uint64_t fnv1a64(const char* s);
 

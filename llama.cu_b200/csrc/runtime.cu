@@ -11,7 +11,7 @@
 //     synchronisation, replayed as one CUDA graph with programmatic dependent launches;
 //   * the position is read from device memory, so the same graph serves every step and greedy
 //     decoding can run chained on the device.
-#include "runtime.cuh"
+#include "context.cuh"
 
 #include <fcntl.h>
 #include <sys/mman.h>
@@ -27,6 +27,7 @@
 #include "attention.cuh"
 #include "gemm_tc.cuh"
 #include "gemv.cuh"
+#include "loader.cuh"
 #include "ops.cuh"
 #include "prefill.cuh"
 
@@ -41,12 +42,6 @@ void set_last_error(const char* fmt, ...) {
   va_end(ap);
 }
 const char* last_error() { return g_err; }
-
-#define LCU_TRY(expr)      \
-  do {                     \
-    int _rc = (expr);      \
-    if (_rc) return _rc;   \
-  } while (0)
 
 // 64 zeroed device words per GPU for the stand-alone operator entry points (word 0: error word of their kernels;
 // word 8: token of lcu_logits_head); allocated at the first use on a device
@@ -88,16 +83,6 @@ std::vector<int> partition::used_gpus() const {
 
 // ------------------------------------------------------------------ model
 namespace {
-constexpr size_t ALIGN = 256;
-struct carve {
-  size_t off = 0;
-  size_t take(size_t bytes) {
-    size_t o = off;
-    off += round_up(bytes, ALIGN);
-    return o;
-  }
-};
-
 struct tensor_slot {  // one named tensor of the weight directory
   std::string name;
   dev_matrix* mat;    // matrix, or
@@ -145,11 +130,14 @@ std::vector<tensor_slot> enumerate(model& m) {
 }
 }  // namespace
 
-model::~model() {
+model_base::~model_base() {
   for (auto& a : arenas) {
     device_guard g(a.first);
     cudaFree(a.second);
   }
+}
+
+model::~model() {
   for (auto& a : shadow_arenas) {
     device_guard g(a.first);
     cudaFree(a.second);
@@ -371,110 +359,6 @@ int load_file_mapped(const std::string& path, void* dst, size_t bytes, size_t fi
   return LCU_OK;
 }
 
-// Staged loader: files are read in pieces into two pinned buffers; while one piece travels to the device
-// (cudaMemcpyAsync on the loader's stream, one copy per piece) the next one is read from the file.  One loader per
-// GPU of the partition; finish() waits for the last copies.
-struct staged_loader {
-  static constexpr size_t PIECE = (size_t)64 << 20;
-  static constexpr int READERS = 8;
-  int device = 0;
-  void* pin[2] = {nullptr, nullptr};
-  cudaEvent_t done[2] = {nullptr, nullptr};
-  bool in_flight[2] = {false, false};
-  cudaStream_t stream = nullptr;
-  int cur = 0;
-
-  int init(int dev) {
-    device = dev;
-    device_guard g(dev);
-    LCU_CUDA(cudaStreamCreateWithFlags(&stream, cudaStreamNonBlocking));
-    for (int i = 0; i < 2; ++i) {
-      LCU_CUDA(cudaMallocHost(&pin[i], PIECE));
-      LCU_CUDA(cudaEventCreateWithFlags(&done[i], cudaEventDisableTiming));
-    }
-    return LCU_OK;
-  }
-  ~staged_loader() {
-    device_guard g(device);
-    if (stream) cudaStreamSynchronize(stream);
-    for (int i = 0; i < 2; ++i) {
-      if (pin[i]) cudaFreeHost(pin[i]);
-      if (done[i]) cudaEventDestroy(done[i]);
-    }
-    if (stream) cudaStreamDestroy(stream);
-  }
-  int copy_file(const std::string& path, void* dst, size_t bytes, size_t file_off, size_t file_bytes) {
-    int fd = open(path.c_str(), O_RDONLY);
-    if (fd < 0) {
-      set_last_error("cannot open %s", path.c_str());
-      return LCU_ERR_IO;
-    }
-    struct stat st;
-    if (fstat(fd, &st) != 0 || (size_t)st.st_size != file_bytes) {
-      close(fd);
-      set_last_error("%s: expected %zu bytes, file has %lld", path.c_str(), file_bytes, (long long)st.st_size);
-      return LCU_ERR_IO;
-    }
-#ifdef POSIX_FADV_SEQUENTIAL
-    posix_fadvise(fd, 0, 0, POSIX_FADV_SEQUENTIAL);
-#endif
-    device_guard g(device);
-    for (size_t off = 0; off < bytes;) {
-      const size_t n = std::min(PIECE, bytes - off);
-      if (in_flight[cur]) {  // the buffer's previous piece must have left it
-        if (cudaEventSynchronize(done[cur]) != cudaSuccess) {
-          close(fd);
-          set_last_error("copy of %s to the device failed", path.c_str());
-          return LCU_ERR_CUDA;
-        }
-        in_flight[cur] = false;
-      }
-      // the piece is read by several threads at once (a single reader copies out of the page cache at a fraction of
-      // what the host-to-device link takes)
-      const int n_readers = n >= ((size_t)4 << 20) ? READERS : 1;
-      const size_t share = (n / n_readers + 4095) & ~(size_t)4095;
-      std::atomic<int> failed{0};
-      auto read_range = [&](size_t lo, size_t hi) {
-        while (lo < hi) {
-          const ssize_t r = pread(fd, (char*)pin[cur] + lo, hi - lo, (off_t)(file_off + off + lo));
-          if (r <= 0) {
-            failed = 1;
-            return;
-          }
-          lo += (size_t)r;
-        }
-      };
-      std::vector<std::thread> readers;
-      for (int t = 1; t < n_readers; ++t) readers.emplace_back(read_range, std::min(n, t * share), std::min(n, (t + 1) * share));
-      read_range(0, std::min(n, share));
-      for (auto& th : readers) th.join();
-      if (failed) {
-        close(fd);
-        set_last_error("short read from %s", path.c_str());
-        return LCU_ERR_IO;
-      }
-      cudaError_t e = cudaMemcpyAsync((char*)dst + off, pin[cur], n, cudaMemcpyHostToDevice, stream);
-      if (e == cudaSuccess) e = cudaEventRecord(done[cur], stream);
-      if (e != cudaSuccess) {
-        close(fd);
-        set_last_error("copy of %s to the device failed: %s", path.c_str(), cudaGetErrorString(e));
-        return LCU_ERR_CUDA;
-      }
-      in_flight[cur] = true;
-      cur ^= 1;
-      off += n;
-    }
-    close(fd);
-    return LCU_OK;
-  }
-  int finish() {
-    device_guard g(device);
-    LCU_CUDA(cudaStreamSynchronize(stream));
-    in_flight[0] = in_flight[1] = false;
-    return LCU_OK;
-  }
-};
-
 int g_loader_staged = 1;
 }  // namespace
 
@@ -594,51 +478,11 @@ scratch_layout scratch_layout_of(const model_params& p, uint32_t ffn, int contex
 size_t context_scratch_bytes(const model_params& p, int context_len) { return scratch_layout_of(p, ffn_dim_of(p), context_len).total; }
 size_t context_kv_bytes_per_layer(const model_params& p, int context_len) { return 2 * round_up((size_t)context_len * p.dim * 2, ALIGN); }
 
-struct gpu_state {
-  int device = 0;
-  cudaStream_t stream = nullptr;
-  cudaEvent_t ev = nullptr;
-  void* arena = nullptr;
-  size_t arena_bytes = 0;
-  __half *x = nullptr, *norm = nullptr, *q = nullptr, *kn = nullptr, *vn = nullptr, *att = nullptr;
-  __half *h1 = nullptr, *h3 = nullptr, *hs = nullptr;
-  __half* scores = nullptr;  // prompt attention on tcgen05: [heads][context_len][round_up(context_len, 128)] scores / probabilities
-  __half* deq = nullptr;  // u8 models: the dequantized matrix (or stack of matrices) of the prompt GEMM in flight
-  size_t deq_halves = 0;
-  // prompt path of u8 models: matrices are expanded to fp16 one job ahead on a side stream, into two alternating buffers
-  __half* deq_buf[2] = {nullptr, nullptr};
-  cudaStream_t side = nullptr;
-  cudaEvent_t deq_done[2] = {nullptr, nullptr}, gemm_done[2] = {nullptr, nullptr};
-  long deq_issued = 0, deq_used = 0;  // jobs expanded / consumed so far (job j lives in buffer j % 2)
-  float2* rope = nullptr;
-  int* state = nullptr;  // [0] position, [1] step counter, [2] last token, [3] error word
-};
-
-struct context_impl {
+struct llama_context_impl : context_impl {
   model* m = nullptr;
-  context_options opt;
-  int start_pos = 0;
-  std::vector<gpu_state> gpus;           // in order of first use
   std::vector<int> layer_slot;           // layer -> index into gpus
   std::vector<__half*> k_cache, v_cache; // per layer, on the layer's GPU
-  std::vector<void*> kv_arenas;          // one per GPU
-  size_t kv_bytes = 0;
-  short* ids = nullptr;                  // token ids on the embedding GPU [context_len]
   __half* logits = nullptr;              // on the output GPU
-  __half* probs = nullptr;
-  short* log = nullptr;                  // generated tokens of a chained run [context_len]
-  int* h_stage = nullptr;                // pinned: [0] position, [1] zero, [2] token read-back
-  short* h_ids = nullptr;                // pinned token staging [context_len]
-  cudaEvent_t t0 = nullptr, t1 = nullptr;
-  // two captured decode steps: [0] for positions whose attention slices stay within the register-path kernel's
-  // 64 rows per CTA, [1] for longer contexts (streaming attention kernel); the host knows the position of every step
-  cudaGraphExec_t graph[2] = {nullptr, nullptr};
-  bool graph_failed = false;
-  bool warmed_variant[2] = {false, false};
-  int last_row = 0;                      // row of x that holds the last token's residual stream
-
-  gpu_state& first() { return gpus.front(); }
-  gpu_state& last() { return gpus.back(); }
 
   gemv_params params_base(gpu_state& g, int K);
   gemv_params params_qkv(int l);
@@ -647,11 +491,17 @@ struct context_impl {
   gemv_params params_w2(int l);
   gemv_params params_out(int row);
   int enqueue_hop(int from, int to, int m_rows);
-  int enqueue_decode_step(int long_ctx);
-  int enqueue_prefill(int m_rows);
-  int build_graph(int variant);
-  int run_decode_step(int n_keys);
-  int stage_inputs(const short* tokens, int n);
+  int enqueue_decode_step(int long_ctx) override;
+  int enqueue_prefill(int m_rows, const pass_request& rq) override;
+  // two captured decode steps: [0] for positions whose attention slices stay within the register-path kernel's
+  // 64 rows per CTA, [1] for longer contexts (streaming attention kernel); the host knows the position of every step
+  int decode_variant(int n_keys) const override { return n_keys > 64 * opt.attn_cluster ? 1 : 0; }
+  int kernels_per_step() const override { return 1 + 5 * (int)m->params.n_layers + 2 + (opt.sampling ? 1 : 0); }
+  bool rows_only() const override { return matmul_type_ref() == 1; }  // (the pedantic matmul type has no fused decode kernels)
+  int read_step_logits(float* out_host) override;
+  int read_hidden(__half* out_host) override;
+  int rollover(int keep) override;
+  int bench_kernel(int which, int reps, float* ms_per_launch, uint64_t* bytes_per_launch) override;
 };
 
 context::~context() {
@@ -678,18 +528,28 @@ context::~context() {
   if (c.h_ids) cudaFreeHost(c.h_ids);
 }
 
-int context::create(std::unique_ptr<context>& out, model* m, const context_options& opt) {
+int context::create(std::unique_ptr<context>& out, model_base* m, const context_options& opt) {
   LCU_REQUIRE(m != nullptr, "context: null model");
   LCU_REQUIRE(opt.context_len >= 1 && opt.context_len <= 32768, "context: context length %d outside 1..32768", opt.context_len);
   LCU_REQUIRE(opt.temperature > 0.f, "context: temperature must be positive");
+  auto ctx = std::make_unique<context>();
+  LCU_TRY(m->new_context(ctx->impl, opt));
+  out = std::move(ctx);
+  return LCU_OK;
+}
+
+int model::new_context(std::unique_ptr<context_impl>& out, const context_options& opt) {
+  model* m = this;
   const model_params& p = m->params;
   const int hd = p.dim / p.n_heads;
   LCU_REQUIRE(hd == 64 || hd == 128, "context: head_dim %d not supported (64 or 128)", hd);
-  auto ctx = std::make_unique<context>();
-  ctx->impl = std::make_unique<context_impl>();
-  context_impl& c = *ctx->impl;
+  auto holder = std::make_unique<context>();  // (its destructor releases what was allocated if a step below fails)
+  holder->impl = std::make_unique<llama_context_impl>();
+  llama_context_impl& c = static_cast<llama_context_impl&>(*holder->impl);
   c.m = m;
   c.opt = opt;
+  c.n_vocab = p.n_vocab;
+  c.width = p.dim;
   const size_t ctxl = opt.context_len, d = p.dim;
   const std::vector<int> used = m->part.used_gpus();
   c.gpus.resize(used.size());
@@ -777,18 +637,21 @@ int context::create(std::unique_ptr<context>& out, model* m, const context_optio
       }
     LCU_CUDA(cudaStreamSynchronize(g.stream));
   }
-  {
-    device_guard dg(c.first().device);
-    LCU_CUDA(cudaMallocHost(&c.h_stage, 64));
-    LCU_CUDA(cudaMallocHost(&c.h_ids, ctxl * 2));
-    memset(c.h_stage, 0, 64);
-    LCU_CUDA(cudaEventCreate(&c.t0));
-    LCU_CUDA(cudaEventCreate(&c.t1));
-  }
+  LCU_TRY(c.open_streams(opt.context_len));
   // u8 models: the fp16 shadow for prompts is set up here, next to the context's own arenas, so that next_token never
   // allocates (a stale shadow is refreshed in place by the next long prompt)
   if (p.q_type && c.opt.context_len >= 2) m->shadow_ready(true);
-  out = std::move(ctx);
+  out = std::move(holder->impl);
+  return LCU_OK;
+}
+
+int context_impl::open_streams(int context_len) {
+  device_guard dg(first().device);
+  LCU_CUDA(cudaMallocHost(&h_stage, 64));
+  LCU_CUDA(cudaMallocHost(&h_ids, (size_t)context_len * 2));
+  memset(h_stage, 0, 64);
+  LCU_CUDA(cudaEventCreate(&t0));
+  LCU_CUDA(cudaEventCreate(&t1));
   return LCU_OK;
 }
 
@@ -801,7 +664,7 @@ size_t context::memory_usage() const {
 }
 int context::tokens_left() const { return impl->opt.context_len - impl->start_pos; }
 int context::position() const { return impl->start_pos; }
-int context::kernels_per_step() const { return 1 + 5 * (int)impl->m->params.n_layers + 2 + (impl->opt.sampling ? 1 : 0); }
+int context::kernels_per_step() const { return impl->kernels_per_step(); }
 
 int context::set_sampling(int mode, uint64_t seed) {
   LCU_REQUIRE(mode == 0 || mode == 1, "set_sampling: mode %d (0 = greedy, 1 = multinomial)", mode);
@@ -818,21 +681,22 @@ int context::set_sampling(int mode, uint64_t seed) {
   return LCU_OK;
 }
 
-int context::rollover(int keep) {
-  context_impl& c = *impl;
-  LCU_REQUIRE(keep >= 1 && keep < c.start_pos, "rollover: keep %d of %d cached positions", keep, c.start_pos);
-  const model_params& p = c.m->params;
-  const int first = c.start_pos - keep;
+int context::rollover(int keep) { return impl->rollover(keep); }
+
+int llama_context_impl::rollover(int keep) {
+  LCU_REQUIRE(keep >= 1 && keep < start_pos, "rollover: keep %d of %d cached positions", keep, start_pos);
+  const model_params& p = m->params;
+  const int first_row = start_pos - keep;
   for (uint32_t l = 0; l < p.n_layers; ++l) {
-    gpu_state& g = c.gpus[c.layer_slot[l]];
+    gpu_state& g = gpus[layer_slot[l]];
     device_guard dg(g.device);
-    LCU_TRY(launch_rollover(c.k_cache[l], c.v_cache[l], p.n_heads, c.opt.context_len, p.dim / p.n_heads, first, keep, 10000.0f, g.stream));
+    LCU_TRY(launch_rollover(k_cache[l], v_cache[l], p.n_heads, opt.context_len, p.dim / p.n_heads, first_row, keep, 10000.0f, g.stream));
   }
-  for (auto& g : c.gpus) {
+  for (auto& g : gpus) {
     device_guard dg(g.device);
     LCU_CUDA(cudaStreamSynchronize(g.stream));
   }
-  c.start_pos = keep;
+  start_pos = keep;
   return LCU_OK;
 }
 
@@ -874,7 +738,7 @@ static int finish_step(context& ctx, const char* who) {
 
 // residual stream hand-off between pipeline stages: m_rows x dim halves over NVLink
 // (the reference copies the whole context-length buffer, llama_cu.cu:1110-1114)
-int context_impl::enqueue_hop(int from, int to, int m_rows) {
+int llama_context_impl::enqueue_hop(int from, int to, int m_rows) {
   gpu_state& a = gpus[from];
   gpu_state& b = gpus[to];
   LCU_CUDA(cudaMemcpyPeerAsync(b.x, b.device, a.x, a.device, (size_t)m_rows * m->params.dim * 2, a.stream));
@@ -885,7 +749,7 @@ int context_impl::enqueue_hop(int from, int to, int m_rows) {
 
 
 // ---- kernel arguments of the decode step
-gemv_params context_impl::params_base(gpu_state& g, int K) {
+gemv_params llama_context_impl::params_base(gpu_state& g, int K) {
   gemv_params a{};
   a.K = K;
   a.bs = m->params.q_type ? m->params.quantization_block_size : 0;
@@ -896,7 +760,7 @@ gemv_params context_impl::params_base(gpu_state& g, int K) {
   a.pos = g.state;
   return a;
 }
-gemv_params context_impl::params_qkv(int l) {
+gemv_params llama_context_impl::params_qkv(int l) {
   gpu_state& g = gpus[layer_slot[l]];
   const layer_weights& L = m->layers[l];
   const int d = m->params.dim;
@@ -915,7 +779,7 @@ gemv_params context_impl::params_qkv(int l) {
   a.head_dim = d / m->params.n_heads;
   return a;
 }
-gemv_params context_impl::params_wo(int l) {
+gemv_params llama_context_impl::params_wo(int l) {
   gpu_state& g = gpus[layer_slot[l]];
   const layer_weights& L = m->layers[l];
   const int d = m->params.dim;
@@ -924,7 +788,7 @@ gemv_params context_impl::params_wo(int l) {
   a.x = g.att; a.out = g.x; a.ldo = d; a.beta = 1.0f;
   return a;
 }
-gemv_params context_impl::params_w13(int l) {
+gemv_params llama_context_impl::params_w13(int l) {
   gpu_state& g = gpus[layer_slot[l]];
   const layer_weights& L = m->layers[l];
   const int d = m->params.dim, f = m->ffn;
@@ -934,7 +798,7 @@ gemv_params context_impl::params_w13(int l) {
   a.x = g.x; a.norm_w = L.ffn_norm; a.out = g.hs; a.ldo = f;
   return a;
 }
-gemv_params context_impl::params_w2(int l) {
+gemv_params llama_context_impl::params_w2(int l) {
   gpu_state& g = gpus[layer_slot[l]];
   const layer_weights& L = m->layers[l];
   const int d = m->params.dim, f = m->ffn;
@@ -945,7 +809,7 @@ gemv_params context_impl::params_w2(int l) {
   if (l + 1 < (int)m->params.n_layers && layer_slot[l + 1] != layer_slot[l]) a.out_peer = gpus[layer_slot[l + 1]].x;
   return a;
 }
-gemv_params context_impl::params_out(int row) {
+gemv_params llama_context_impl::params_out(int row) {
   gpu_state& g = last();
   const int d = m->params.dim;
   gemv_params a = params_base(g, d);
@@ -954,7 +818,7 @@ gemv_params context_impl::params_out(int row) {
   return a;
 }
 
-int context_impl::enqueue_decode_step(int long_ctx) {
+int llama_context_impl::enqueue_decode_step(int long_ctx) {
   const model_params& p = m->params;
   const int d = p.dim, hd = d / p.n_heads, bs = p.q_type ? p.quantization_block_size : 0;
   const int pdl = opt.use_pdl;
@@ -1018,7 +882,8 @@ int context_impl::enqueue_decode_step(int long_ctx) {
   return LCU_OK;
 }
 
-int context_impl::enqueue_prefill(int m_rows) {
+int llama_context_impl::enqueue_prefill(int m_rows, const pass_request& rq) {
+  LCU_REQUIRE(rq.n_want == 0 || (rq.n_want == 1 && rq.want[0] == m_rows - 1), "step: this model gives logits for the last token of a step only");
   const model_params& p = m->params;
   const int d = p.dim, hd = d / p.n_heads, f = m->ffn, bs = p.q_type ? p.quantization_block_size : 0;
   // u8 weights, prompts long enough for the tcgen05 GEMM: every matrix (or stack of matrices) is expanded to fp16 - the
@@ -1179,6 +1044,19 @@ int context_impl::enqueue_prefill(int m_rows) {
       LCU_CUDA(cudaStreamWaitEvent(first().stream, g.ev, 0));
     }
   }
+  if (rq.n_want) {
+    device_guard dg(last().device);
+    LCU_CUDA(cudaStreamSynchronize(last().stream));
+    LCU_TRY(read_step_logits(rq.logits_out));
+  }
+  return LCU_OK;
+}
+
+int llama_context_impl::read_step_logits(float* out_host) {
+  device_guard dg(last().device);
+  std::vector<__half> h(n_vocab);
+  LCU_CUDA(cudaMemcpy(h.data(), logits, (size_t)n_vocab * 2, cudaMemcpyDeviceToHost));
+  for (int i = 0; i < n_vocab; ++i) out_host[i] = __half2float(h[i]);
   return LCU_OK;
 }
 
@@ -1209,7 +1087,7 @@ int context_impl::build_graph(int variant) {
 }
 
 int context_impl::run_decode_step(int n_keys) {
-  const int variant = n_keys > 64 * opt.attn_cluster ? 1 : 0;
+  const int variant = decode_variant(n_keys);
   if (!warmed_variant[variant]) {  // first use of a variant runs un-captured (function attributes, tensor maps, ...)
     warmed_variant[variant] = true;
     return enqueue_decode_step(variant);
@@ -1256,25 +1134,38 @@ int context_impl::stage_inputs(const short* tokens, int n) {
   return LCU_OK;
 }
 
-int context::next_token(const short* tokens, int n, int* token_out) {
+int context::next_token(const short* tokens, int n, int* token_out) { return step(tokens, n, nullptr, 0, nullptr, token_out); }
+
+int context::step(const short* tokens, int n, const int* want, int n_want, float* logits_out, int* token_out) {
   context_impl& c = *impl;
   LCU_REQUIRE(n >= 1, "next_token: no tokens given");
   LCU_REQUIRE(n + c.start_pos <= c.opt.context_len, "next_token: %d new tokens at position %d exceed the context length %d", n,
               c.start_pos, c.opt.context_len);
   for (int i = 0; i < n; ++i)
-    LCU_REQUIRE(tokens[i] >= 0 && (uint32_t)tokens[i] < c.m->params.n_vocab, "next_token: token id %d outside the vocabulary", tokens[i]);
+    LCU_REQUIRE(tokens[i] >= 0 && tokens[i] < c.n_vocab, "next_token: token id %d outside the vocabulary", tokens[i]);
+  for (int i = 0; i < n_want; ++i) LCU_REQUIRE(want[i] >= 0 && want[i] < n, "step: place %d outside the %d tokens", want[i], n);
+  LCU_REQUIRE(n_want == 0 || logits_out != nullptr, "step: no memory for the logits");
   LCU_TRY(c.stage_inputs(tokens, n));
-  if (n == 1 && matmul_type_ref() != 1)  // (the pedantic matmul type has no fused decode kernels: it takes the operator sequence below)
+  const bool single = n == 1 && !c.rows_only();
+  if (single) {
     LCU_TRY(c.run_decode_step(c.start_pos + 1));
-  else
-    LCU_TRY(c.enqueue_prefill(n));
+  } else {
+    pass_request rq;
+    rq.want = want;
+    rq.n_want = n_want;
+    rq.logits_out = logits_out;
+    rq.token = token_out != nullptr;
+    LCU_TRY(c.enqueue_prefill(n, rq));
+  }
   c.last_row = n == 1 ? 0 : n - 1;
   device_guard dg(c.first().device);
   LCU_CUDA(cudaMemcpyAsync(c.h_stage + 2, c.last().state + 2, 8, cudaMemcpyDeviceToHost, c.first().stream));
   LCU_CUDA(cudaStreamSynchronize(c.first().stream));
   LCU_TRY(finish_step(*this, "next_token"));
   c.start_pos += n;
-  *token_out = c.h_stage[2];
+  if (single)
+    for (int i = 0; i < n_want; ++i) LCU_TRY(c.read_step_logits(logits_out + (size_t)i * c.n_vocab));
+  if (token_out) *token_out = c.h_stage[2];
   return LCU_OK;
 }
 
@@ -1282,8 +1173,8 @@ int context::decode_chained(short first_token, int n_steps, short* tokens_out, f
   context_impl& c = *impl;
   LCU_REQUIRE(n_steps >= 1 && n_steps + c.start_pos <= c.opt.context_len, "decode_chained: %d steps at position %d exceed the context length %d",
               n_steps, c.start_pos, c.opt.context_len);
-  LCU_REQUIRE(first_token >= 0 && (uint32_t)first_token < c.m->params.n_vocab, "decode_chained: token id %d outside the vocabulary", first_token);
-  LCU_REQUIRE(matmul_type_ref() != 1, "decode_chained: matmul_type 1 runs host-driven steps only (lcu_context_next_token)");
+  LCU_REQUIRE(first_token >= 0 && first_token < c.n_vocab, "decode_chained: token id %d outside the vocabulary", first_token);
+  LCU_REQUIRE(!c.rows_only(), "decode_chained: matmul_type 1 runs host-driven steps only (lcu_context_next_token)");
   LCU_TRY(c.stage_inputs(&first_token, 1));
   device_guard dg(c.first().device);
   LCU_CUDA(cudaEventRecord(c.t0, c.first().stream));
@@ -1303,21 +1194,26 @@ int context::decode_chained(short first_token, int n_steps, short* tokens_out, f
 int context::read_probs(__half* out_host) {
   context_impl& c = *impl;
   device_guard dg(c.last().device);
-  LCU_CUDA(cudaMemcpy(out_host, c.probs, (size_t)c.m->params.n_vocab * 2, cudaMemcpyDeviceToHost));
+  LCU_CUDA(cudaMemcpy(out_host, c.probs, (size_t)c.n_vocab * 2, cudaMemcpyDeviceToHost));
   return LCU_OK;
 }
 
-int context::read_hidden(__half* out_host) {
-  context_impl& c = *impl;
-  device_guard dg(c.last().device);
+int context::read_hidden(__half* out_host) { return impl->read_hidden(out_host); }
+
+int llama_context_impl::read_hidden(__half* out_host) {
+  device_guard dg(last().device);
   // decode leaves the token's row at x[0]; a prefill of n rows leaves it at x[n-1] - the caller
   // reads right after next_token, so the row index is kept
-  LCU_CUDA(cudaMemcpy(out_host, c.last().x + (size_t)c.last_row * c.m->params.dim, (size_t)c.m->params.dim * 2, cudaMemcpyDeviceToHost));
+  LCU_CUDA(cudaMemcpy(out_host, last().x + (size_t)last_row * width, (size_t)width * 2, cudaMemcpyDeviceToHost));
   return LCU_OK;
 }
 
 int context::bench_kernel(int which, int reps, float* ms_per_launch, uint64_t* bytes_per_launch) {
-  context_impl& c = *impl;
+  return impl->bench_kernel(which, reps, ms_per_launch, bytes_per_launch);
+}
+
+int llama_context_impl::bench_kernel(int which, int reps, float* ms_per_launch, uint64_t* bytes_per_launch) {
+  llama_context_impl& c = *this;
   LCU_REQUIRE(which >= 0 && which <= 4 && reps >= 1, "bench_kernel: bad arguments");
   // layers of one pipeline stage in rotation: the first stage, or the last one for the output matrix
   const int stage = which == 4 ? (int)c.gpus.size() - 1 : 0;

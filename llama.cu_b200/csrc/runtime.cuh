@@ -74,15 +74,31 @@ struct layer_weights {
   __half* ffn_norm = nullptr;
 };
 
-struct model {
+struct context_impl;  // context.cuh
+struct context_options;
+
+// What every model family shares: weights in per-GPU arenas behind one handle, and the contexts made from it.
+struct model_base {
+  std::vector<std::pair<int, void*>> arenas;  // (device, base) one allocation per GPU
+  size_t weight_bytes_total = 0;
+  virtual ~model_base();
+  virtual const char* family() const = 0;
+  virtual int vocab() const = 0;
+  virtual int width() const = 0;
+  virtual int n_layers() const = 0;
+  // fills every tensor with seeded synthetic data
+  virtual int fill_synthetic(uint64_t seed, float scale) = 0;
+  virtual int new_context(std::unique_ptr<context_impl>& out, const context_options& opt) = 0;
+};
+
+// the LLaMA family
+struct model : model_base {
   model_params params{};
   uint32_t ffn = 0;
   partition part;
   dev_matrix tok_embeddings, output;
   __half* norm = nullptr;
   std::vector<layer_weights> layers;
-  std::vector<std::pair<int, void*>> arenas;  // (device, base) one allocation per GPU
-  size_t weight_bytes_total = 0;
   // tensor-parallel shard: rows [tp_rank, tp_rank + 1) * rows / tp_size of every layer matrix and of the output matrix
   // (whole heads of wq / wk / wv); norm vectors and the embedding table are whole.  tp_size 1 = the whole model.
   int tp_rank = 0, tp_size = 1;
@@ -104,14 +120,19 @@ struct model {
   bool shadow_ready(bool may_allocate);
   void shadow_touch();   // a tensor may have been written
 
-  ~model();
+  ~model() override;
+  const char* family() const override { return "llama"; }
+  int vocab() const override { return (int)params.n_vocab; }
+  int width() const override { return (int)params.dim; }
+  int n_layers() const override { return (int)params.n_layers; }
+  int new_context(std::unique_ptr<context_impl>& out, const context_options& opt) override;
   // allocates all tensors (uninitialised) according to params and the partition
   static int create(std::unique_ptr<model>& out, const model_params& p, const partition& part, int tp_rank = 0, int tp_size = 1);
   // reads a weight directory in the reference's layout (llama_cu.cu:929-984)
   int load_dir(const std::string& dir);
   // fills every tensor with seeded synthetic data (matrices ~ scale * z, norm weights 1.0); a
   // quantized model is generated in fp16 tensor by tensor and quantized on the device
-  int fill_synthetic(uint64_t seed, float scale);
+  int fill_synthetic(uint64_t seed, float scale) override;
   // looks a tensor up by its file stem ("layers.3.attention.wq", "norm", ...): which 0 = values, 1 = scales
   int find_tensor(const std::string& name, int which, void** ptr, size_t* bytes, int* device);
   // writes params and every tensor as a weight directory in the reference's layout
@@ -147,17 +168,18 @@ struct context_options {
   uint64_t sample_seed = 0;
 };
 
-struct context_impl;  // defined in runtime.cu
-
 struct context {
   ~context();
-  static int create(std::unique_ptr<context>& out, model* m, const context_options& opt);
+  static int create(std::unique_ptr<context>& out, model_base* m, const context_options& opt);
   void clear_tokens();
   size_t memory_usage() const;
   int tokens_left() const;
   int position() const;
   // feeds n new tokens (prefill when n > 1), returns the greedy next token in *token_out
   int next_token(const short* tokens, int n, int* token_out);
+  // the same step with binary32 logits of the tokens at `want` (places among the n tokens) copied to logits_out
+  // [n_want][n_vocab]; token_out may be null (no token is picked after a multi-row pass then)
+  int step(const short* tokens, int n, const int* want, int n_want, float* logits_out, int* token_out);
   // device-chained greedy decode: n_steps single-token steps starting from first_token, each
   // step's argmax feeding the next without a host round trip.  Returns the tokens and the device
   // time of the whole loop (CUDA events on the launching stream).

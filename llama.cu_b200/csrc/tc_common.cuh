@@ -2,10 +2,34 @@
 // tcgen05 fences / commit / MMA / tensor-memory loads, shared-memory matrix descriptors.
 #pragma once
 #include <cuda.h>
+#include <cuda_bf16.h>
 
 #include "common.cuh"
 
 namespace lcu {
+
+// 16-bit operand formats of the tcgen05 kind::f16 products: conversions, and the operand-format bits of the instruction
+// descriptor (A at bit 7, B at bit 10; both operands always have the same format)
+template <typename T>
+struct tc_elem;
+template <>
+struct tc_elem<__half> {
+  static constexpr uint32_t IDESC_FORMAT = 0;
+  __device__ static __forceinline__ uint32_t pack(float a, float b) {
+    const __half2 h = __floats2half2_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&h);
+  }
+  __device__ static __forceinline__ float2 unpack(uint32_t w) { return __half22float2(*reinterpret_cast<const __half2*>(&w)); }
+};
+template <>
+struct tc_elem<__nv_bfloat16> {
+  static constexpr uint32_t IDESC_FORMAT = (1u << 7) | (1u << 10);
+  __device__ static __forceinline__ uint32_t pack(float a, float b) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&h);
+  }
+  __device__ static __forceinline__ float2 unpack(uint32_t w) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w)); }
+};
 
 __device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
   asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst),
