@@ -572,6 +572,78 @@ def tensor_parallel_leg(lcu, n_gpus, K, W):
             "exchange": "peer stores from the GEMV epilogues over NVLink + flag words with bounded waits; 4 exchanges per layer (16-44 KB rows)"}
 
 
+# Block models at the sizes of real layers beside the LLaMA family at equal width, feed-forward and layer count: half of the
+# layers window-and-blocks attention with retention (grouped keys, stacked projection of about 3 x width rows), half wkv.
+BLOCK_SIZES = {
+    "1024": dict(width=1024, ff=2816, layers=8, heads=8, n_heads_llama=8),
+    "2048": dict(width=2048, ff=5632, layers=8, heads=16, n_heads_llama=16),
+    "4096": dict(width=4096, ff=11008, layers=8, heads=32, n_heads_llama=32),
+}
+
+
+def block_config(size, vocab=32000, window=1024, pool=16):
+    z = BLOCK_SIZES[size]
+    h = z["heads"] // 2
+    parallel = {"type": "parallel", "mlp": {"kind": "dense", "ff": z["ff"]},
+                "mixer": {"left": {"heads": h, "kv_heads": max(1, h // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                   "mask": {"size": window, "pool": pool}}, "left_scale": 0.7,
+                          "right": {"heads": h, "dim": 128, "vdim": 128, "decay": [1 - 2.0 ** (-5 - 7 * i / h) for i in range(h)],
+                                    "rot": {"base": 10000.0, "dims": 128}}, "right_scale": 0.7}}
+    wkv = {"type": "wkv", "mlp": {"kind": "dense", "ff": z["ff"]}, "mixer": {"heads": z["width"] // 64, "dim": 64}}
+    return {"architecture": "Filulix", "vocab": vocab, "width": z["width"], "streams": 4, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 4093, "mul_cur": 31, "mul_prev": 1009}},
+            "layers": [parallel if i % 2 == 0 else wkv for i in range(z["layers"])], "loop": None}
+
+
+def block_leg(lcu, size, K, W, profile=None):
+    """Decode and prompt throughput of a block model and of a LLaMA-shaped fp16 model of the same width, feed-forward, layer
+    count and vocabulary, random weights, batch 1: decode as `K` device-chained greedy steps between CUDA events after a
+    prompt of 128 and of 1900 tokens, prompts of 512 and 2000 tokens through next_token (host clock, median of 5)."""
+    z = BLOCK_SIZES[size]
+    rng = __import__("numpy").random.default_rng(SEED)
+    out = {"size": size, "layers": z["layers"], "width": z["width"], "ff": z["ff"], "data": "synthetic", "steps": K}
+    clk = ClockSampler(0)
+    clk.start()
+    for name in ("filulix", "llama"):
+        if name == "filulix":
+            model = lcu.Model.from_config(block_config(size), seed=SEED, scale=SCALE)
+        else:
+            model = lcu.Model.synthetic(dim=z["width"], n_heads=z["n_heads_llama"], n_layers=z["layers"], n_vocab=32000, seed=SEED, scale=SCALE,
+                                        multiple_of=256)
+        ctx = lcu.Context(model, context_len=4096, temperature=TEMPERATURE)
+        rec = {"weight_bytes": model.weight_bytes()}
+        for n in (512, 2000):
+            toks = rng.integers(3, 32000, n)
+            times = []
+            for i in range(2 + 5):
+                ctx.clear_tokens()
+                if profile == "prefill" and i == 2 and n == 2000:
+                    lcu.check(lcu.lib.lcu_profiler_start())
+                t0 = time.perf_counter()
+                ctx.next_token(toks)
+                times.append(time.perf_counter() - t0)
+                if profile == "prefill" and i == 2 and n == 2000:
+                    lcu.check(lcu.lib.lcu_profiler_stop())
+            ms = sorted(times[2:])[2] * 1e3
+            rec[f"prompt_{n}"] = {"ms": round(ms, 3), "tok_s": round(n / ms * 1e3)}
+        for n in (128, 1900):
+            ctx.clear_tokens()
+            t = ctx.next_token(rng.integers(3, 32000, n))
+            warm, _ = ctx.decode_chained(t, W)
+            if profile == "decode" and n == 1900:
+                lcu.check(lcu.lib.lcu_profiler_start())
+            _, ms = ctx.decode_chained(int(warm[-1]), K)
+            if profile == "decode" and n == 1900:
+                lcu.check(lcu.lib.lcu_profiler_stop())
+            rec[f"decode_at_{n}"] = {"us_per_step": round(ms / K * 1e3, 2), "tok_s": round(K / ms * 1e3, 1)}
+        rec["kernels_per_step"] = ctx.kernels_per_step()
+        out[name] = rec
+        ctx.close()
+        model.close()
+    out["clocks"] = clk.stop()
+    return out
+
+
 def run_ours(args):
     world, rank, local, dist = dist_setup()
     lcu = load_package()
@@ -820,6 +892,8 @@ def main():
     ap.add_argument("--prefill-len", type=int, default=PREFILL_LEN, help="prompt length of the prefill sample (512; from 768 rows the tcgen05 attention path runs)")
     ap.add_argument("--pipeline", type=int, default=1, help="single process: split the layers evenly over this many GPUs")
     ap.add_argument("--tp", type=int, default=0, help="single process: only the tensor-parallel leg (65B-shaped u8 model) over this many GPUs")
+    ap.add_argument("--blocks", nargs="+", default=None, choices=sorted(BLOCK_SIZES), metavar="WIDTH",
+                    help="only the block-model leg: Filulix beside a LLaMA-shaped model at these widths (1024, 2048, 4096)")
     ap.add_argument("--profile", nargs="?", const="decode", default=None, choices=["decode", "prefill"],
                     help="cudaProfilerStart/Stop around the device-chained timed region (decode) or around the prompt pass and GEMM (prefill)")
     args = ap.parse_args()
@@ -828,7 +902,10 @@ def main():
     sys.stdout.flush()
     _RESULT_FD = os.dup(1)
     os.dup2(2, 1)
-    if args.tp > 1:
+    if args.blocks:
+        lcu = load_package()
+        emit({"blocks": [block_leg(lcu, size, args.steps, args.warmup, args.profile) for size in args.blocks]})
+    elif args.tp > 1:
         lcu = load_package()
         emit({"tensor_parallel": tensor_parallel_leg(lcu, args.tp, args.steps, args.warmup)})
     elif args.impl == "reference":

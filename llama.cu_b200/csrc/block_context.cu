@@ -38,7 +38,7 @@ struct block_context : context_impl {
   std::vector<run_cache<T>> runs;
   std::vector<std::pair<std::pair<int, double>, float2*>> rotations;  // (dims, base) -> table
   // activations [rows_cap]
-  float *xs = nullptr, *y = nullptr, *raw = nullptr, *decays = nullptr, *low = nullptr, *hidden = nullptr, *logits = nullptr;
+  float *xs = nullptr, *y = nullptr, *raw = nullptr, *packed = nullptr, *packed_v = nullptr, *low = nullptr, *hidden = nullptr, *logits = nullptr;
   T *h = nullptr, *mix = nullptr, *proj = nullptr, *cat = nullptr, *gu = nullptr, *act = nullptr;
   T* shifted[4] = {};
   int ld_raw = 0, ld_shift = 0;
@@ -78,7 +78,7 @@ struct block_context : context_impl {
     return nullptr;
   }
   int product(void* out, bool f32_out, const T* x, int ldx, const void* w, int rows, int N, int K);
-  int hyper(const hyper_weights& in, const float* norm_w, bool first, const hyper_weights* done, int rows, const block_layer* shift, T* prev);
+  int hyper(const hyper_weights& in, const float* norm_w, const hyper_weights* done, int rows, const block_layer* shift, T* prev);
   attn_rows<T> attention(int run, int b, int ld);
   scan_rows<T> recurrence(int run, int b, int ld);
   int mixer_rows(int run, int rows, int pos0);
@@ -111,7 +111,7 @@ int block_context<T>::product(void* out, bool f32_out, const T* x, int ldx, cons
 
 // residual pass in front of a sublayer (done: the sublayer whose result is in y, or null)
 template <typename T>
-int block_context<T>::hyper(const hyper_weights& in, const float* norm_w, bool, const hyper_weights* done, int rows, const block_layer* shift, T* prev) {
+int block_context<T>::hyper(const hyper_weights& in, const float* norm_w, const hyper_weights* done, int rows, const block_layer* shift, T* prev) {
   hyper_params<T> p{};
   p.xs = xs;
   p.width = width;
@@ -179,7 +179,6 @@ scan_rows<T> block_context<T>::recurrence(int run, int b, int ld) {
     s.k = shifted[1];
     s.v = shifted[2];
     s.ldq = s.ldk = s.ldv = L.shifted_rows[0];
-    s.w = decays;
     s.u = L.u;
   } else {
     const branch_weights& bw = L.branches[b];
@@ -194,6 +193,9 @@ scan_rows<T> block_context<T>::recurrence(int run, int b, int ld) {
   }
   s.out = raw;
   s.ldo = bs.out_cols();
+  s.packed = packed;
+  s.packed_v = packed_v;
+  s.err = gpus[0].state + 3;
   return s;
 }
 
@@ -210,7 +212,9 @@ int block_context<T>::mixer_rows(int run, int rows, int pos0) {
     LCU_TRY(launch_token_shift(h, K, runs[run].prev, L.mu, mix, stride, 5, rows, width, pos0, stream()));
     for (int j = 0; j < 4; ++j) LCU_TRY(product(shifted[j], false, mix + j * stride, K, L.shifted[j], rows, L.shifted_rows[j], K));
     LCU_TRY(product(low, true, mix + 4 * stride, K, L.shifted[4], rows, L.shifted_rows[4], K));
-    LCU_TRY(launch_wkv_decay(decays, low, L.shifted_rows[4], L.w2t, L.w0, L.rank, bs.out_cols(), rows, stream()));
+    size_t head_stride, row_stride, offset;
+    scan_decay_layout(bs.dim, bs.vdim, rows, &head_stride, &row_stride, &offset);
+    LCU_TRY(launch_wkv_decay(packed + offset, head_stride, row_stride, low, L.shifted_rows[4], L.w2t, L.w0, L.rank, bs.heads, bs.dim, rows, stream()));
     LCU_TRY(launch_scan(recurrence(run, 0, 0), true, rows, pos0, stream()));
     LCU_TRY(launch_head_gate(cat, L.out_k, raw, bs.out_cols(), shifted[3], L.shifted_rows[3], L.head_norm, bs.heads, bs.vdim, m->spec.eps, bs.out_scale,
                              rows, stream()));
@@ -222,7 +226,7 @@ int block_context<T>::mixer_rows(int run, int rows, int pos0) {
       if (bs.kind == BRANCH_WINDOW_ATTN) {
         const attn_rows<T> a = attention(run, (int)b, L.proj_rows);
         LCU_TRY(launch_window_append(a, rows, pos0, stream()));
-        LCU_TRY(launch_window_attention(a, rows, pos0, err(), stream()));
+        LCU_TRY(launch_window_attention(a, rows, pos0, stream()));
       } else {
         LCU_TRY(launch_scan(recurrence(run, (int)b, L.proj_rows), false, rows, pos0, stream()));
         LCU_TRY(launch_head_gate(cat + bw.out_col, L.out_k, raw, bs.out_cols(), proj + bw.g, L.proj_rows, (const float*)nullptr, bs.heads, bs.vdim,
@@ -390,11 +394,11 @@ int block_context<T>::enqueue_decode_step(int) {
     const int l = m->spec.runs[run];
     const block_layer& L = m->layers[l];
     const bool wkv = m->spec.layers[l].is_wkv();
-    LCU_TRY(hyper(L.hc1, L.norm1, run == 0, done, 1, wkv ? &L : nullptr, runs[run].prev));
+    LCU_TRY(hyper(L.hc1, L.norm1, done, 1, wkv ? &L : nullptr, runs[run].prev));
     LCU_TRY(mixer_one((int)run));
     done = &L.hc1;
     if (m->spec.layers[l].ff > 0) {
-      LCU_TRY(hyper(L.hc2, L.norm2, false, done, 1, nullptr, nullptr));
+      LCU_TRY(hyper(L.hc2, L.norm2, done, 1, nullptr, nullptr));
       LCU_TRY(feed_forward(L, 1));
       done = &L.hc2;
     }
@@ -430,11 +434,11 @@ int block_context<T>::enqueue_prefill(int m_rows, const pass_request& rq) {
     for (size_t run = 0; run < m->spec.runs.size(); ++run) {
       const int l = m->spec.runs[run];
       const block_layer& L = m->layers[l];
-      LCU_TRY(hyper(L.hc1, L.norm1, run == 0, done, rows, nullptr, nullptr));
+      LCU_TRY(hyper(L.hc1, L.norm1, done, rows, nullptr, nullptr));
       LCU_TRY(mixer_rows((int)run, rows, pos0));
       done = &L.hc1;
       if (m->spec.layers[l].ff > 0) {
-        LCU_TRY(hyper(L.hc2, L.norm2, false, done, rows, nullptr, nullptr));
+        LCU_TRY(hyper(L.hc2, L.norm2, done, rows, nullptr, nullptr));
         LCU_TRY(feed_forward(L, rows));
         done = &L.hc2;
       }
@@ -479,7 +483,7 @@ int block_context<T>::create(block_model* model, const context_options& o) {
   LCU_CUDA(cudaStreamCreateWithFlags(&g.stream, cudaStreamNonBlocking));
   LCU_CUDA(cudaEventCreateWithFlags(&g.ev, cudaEventDisableTiming));
   // widest rows over the layers
-  size_t w_proj = 0, w_cat = 0, w_gu = 0, w_raw = 0, w_shift = 0, w_low = 0;
+  size_t w_proj = 0, w_cat = 0, w_gu = 0, w_raw = 0, w_shift = 0, w_low = 0, w_packed = 0, w_values = 0;
   for (size_t i = 0; i < m->layers.size(); ++i) {
     const block_layer& L = m->layers[i];
     w_proj = std::max(w_proj, (size_t)L.proj_rows);
@@ -487,7 +491,14 @@ int block_context<T>::create(block_model* model, const context_options& o) {
     w_gu = std::max(w_gu, (size_t)L.ff_pad);
     w_shift = std::max(w_shift, (size_t)L.shifted_rows[0]);
     w_low = std::max(w_low, (size_t)L.shifted_rows[4]);
-    for (auto& b : m->spec.layers[i].branches) w_raw = std::max(w_raw, (size_t)b.out_cols());
+    for (auto& b : m->spec.layers[i].branches) {
+      w_raw = std::max(w_raw, (size_t)b.out_cols());
+      if (b.kind == BRANCH_WINDOW_ATTN) continue;
+      size_t pk = 0, pv = 0;
+      scan_scratch(b.heads, b.dim, b.vdim, b.kind == BRANCH_WKV, rows_cap, &pk, &pv);
+      w_packed = std::max(w_packed, pk);
+      w_values = std::max(w_values, pv);
+    }
   }
   const size_t R = rows_cap, K = m->k_width, es = sizeof(T);
   for (int pass = 0; pass < 2; ++pass) {
@@ -502,7 +513,8 @@ int block_context<T>::create(block_model* model, const context_options& o) {
     take(xs, R * m->spec.streams * width * 4);
     take(y, R * m->n_width * 4);
     take(raw, R * w_raw * 4);
-    take(decays, R * w_shift * 4);
+    take(packed, w_packed * 4);
+    take(packed_v, w_values * 4);
     take(low, R * w_low * 4);
     take(hidden, (size_t)width * 4);
     take(logits, std::min<size_t>(R, LOGIT_ROWS) * m->n_vocab_pad * 4);

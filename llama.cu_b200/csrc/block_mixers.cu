@@ -201,124 +201,185 @@ __global__ void __launch_bounds__(128) window_pool_kernel(const attn_rows<T> p, 
 }
 
 // ------------------------------------------------------------------ recurrences over rows
-// One CTA owns COLS = 128 / G value columns of one head; G neighbouring lanes share a column, each holding KC of its state
-// entries in registers for the whole pass.  Rows come through shared memory SC_ROWS at a time.  Lane `sub` of a column holds
-// channels (c / 4) * 4 G + 4 sub + c % 4, so that a warp reads its row vectors as contiguous 16-byte pieces.
+// Two launches.  The first lays a pass's rows out for the second, in binary32: per head and row q, k (rotated and scaled),
+// the decays of a wkv layer and its bonus sum_i q_i u_i k_i (the same for every value column) as one run of `stride`
+// floats, and the values by blocks of `cols` columns.  The second walks the rows: a CTA owns `cols` value columns of one
+// head with their whole state in registers - G lanes share NC columns, each lane holding KC channels of each - and rows
+// come in SC_ROWS at a time by bulk copies into a ring of stages.  Lane `sub` of a group holds channels
+// (c / 4) * 4 G + 4 sub + c % 4, so that a warp reads row vectors as contiguous 16-byte pieces.  The state is updated once
+// per row in row order, so neither the cut of a sequence into passes nor the pass length enters the arithmetic.
 constexpr int SC_THREADS = 128;
 constexpr int SC_ROWS = 16;
+constexpr int SC_MAX_STAGES = 4;
+constexpr int SC_NC = 2;
 
-template <typename T, int KC, bool WKV>
-__global__ void __launch_bounds__(SC_THREADS) scan_kernel(const scan_rows<T> p, int m, int pos0, int G) {
-  extern __shared__ __align__(16) float sm[];
-  const int dimp = G * KC, cols = SC_THREADS / G;
-  float* qs = sm;                       // [SC_ROWS][dimp]
-  float* ks = qs + SC_ROWS * dimp;      // [SC_ROWS][dimp]
-  float* ws = ks + SC_ROWS * dimp;      // [SC_ROWS][dimp], wkv
-  float* vs = ws + (WKV ? SC_ROWS * dimp : 0);  // [SC_ROWS][cols]
-  float* os = vs + SC_ROWS * cols;      // [SC_ROWS][cols]
-  const int tid = threadIdx.x, sub = tid % G, col = tid / G;
-  const int head = blockIdx.x, v0 = blockIdx.y * cols, D = p.dim, DV = p.vdim;
+struct scan_shape {
+  int kc, G, dimp, cols, blocks, stride;
+};
+scan_shape scan_shape_of(int dim, int vdim, bool wkv) {
+  scan_shape s;
+  s.kc = dim <= 16 ? 4 : dim <= 256 ? 8 : 16;
+  s.G = std::max(2, pow2_at_least((dim + s.kc - 1) / s.kc));
+  s.dimp = s.G * s.kc;
+  s.cols = SC_THREADS / s.G * SC_NC;
+  s.blocks = (vdim + s.cols - 1) / s.cols;
+  s.stride = (wkv ? 3 : 2) * s.dimp + 4;
+  return s;
+}
+
+template <typename T, bool WKV>
+__global__ void __launch_bounds__(128) scan_prepare_kernel(const scan_rows<T> p, const scan_shape z, int m, int pos0) {
   pdl_launch_dependents();
   pdl_wait();
-  float S[KC], u[KC];
-  float* st = p.state + (size_t)head * D * DV;
-  const bool live = v0 + col < DV;
-#pragma unroll
-  for (int c = 0; c < KC; ++c) {
-    const int i = (c >> 2) * 4 * G + 4 * sub + (c & 3);
-    S[c] = pos0 > 0 && live && i < D ? st[(size_t)i * DV + v0 + col] : 0.f;
-    u[c] = WKV && i < D ? p.u[head * D + i] : 0.f;
-  }
-  const float dec = WKV ? 0.f : p.decay[head];
-  for (int i = tid; i < SC_ROWS * dimp; i += SC_THREADS) {  // (channels past the head's size stay zero)
-    qs[i] = 0.f;
-    ks[i] = 0.f;
-    if (WKV) ws[i] = 0.f;
-  }
-  const int half = p.rot_dims >> 1;
-  for (int r0 = 0; r0 < m; r0 += SC_ROWS) {
-    const int nr = min(SC_ROWS, m - r0);
-    __syncthreads();
-    for (int i = tid; i < nr * D; i += SC_THREADS) {
-      const int r = i / D, d = i - r * D, row = r0 + r;
-      const T* qr = p.q + (size_t)row * p.ldq + head * D;
-      const T* kr = p.k + (size_t)row * p.ldk + head * D;
-      float qv = to_f(qr[d]), kv = to_f(kr[d]);
-      if (!WKV) {
-        if (d < p.rot_dims) {
-          const bool low = d < half;
-          const float2 cs = p.rope[(size_t)(pos0 + row) * half + (low ? d : d - half)];
-          const int pd = low ? d + half : d - half;
-          const float qo = to_f(qr[pd]), ko = to_f(kr[pd]);
-          qv = low ? qv * cs.x - qo * cs.y : qv * cs.x + qo * cs.y;
-          kv = low ? kv * cs.x - ko * cs.y : kv * cs.x + ko * cs.y;
-        }
-        kv *= p.kscale;
-      } else {
-        ws[r * dimp + d] = p.w[(size_t)row * p.heads * D + head * D + d];
-      }
-      qs[r * dimp + d] = qv;
-      ks[r * dimp + d] = kv;
-    }
-    for (int i = tid; i < nr * cols; i += SC_THREADS) {
-      const int r = i / cols, j = i - r * cols;
-      vs[i] = v0 + j < DV ? to_f(p.v[(size_t)(r0 + r) * p.ldv + head * DV + v0 + j]) : 0.f;
-    }
-    __syncthreads();
-#pragma unroll 4
-    for (int r = 0; r < nr; ++r) {
-      const float v = vs[r * cols + col];
-      float o = 0.f;
-#pragma unroll
-      for (int c4 = 0; c4 < KC / 4; ++c4) {
-        const int at = r * dimp + c4 * 4 * G + 4 * sub;
-        const float4 q4 = *reinterpret_cast<const float4*>(qs + at), k4 = *reinterpret_cast<const float4*>(ks + at);
-        float4 w4 = make_float4(dec, dec, dec, dec);
-        if (WKV) w4 = *reinterpret_cast<const float4*>(ws + at);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int c = c4 * 4 + e;
-          const float q = reinterpret_cast<const float*>(&q4)[e], k = reinterpret_cast<const float*>(&k4)[e], w = reinterpret_cast<const float*>(&w4)[e];
-          const float kv = k * v;
-          if (WKV) {
-            o = fmaf(q, fmaf(u[c], kv, S[c]), o);
-            S[c] = fmaf(w, S[c], kv);
-          } else {
-            S[c] = fmaf(w, S[c], kv);
-            o = fmaf(q, S[c], o);
+  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = p.rot_dims >> 1;
+  for (int head = blockIdx.y * 4 + warp; head < p.heads; head += gridDim.y * 4) {
+    const T* qr = p.q + (size_t)row * p.ldq + head * p.dim;
+    const T* kr = p.k + (size_t)row * p.ldk + head * p.dim;
+    float* out = p.packed + ((size_t)head * m + row) * z.stride;
+    float bonus = 0.f;
+    for (int d = lane; d < z.dimp; d += 32) {
+      float q = 0.f, k = 0.f;
+      if (d < p.dim) {
+        q = to_f(qr[d]);
+        k = to_f(kr[d]);
+        if (WKV) {
+          bonus = fmaf(q * p.u[head * p.dim + d], k, bonus);
+        } else {
+          if (d < p.rot_dims) {
+            const bool low = d < half;
+            const float2 cs = p.rope[(size_t)(pos0 + row) * half + (low ? d : d - half)];
+            const int pd = low ? d + half : d - half;
+            const float qo = to_f(qr[pd]), ko = to_f(kr[pd]);
+            q = low ? q * cs.x - qo * cs.y : q * cs.x + qo * cs.y;
+            k = low ? k * cs.x - ko * cs.y : k * cs.x + ko * cs.y;
           }
+          k *= p.kscale;
         }
       }
-      for (int s = G >> 1; s > 0; s >>= 1) o += __shfl_xor_sync(0xffffffffu, o, s);
-      if (sub == 0) os[r * cols + col] = o;
+      out[d] = q;
+      out[z.dimp + d] = k;
+      if (WKV && d >= p.dim) out[2 * z.dimp + d] = 0.f;  // (the other channels' decays are written by their own kernel)
     }
-    __syncthreads();
-    for (int i = tid; i < nr * cols; i += SC_THREADS) {
-      const int r = i / cols, j = i - r * cols;
-      if (v0 + j < DV) p.out[(size_t)(r0 + r) * p.ldo + head * DV + v0 + j] = os[i];
+    bonus = warp_sum(bonus);
+    if (lane < 4) out[z.stride - 4 + lane] = lane == 0 && WKV ? bonus : 0.f;
+    float* v = p.packed_v + (size_t)head * z.blocks * m * z.cols;
+    for (int j = lane; j < z.blocks * z.cols; j += 32) {
+      const int b = j / z.cols, c = j - b * z.cols;
+      v[((size_t)b * m + row) * z.cols + c] = j < p.vdim ? to_f(p.v[(size_t)row * p.ldv + head * p.vdim + j]) : 0.f;
     }
-  }
-#pragma unroll
-  for (int c = 0; c < KC; ++c) {
-    const int i = (c >> 2) * 4 * G + 4 * sub + (c & 3);
-    if (live && i < D) st[(size_t)i * DV + v0 + col] = S[c];
   }
 }
 
 template <typename T, int KC, bool WKV>
-int launch_scan_one(const scan_rows<T>& p, int m, int pos0, cudaStream_t stream) {
-  const int G = pow2_at_least((p.dim + KC - 1) / KC);
-  LCU_REQUIRE(G <= 32, "scan: head size %d", p.dim);
-  const int cols = SC_THREADS / G;
-  const size_t smem = (size_t)SC_ROWS * ((WKV ? 3 : 2) * G * KC + 2 * cols) * sizeof(float);
+__global__ void __launch_bounds__(SC_THREADS) scan_kernel(const scan_rows<T> p, const scan_shape z, int m, int pos0, int n_stages) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ uint64_t bars[SC_MAX_STAGES];
+  const int tid = threadIdx.x, G = z.G, sub = tid % G, grp = tid / G;
+  const int head = blockIdx.x, v0 = blockIdx.y * z.cols, D = p.dim, DV = p.vdim;
+  const int stage_floats = SC_ROWS * (z.stride + z.cols);
+  const int n_tiles = (m + SC_ROWS - 1) / SC_ROWS;
+  if (tid == 0) {
+    for (int i = 0; i < n_stages; ++i) mbar_init(smem_u32(&bars[i]), 1);
+    fence_mbar_init();
+  }
+  __syncthreads();
+  pdl_launch_dependents();
+  pdl_wait();
+  const float* rows = p.packed + (size_t)head * m * z.stride;
+  const float* vals = p.packed_v + ((size_t)head * z.blocks + blockIdx.y) * m * z.cols;
+  auto fetch = [&](int tile) {
+    const int s = tile % n_stages, nr = min(SC_ROWS, m - tile * SC_ROWS);
+    const uint32_t bar = smem_u32(&bars[s]), dst = smem_u32(sm + s * stage_floats);
+    const uint32_t b0 = (uint32_t)(nr * z.stride) * 4, b1 = (uint32_t)(nr * z.cols) * 4;
+    mbar_arrive_expect_tx(bar, b0 + b1);
+    bulk_g2s(dst, rows + (size_t)tile * SC_ROWS * z.stride, b0, bar);
+    bulk_g2s(dst + SC_ROWS * z.stride * 4, vals + (size_t)tile * SC_ROWS * z.cols, b1, bar);
+  };
+  if (tid == 0)
+    for (int t = 0; t < n_stages && t < n_tiles; ++t) fetch(t);
+
+  float S[SC_NC][KC];
+  float* st = p.state + (size_t)head * D * DV;
+  const int c0 = v0 + grp * SC_NC;  // first of this group's columns
+#pragma unroll
+  for (int n = 0; n < SC_NC; ++n)
+#pragma unroll
+    for (int c = 0; c < KC; ++c) {
+      const int i = (c >> 2) * 4 * G + 4 * sub + (c & 3);
+      S[n][c] = pos0 > 0 && c0 + n < DV && i < D ? st[(size_t)i * DV + c0 + n] : 0.f;
+    }
+  const float dec = WKV ? 0.f : p.decay[head];
+  const bool odd = sub & 1;
+  const int my_col = c0 + (odd ? 1 : 0);
+  float* out = p.out + head * DV + my_col;
+  const bool writes = sub < 2 && my_col < DV;
+  for (int tile = 0; tile < n_tiles; ++tile) {
+    const int s = tile % n_stages, nr = min(SC_ROWS, m - tile * SC_ROWS);
+    const bool ok = mbar_wait(smem_u32(&bars[s]), (uint32_t)(tile / n_stages) & 1u, p.err, DEV_ERR_FULL_WAIT);
+    const float* rs = sm + s * stage_floats;
+    const float* vs = rs + SC_ROWS * z.stride + grp * SC_NC;
+    if (ok) {
+#pragma unroll 4
+      for (int r = 0; r < nr; ++r) {
+        const float* row = rs + r * z.stride;
+        const float2 v = *reinterpret_cast<const float2*>(vs + r * z.cols);
+        float o0 = 0.f, o1 = 0.f;
+#pragma unroll
+        for (int c4 = 0; c4 < KC / 4; ++c4) {
+          const int at = c4 * 4 * G + 4 * sub;
+          const float4 q4 = *reinterpret_cast<const float4*>(row + at), k4 = *reinterpret_cast<const float4*>(row + z.dimp + at);
+          float4 w4 = make_float4(dec, dec, dec, dec);
+          if (WKV) w4 = *reinterpret_cast<const float4*>(row + 2 * z.dimp + at);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int c = c4 * 4 + e;
+            const float q = reinterpret_cast<const float*>(&q4)[e], k = reinterpret_cast<const float*>(&k4)[e], w = reinterpret_cast<const float*>(&w4)[e];
+            if (WKV) {
+              o0 = fmaf(q, S[0][c], o0);
+              o1 = fmaf(q, S[1][c], o1);
+              S[0][c] = fmaf(w, S[0][c], k * v.x);
+              S[1][c] = fmaf(w, S[1][c], k * v.y);
+            } else {
+              S[0][c] = fmaf(w, S[0][c], k * v.x);
+              S[1][c] = fmaf(w, S[1][c], k * v.y);
+              o0 = fmaf(q, S[0][c], o0);
+              o1 = fmaf(q, S[1][c], o1);
+            }
+          }
+        }
+        // even lanes go on with column 0, odd lanes with column 1
+        float o = (odd ? o1 : o0) + __shfl_xor_sync(0xffffffffu, odd ? o0 : o1, 1);
+        for (int x = 2; x < G; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
+        if (WKV) o = fmaf(row[z.stride - 4], odd ? v.y : v.x, o);
+        if (writes) out[(size_t)(tile * SC_ROWS + r) * p.ldo] = o;
+      }
+    }
+    __syncthreads();  // the stage may be overwritten
+    if (tid == 0 && tile + n_stages < n_tiles) fetch(tile + n_stages);
+  }
+#pragma unroll
+  for (int n = 0; n < SC_NC; ++n)
+#pragma unroll
+    for (int c = 0; c < KC; ++c) {
+      const int i = (c >> 2) * 4 * G + 4 * sub + (c & 3);
+      if (c0 + n < DV && i < D) st[(size_t)i * DV + c0 + n] = S[n][c];
+    }
+}
+
+template <typename T, int KC, bool WKV>
+int launch_scan_one(const scan_rows<T>& p, const scan_shape& z, int m, int pos0, cudaStream_t stream) {
+  const size_t stage = (size_t)SC_ROWS * (z.stride + z.cols) * sizeof(float);
+  const int n_stages = (int)std::min<size_t>(SC_MAX_STAGES, (200 * 1024) / stage);
+  LCU_REQUIRE(z.G <= 32 && n_stages >= 1, "scan: head size %d", p.dim);
   static bool attr_done[16] = {};
   int dev = 0;
   LCU_CUDA(cudaGetDevice(&dev));
   if (dev < 16 && !attr_done[dev]) {
-    LCU_CUDA(cudaFuncSetAttribute((scan_kernel<T, KC, WKV>), cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+    LCU_CUDA(cudaFuncSetAttribute((scan_kernel<T, KC, WKV>), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     attr_done[dev] = true;
   }
-  LCU_CUDA(launch_after(scan_kernel<T, KC, WKV>, dim3(p.heads, (p.vdim + cols - 1) / cols), dim3(SC_THREADS), smem, stream, p, m, pos0, G));
+  LCU_CUDA(launch_after(scan_prepare_kernel<T, WKV>, dim3(m, (p.heads + 3) / 4), dim3(128), 0, stream, p, z, m, pos0));
+  LCU_CUDA(launch_after(scan_kernel<T, KC, WKV>, dim3(p.heads, z.blocks), dim3(SC_THREADS), stage * n_stages, stream, p, z, m, pos0, n_stages));
   return LCU_OK;
 }
 
@@ -507,6 +568,11 @@ int most_keys(const attn_rows<T>& p, int last_pos) {
 
 }  // namespace
 
+int& window_mma_mode() {
+  static int mode = 1;
+  return mode;
+}
+
 template <typename T>
 int launch_window_append(const attn_rows<T>& p, int m, int pos0, cudaStream_t stream) {
   LCU_REQUIRE(pos0 >= 0 && pos0 + m <= p.cache.ctx_len, "window attention: rows %d..%d outside the cache of %d", pos0, pos0 + m, p.cache.ctx_len);
@@ -519,8 +585,9 @@ int launch_window_append(const attn_rows<T>& p, int m, int pos0, cudaStream_t st
 }
 
 template <typename T>
-int launch_window_attention(const attn_rows<T>& p, int m, int pos0, int* err, cudaStream_t stream) {
-  (void)err;
+int launch_window_attention(const attn_rows<T>& p, int m, int pos0, cudaStream_t stream) {
+  if constexpr (sizeof(T) == 2)
+    if (window_mma_mode() && window_mma_supported(p.dim, p.vdim)) return launch_window_mma(p, m, pos0, stream);
   const int keys = most_keys(p, pos0 + m - 1);
   const size_t smem = attention_smem(p, keys, false);
   LCU_REQUIRE(smem <= 220 * 1024, "window attention: %d visible keys", keys);
@@ -537,11 +604,24 @@ int launch_window_attention(const attn_rows<T>& p, int m, int pos0, int* err, cu
 
 template <typename T>
 int launch_scan(const scan_rows<T>& p, bool wkv, int m, int pos0, cudaStream_t stream) {
-#define LCU_SCAN(KC) return wkv ? launch_scan_one<T, KC, true>(p, m, pos0, stream) : launch_scan_one<T, KC, false>(p, m, pos0, stream)
-  if (p.dim <= 32) LCU_SCAN(4);
-  if (p.dim <= 64) LCU_SCAN(8);
+  const scan_shape z = scan_shape_of(p.dim, p.vdim, wkv);
+#define LCU_SCAN(KC) return wkv ? launch_scan_one<T, KC, true>(p, z, m, pos0, stream) : launch_scan_one<T, KC, false>(p, z, m, pos0, stream)
+  if (z.kc == 4) LCU_SCAN(4);
+  if (z.kc == 8) LCU_SCAN(8);
   LCU_SCAN(16);
 #undef LCU_SCAN
+}
+
+void scan_scratch(int heads, int dim, int vdim, bool wkv, size_t rows, size_t* packed_floats, size_t* value_floats) {
+  const scan_shape z = scan_shape_of(dim, vdim, wkv);
+  *packed_floats = heads * rows * z.stride;
+  *value_floats = heads * rows * z.blocks * z.cols;
+}
+void scan_decay_layout(int dim, int vdim, int m, size_t* head_stride, size_t* row_stride, size_t* offset) {
+  const scan_shape z = scan_shape_of(dim, vdim, true);
+  *head_stride = (size_t)m * z.stride;
+  *row_stride = z.stride;
+  *offset = 2 * (size_t)z.dimp;
 }
 
 template <typename T>
@@ -565,7 +645,7 @@ int launch_mixer_step(const mixer_step<T>& p, int ctx_len, cudaStream_t stream) 
 
 #define LCU_BLOCK_MIXERS(T)                                                                    \
   template int launch_window_append<T>(const attn_rows<T>&, int, int, cudaStream_t);           \
-  template int launch_window_attention<T>(const attn_rows<T>&, int, int, int*, cudaStream_t);  \
+  template int launch_window_attention<T>(const attn_rows<T>&, int, int, cudaStream_t);  \
   template int launch_scan<T>(const scan_rows<T>&, bool, int, int, cudaStream_t);              \
   template int launch_mixer_step<T>(const mixer_step<T>&, int, cudaStream_t);
 LCU_BLOCK_MIXERS(__nv_bfloat16)

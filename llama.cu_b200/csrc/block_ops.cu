@@ -166,23 +166,34 @@ int launch_hyper_one(const hyper_params<T>& p, int n_rows, cudaStream_t stream) 
 }
 
 // ------------------------------------------------------------------ token shift
-template <typename T>
+// V elements per thread and step (width a multiple of V)
+template <typename T, int V>
 __global__ void __launch_bounds__(256) token_shift_kernel(const T* h, int ldh, T* prev, const float* mu, T* mix, size_t mix_stride, int n_mix, int m,
                                                           int width, int pos0) {
+  struct __align__(V * sizeof(T) >= 16 ? 16 : sizeof(T)) pack { T e[V]; };
   pdl_launch_dependents();
   pdl_wait();
   const int r = blockIdx.x;
-  for (int c = threadIdx.x; c < width; c += 256) {
-    const float hf = to_f(h[(size_t)r * ldh + c]);
-    float hp;
+  for (int c = threadIdx.x * V; c < width; c += 256 * V) {
+    const pack hv = *reinterpret_cast<const pack*>(h + (size_t)r * ldh + c);
+    pack pv;
     if (r > 0) {
-      hp = to_f(h[(size_t)(r - 1) * ldh + c]);
+      pv = *reinterpret_cast<const pack*>(h + (size_t)(r - 1) * ldh + c);
     } else {
-      hp = pos0 == 0 ? 0.f : to_f(prev[c]);
-      prev[c] = h[(size_t)(m - 1) * ldh + c];  // (only row 0 touches prev)
+      pv = *reinterpret_cast<const pack*>(prev + c);
+      if (pos0 == 0)
+        for (int e = 0; e < V; ++e) pv.e[e] = from_f<T>(0.f);
+      *reinterpret_cast<pack*>(prev + c) = *reinterpret_cast<const pack*>(h + (size_t)(m - 1) * ldh + c);  // (only row 0 touches prev)
     }
-    const float d = hp - hf;
-    for (int i = 0; i < n_mix; ++i) mix[i * mix_stride + (size_t)r * ldh + c] = from_f<T>(fmaf(d, mu[(size_t)i * width + c], hf));
+    for (int i = 0; i < n_mix; ++i) {
+      pack o;
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        const float hf = to_f(hv.e[e]);
+        o.e[e] = from_f<T>(fmaf(to_f(pv.e[e]) - hf, mu[(size_t)i * width + c + e], hf));
+      }
+      *reinterpret_cast<pack*>(mix + i * mix_stride + (size_t)r * ldh + c) = o;
+    }
   }
 }
 
@@ -195,33 +206,44 @@ __global__ void rotation_table_kernel(float2* table, int n_pos, int half, double
 }
 
 // ------------------------------------------------------------------ wkv decays
-constexpr int WD_ROWS = 8;
-__global__ void __launch_bounds__(256) wkv_decay_kernel(float* w, const float* low, int ld_low, const float* w2t, const float* w0, int rank,
-                                                        int channels, int m) {
-  extern __shared__ float th[];  // [WD_ROWS][rank]
+constexpr int WD_ROWS = 32;
+__global__ void __launch_bounds__(128) wkv_decay_kernel(float* w, size_t head_stride, size_t row_stride, const float* low, int ld_low, const float* w2t,
+                                                        const float* w0, int rank, int heads, int dim, int m) {
+  extern __shared__ __align__(16) float th[];  // [WD_ROWS][rank rounded up to 4]
   pdl_launch_dependents();
   pdl_wait();
-  const int r0 = blockIdx.y * WD_ROWS, nr = min(WD_ROWS, m - r0);
-  for (int i = threadIdx.x; i < WD_ROWS * rank; i += 256) {
-    const int r = i / rank, j = i - r * rank;
-    th[i] = r < nr ? tanhf(low[(size_t)(r0 + r) * ld_low + j]) : 0.f;
+  const int r0 = blockIdx.y * WD_ROWS, nr = min(WD_ROWS, m - r0), rp = (rank + 3) / 4 * 4, channels = heads * dim;
+  for (int i = threadIdx.x; i < WD_ROWS * rp; i += 128) {
+    const int r = i / rp, j = i - r * rp;
+    th[i] = r < nr && j < rank ? tanhf(low[(size_t)(r0 + r) * ld_low + j]) : 0.f;
   }
   __syncthreads();
-  const int ch = blockIdx.x * 256 + threadIdx.x;
+  const int ch = blockIdx.x * 128 + threadIdx.x;
   if (ch >= channels) return;
   float acc[WD_ROWS];
+  const float z0 = w0[ch];
 #pragma unroll
-  for (int r = 0; r < WD_ROWS; ++r) acc[r] = w0[ch];
-  for (int j = 0; j < rank; ++j) {
-    const float a = w2t[(size_t)j * channels + ch];
+  for (int r = 0; r < WD_ROWS; ++r) acc[r] = z0;
+  for (int j = 0; j < rank; j += 4) {
+    float a[4];
 #pragma unroll
-    for (int r = 0; r < WD_ROWS; ++r) acc[r] = fmaf(a, th[r * rank + j], acc[r]);
+    for (int e = 0; e < 4; ++e) a[e] = j + e < rank ? w2t[(size_t)(j + e) * channels + ch] : 0.f;
+#pragma unroll
+    for (int r = 0; r < WD_ROWS; ++r) {
+      const float4 t = *reinterpret_cast<const float4*>(th + r * rp + j);
+      acc[r] = fmaf(a[3], t.w, fmaf(a[2], t.z, fmaf(a[1], t.y, fmaf(a[0], t.x, acc[r]))));
+    }
   }
-  for (int r = 0; r < nr; ++r) w[(size_t)(r0 + r) * channels + ch] = expf(-expf(acc[r]));
+  const int head = ch / dim, d = ch - head * dim;
+  float* out = w + head * head_stride + r0 * row_stride + d;
+#pragma unroll
+  for (int r = 0; r < WD_ROWS; ++r)
+    if (r < nr) out[r * row_stride] = expf(-expf(acc[r]));
 }
 
 // ------------------------------------------------------------------ normalised, gated heads (one warp per row and head)
-template <typename T>
+// VEC 4: head sizes that are multiples of 4 with aligned rows, up to 512; VEC 1: anything
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) head_gate_kernel(T* out, int ldo, const float* o, int ld_raw, const T* g, int ldg, const float* norm, int heads,
                                                         int vdim, float eps, float out_scale, int m) {
   pdl_launch_dependents();
@@ -229,16 +251,49 @@ __global__ void __launch_bounds__(256) head_gate_kernel(T* out, int ldo, const f
   const int idx = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (idx >= m * heads) return;
   const int r = idx / heads, hd = idx - r * heads;
+  constexpr int N = 512 / (32 * VEC);  // vectors per lane
   const float* x = o + (size_t)r * ld_raw + hd * vdim;
+  const T* gr = g + (size_t)r * ldg + hd * vdim;
+  __align__(16) float xv[N][VEC];
+  __align__(16) T gv[N][VEC];
   float ss = 0.f;
-  for (int j = lane; j < vdim; j += 32) ss = fmaf(x[j], x[j], ss);
+#pragma unroll
+  for (int n = 0; n < N; ++n) {
+    const int j = (n * 32 + lane) * VEC;
+    if (j < vdim) {
+      if (VEC == 4) {
+        *reinterpret_cast<float4*>(xv[n]) = *reinterpret_cast<const float4*>(x + j);
+        if (sizeof(T) == 2) *reinterpret_cast<uint2*>(gv[n]) = *reinterpret_cast<const uint2*>(gr + j);
+        else *reinterpret_cast<uint4*>(gv[n]) = *reinterpret_cast<const uint4*>(gr + j);
+      } else {
+        xv[n][0] = x[j];
+        gv[n][0] = gr[j];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss = fmaf(xv[n][e], xv[n][e], ss);
+    }
+  }
   ss = warp_sum(ss);
   const float inv = 1.0f / sqrtf(ss / (float)vdim + eps);
-  for (int j = lane; j < vdim; j += 32) {
-    const int c = hd * vdim + j;
-    float v = x[j] * inv;
-    if (norm) v *= norm[c];
-    out[(size_t)r * ldo + c] = from_f<T>(v * silu_f(to_f(g[(size_t)r * ldg + c])) * out_scale);
+#pragma unroll
+  for (int n = 0; n < N; ++n) {
+    const int j = (n * 32 + lane) * VEC;
+    if (j < vdim) {
+      __align__(16) T y[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        float v = xv[n][e] * inv;
+        if (norm) v *= norm[hd * vdim + j + e];
+        y[e] = from_f<T>(v * silu_f(to_f(gv[n][e])) * out_scale);
+      }
+      T* dst = out + (size_t)r * ldo + hd * vdim + j;
+      if (VEC == 4) {
+        if (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(y);
+        else *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(y);
+      } else {
+        dst[0] = y[0];
+      }
+    }
   }
 }
 
@@ -354,7 +409,8 @@ int launch_hyper_rows(const hyper_params<T>& p, int n_rows, cudaStream_t stream)
 template <typename T>
 int launch_token_shift(const T* h, int ldh, T* prev, const float* mu, T* mix, size_t mix_stride, int n_mix, int m, int width, int pos0,
                        cudaStream_t stream) {
-  LCU_CUDA(launch_after(token_shift_kernel<T>, dim3(m), dim3(256), 0, stream, h, ldh, prev, mu, mix, mix_stride, n_mix, m, width, pos0));
+  if (width % 8 == 0) LCU_CUDA(launch_after(token_shift_kernel<T, 8>, dim3(m), dim3(256), 0, stream, h, ldh, prev, mu, mix, mix_stride, n_mix, m, width, pos0));
+  else LCU_CUDA(launch_after(token_shift_kernel<T, 1>, dim3(m), dim3(256), 0, stream, h, ldh, prev, mu, mix, mix_stride, n_mix, m, width, pos0));
   return LCU_OK;
 }
 
@@ -365,18 +421,25 @@ int launch_rotation_table(float2* table, int n_pos, int dims, double base, cudaS
   return LCU_OK;
 }
 
-int launch_wkv_decay(float* w, const float* low, int ld_low, const float* w2t, const float* w0, int rank, int channels, int m, cudaStream_t stream) {
-  LCU_REQUIRE((size_t)WD_ROWS * rank * 4 <= 48 * 1024, "wkv_decay: rank %d", rank);
-  LCU_CUDA(launch_after(wkv_decay_kernel, dim3((channels + 255) / 256, (m + WD_ROWS - 1) / WD_ROWS), dim3(256), (size_t)WD_ROWS * rank * 4, stream, w, low,
-                        ld_low, w2t, w0, rank, channels, m));
+int launch_wkv_decay(float* w, size_t head_stride, size_t row_stride, const float* low, int ld_low, const float* w2t, const float* w0, int rank, int heads,
+                     int dim, int m, cudaStream_t stream) {
+  const size_t smem = (size_t)WD_ROWS * round_up(rank, 4) * 4;
+  LCU_REQUIRE(smem <= 160 * 1024, "wkv_decay: rank %d", rank);
+  if (smem > 48 * 1024) LCU_CUDA(cudaFuncSetAttribute(wkv_decay_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  LCU_CUDA(launch_after(wkv_decay_kernel, dim3((heads * dim + 127) / 128, (m + WD_ROWS - 1) / WD_ROWS), dim3(128), smem, stream, w, head_stride, row_stride, low,
+                        ld_low, w2t, w0, rank, heads, dim, m));
   return LCU_OK;
 }
 
 template <typename T>
 int launch_head_gate(T* out, int ldo, const float* o, int ld_raw, const T* g, int ldg, const float* norm, int heads, int vdim, float eps,
                      float out_scale, int m, cudaStream_t stream) {
-  LCU_CUDA(launch_after(head_gate_kernel<T>, dim3((unsigned)ceil_div((size_t)m * heads, 8)), dim3(256), 0, stream, out, ldo, o, ld_raw, g, ldg, norm, heads,
-                        vdim, eps, out_scale, m));
+  LCU_REQUIRE(vdim <= 512, "head_gate: head size %d", vdim);
+  const dim3 grid((unsigned)ceil_div((size_t)m * heads, 8));
+  const size_t al = 4 * sizeof(T) - 1;
+  const bool vec = vdim % 4 == 0 && ldo % 4 == 0 && ldg % 4 == 0 && ld_raw % 4 == 0 && (((uintptr_t)out | (uintptr_t)g) & al) == 0 && ((uintptr_t)o & 15) == 0;
+  if (vec) LCU_CUDA(launch_after(head_gate_kernel<T, 4>, grid, dim3(256), 0, stream, out, ldo, o, ld_raw, g, ldg, norm, heads, vdim, eps, out_scale, m));
+  else LCU_CUDA(launch_after(head_gate_kernel<T, 1>, grid, dim3(256), 0, stream, out, ldo, o, ld_raw, g, ldg, norm, heads, vdim, eps, out_scale, m));
   return LCU_OK;
 }
 

@@ -87,8 +87,12 @@ struct attn_rows {
 // cache rows pos0 .. pos0+m-1, then the blocks they complete, then attention of the rows
 template <typename T>
 int launch_window_append(const attn_rows<T>& p, int m, int pos0, cudaStream_t stream);
+// (bfloat16 rows with heads of up to 128 take the tensor-core kernel of block_attn.cu)
+bool window_mma_supported(int dim, int vdim);
+int launch_window_mma(const attn_rows<__nv_bfloat16>& p, int m, int pos0, cudaStream_t stream);
+int& window_mma_mode();  // 1 (default) = where supported, 0 = never
 template <typename T>
-int launch_window_attention(const attn_rows<T>& p, int m, int pos0, int* err, cudaStream_t stream);
+int launch_window_attention(const attn_rows<T>& p, int m, int pos0, cudaStream_t stream);
 
 // ---- linear recurrences over rows, per head:
 //   retention: S <- decay S + k v^T, o = S^T q          (k and q rotated, k times kscale)
@@ -103,16 +107,21 @@ struct scan_rows {
   int rot_dims;
   float kscale;
   const float* decay;     // retention: per head
-  const float* w;         // wkv: [rows][heads * dim]
   const float* u;         // wkv: [heads][dim]
   float* out;             // [rows][ldo] binary32
   int ldo;
+  float *packed, *packed_v;  // scratch of scan_scratch() floats; wkv: the decays are in `packed` already (scan_decay_layout)
+  int* err;
 };
+void scan_scratch(int heads, int dim, int vdim, bool wkv, size_t rows, size_t* packed_floats, size_t* value_floats);
+// where the decay of (head, row, channel) of an m-row pass goes: packed[offset + head * head_stride + row * row_stride + channel]
+void scan_decay_layout(int dim, int vdim, int m, size_t* head_stride, size_t* row_stride, size_t* offset);
 template <typename T>
 int launch_scan(const scan_rows<T>& p, bool wkv, int m, int pos0, cudaStream_t stream);
 
-// w[row][ch] = exp(-exp(w0[ch] + sum_r w2t[r][ch] tanh(low[row][r])))
-int launch_wkv_decay(float* w, const float* low, int ld_low, const float* w2t, const float* w0, int rank, int channels, int m, cudaStream_t stream);
+// decay of channel ch = head * dim + d: w[head * head_stride + row * row_stride + d] = exp(-exp(w0[ch] + sum_r w2t[r][ch] tanh(low[row][r])))
+int launch_wkv_decay(float* w, size_t head_stride, size_t row_stride, const float* low, int ld_low, const float* w2t, const float* w0, int rank, int heads,
+                     int dim, int m, cudaStream_t stream);
 
 // out[row][head * vdim + j] = o / rms(o of the head) * norm * silu(g) * out_scale
 template <typename T>
@@ -125,7 +134,7 @@ struct step_branch {
   int kind;               // branch_kind
   int first;              // first cluster of the launch
   attn_rows<T> attn;      // attention (row pointers: the token's row)
-  scan_rows<T> scan;      // recurrences; w unused
+  scan_rows<T> scan;      // recurrences
   const T* g;             // gate projection of the token
   const float* low;       // wkv: input of the decay's second product
   const float *w2t, *w0;

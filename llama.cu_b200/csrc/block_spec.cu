@@ -33,6 +33,15 @@ int need_float(const json_value& o, const char* key, float* out) {
   *out = (float)v->number;
   return LCU_OK;
 }
+// an integer factor of a sum that is taken modulo `mod`
+int need_residue(const json_value& o, const char* key, int mod, long long* out) {
+  const json_value* v = nullptr;
+  int rc = need(o, key, json_value::NUMBER, &v);
+  if (rc) return rc;
+  LCU_REQUIRE(v->number == std::floor(v->number) && std::fabs(v->number) <= 9007199254740992.0, "config.json: '%s' = %g is not an integer", key, v->number);
+  *out = ((long long)v->number % mod + mod) % mod;
+  return LCU_OK;
+}
 #define SPEC_TRY(expr)   \
   do {                   \
     int _rc = (expr);    \
@@ -97,12 +106,9 @@ int read_stack(const json_value& c, block_spec& s) {
   if (const json_value* e = c.get("embedding")) {
     if (e->get("scale")) SPEC_TRY(need_float(*e, "scale", &s.embed_scale));
     if (const json_value* b = e->get("bigram")) {
-      int cur = 0, prev = 0;
       SPEC_TRY(need_int(*b, "buckets", &s.buckets));
-      SPEC_TRY(need_int(*b, "mul_cur", &cur, 0));
-      SPEC_TRY(need_int(*b, "mul_prev", &prev, 0));
-      s.mul_cur = cur;
-      s.mul_prev = prev;
+      SPEC_TRY(need_residue(*b, "mul_cur", s.buckets, &s.mul_cur));
+      SPEC_TRY(need_residue(*b, "mul_prev", s.buckets, &s.mul_prev));
     }
   }
   return LCU_OK;

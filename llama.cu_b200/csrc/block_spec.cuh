@@ -44,7 +44,7 @@ struct block_spec {
   int vocab = 0, width = 0, streams = 1;
   float eps = 0.f, embed_scale = 1.f;
   int buckets = 0;  // 0: no bigram embedding
-  long long mul_prev = 0, mul_cur = 0;
+  long long mul_prev = 0, mul_cur = 0;  // modulo buckets
   std::vector<layer_spec> layers;
   std::vector<int> runs;  // layer of every layer run, in order: a looped range appears once per pass
 };
