@@ -227,56 +227,88 @@ scan_shape scan_shape_of(int dim, int vdim, bool wkv) {
   return s;
 }
 
+constexpr int SP_ROWS = 4;  // rows per warp
 template <typename T, bool WKV>
-__global__ void __launch_bounds__(128) scan_prepare_kernel(const scan_rows<T> p, const scan_shape z, int m, int pos0) {
+__global__ void __launch_bounds__(256) scan_prepare_kernel(const scan_rows<T> p, const scan_shape z, int m, int pos0) {
   pdl_launch_dependents();
   pdl_wait();
-  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = p.rot_dims >> 1;
-  for (int head = blockIdx.y * 4 + warp; head < p.heads; head += gridDim.y * 4) {
-    const T* qr = p.q + (size_t)row * p.ldq + head * p.dim;
-    const T* kr = p.k + (size_t)row * p.ldk + head * p.dim;
-    float* out = p.packed + ((size_t)head * m + row) * z.stride;
-    float bonus = 0.f;
-    for (int d = lane; d < z.dimp; d += 32) {
-      float q = 0.f, k = 0.f;
-      if (d < p.dim) {
-        q = to_f(qr[d]);
-        k = to_f(kr[d]);
-        if (WKV) {
-          bonus = fmaf(q * p.u[head * p.dim + d], k, bonus);
-        } else {
-          if (d < p.rot_dims) {
-            const bool low = d < half;
-            const float2 cs = p.rope[(size_t)(pos0 + row) * half + (low ? d : d - half)];
-            const int pd = low ? d + half : d - half;
-            const float qo = to_f(qr[pd]), ko = to_f(kr[pd]);
-            q = low ? q * cs.x - qo * cs.y : q * cs.x + qo * cs.y;
-            k = low ? k * cs.x - ko * cs.y : k * cs.x + ko * cs.y;
-          }
-          k *= p.kscale;
-        }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = p.rot_dims >> 1;
+  const int head = blockIdx.y * 8 + warp, r0 = blockIdx.x * SP_ROWS, nr = min(SP_ROWS, m - r0);
+  if (head >= p.heads) return;
+  float* out = p.packed + ((size_t)head * m + r0) * z.stride;
+  float bonus[SP_ROWS] = {};
+  for (int d = lane; d < z.dimp; d += 32) {
+    const bool in = d < p.dim, turn = !WKV && d < p.rot_dims, low = d < half;
+    const int pd = low ? d + half : d - half;
+    const float u = WKV && in ? p.u[head * p.dim + d] : 0.f;
+    float q[SP_ROWS], k[SP_ROWS], qo[SP_ROWS], ko[SP_ROWS];
+    float2 cs[SP_ROWS];
+#pragma unroll
+    for (int r = 0; r < SP_ROWS; ++r) {
+      const T* qr = p.q + (size_t)(r0 + r) * p.ldq + head * p.dim;
+      const T* kr = p.k + (size_t)(r0 + r) * p.ldk + head * p.dim;
+      const bool live = in && r < nr;
+      q[r] = live ? to_f(qr[d]) : 0.f;
+      k[r] = live ? to_f(kr[d]) : 0.f;
+      if (live && turn) {
+        qo[r] = to_f(qr[pd]);
+        ko[r] = to_f(kr[pd]);
+        cs[r] = p.rope[(size_t)(pos0 + r0 + r) * half + (low ? d : d - half)];
       }
-      out[d] = q;
-      out[z.dimp + d] = k;
-      if (WKV && d >= p.dim) out[2 * z.dimp + d] = 0.f;  // (the other channels' decays are written by their own kernel)
     }
-    bonus = warp_sum(bonus);
-    if (lane < 4) out[z.stride - 4 + lane] = lane == 0 && WKV ? bonus : 0.f;
-    float* v = p.packed_v + (size_t)head * z.blocks * m * z.cols;
-    for (int j = lane; j < z.blocks * z.cols; j += 32) {
-      const int b = j / z.cols, c = j - b * z.cols;
-      v[((size_t)b * m + row) * z.cols + c] = j < p.vdim ? to_f(p.v[(size_t)row * p.ldv + head * p.vdim + j]) : 0.f;
+#pragma unroll
+    for (int r = 0; r < SP_ROWS; ++r) {
+      if (r >= nr) continue;
+      if (WKV) {
+        bonus[r] = fmaf(q[r] * u, k[r], bonus[r]);
+      } else {
+        if (turn) {
+          q[r] = low ? q[r] * cs[r].x - qo[r] * cs[r].y : q[r] * cs[r].x + qo[r] * cs[r].y;
+          k[r] = low ? k[r] * cs[r].x - ko[r] * cs[r].y : k[r] * cs[r].x + ko[r] * cs[r].y;
+        }
+        k[r] *= p.kscale;
+      }
+      float* o = out + (size_t)r * z.stride;
+      o[d] = q[r];
+      o[z.dimp + d] = k[r];
+      if (WKV && !in) o[2 * z.dimp + d] = 0.f;  // (the other channels' decays are written by their own kernel)
     }
+  }
+#pragma unroll
+  for (int r = 0; r < SP_ROWS; ++r) {
+    const float b = warp_sum(bonus[r]);
+    if (lane < 4 && r < nr) out[(size_t)r * z.stride + z.stride - 4 + lane] = lane == 0 && WKV ? b : 0.f;
+  }
+  float* v = p.packed_v + (size_t)head * z.blocks * m * z.cols;
+  for (int j = lane; j < z.blocks * z.cols; j += 32) {
+    const int b = j / z.cols, c = j - b * z.cols;
+    float x[SP_ROWS];
+#pragma unroll
+    for (int r = 0; r < SP_ROWS; ++r) x[r] = j < p.vdim && r < nr ? to_f(p.v[(size_t)(r0 + r) * p.ldv + head * p.vdim + j]) : 0.f;
+#pragma unroll
+    for (int r = 0; r < SP_ROWS; ++r)
+      if (r < nr) v[((size_t)b * m + r0 + r) * z.cols + c] = x[r];
   }
 }
 
-template <typename T, int KC, bool WKV>
-__global__ void __launch_bounds__(SC_THREADS) scan_kernel(const scan_rows<T> p, const scan_shape z, int m, int pos0, int n_stages) {
+struct scan_args {  // what the second launch needs of scan_rows
+  const float *packed, *packed_v, *decay;
+  float *state, *out;
+  int dim, vdim, ldo;
+  int* err;
+};
+
+template <int KC, int G, bool WKV>
+__global__ void __launch_bounds__(SC_THREADS) scan_kernel(const scan_args p, const scan_shape z, int m, int pos0, int n_stages) {
+  constexpr int RB = 4;                         // rows reduced together
+  constexpr int SPREAD = G < 8 ? G : 8;         // lanes of a group that end up with results
+  constexpr int KEEP = RB * SC_NC / SPREAD;     // results per such lane
+  constexpr int DIMP = G * KC, STRIDE = (WKV ? 3 : 2) * DIMP + 4, COLS = SC_THREADS / G * SC_NC;
   extern __shared__ __align__(16) float sm[];
   __shared__ uint64_t bars[SC_MAX_STAGES];
-  const int tid = threadIdx.x, G = z.G, sub = tid % G, grp = tid / G;
-  const int head = blockIdx.x, v0 = blockIdx.y * z.cols, D = p.dim, DV = p.vdim;
-  const int stage_floats = SC_ROWS * (z.stride + z.cols);
+  const int tid = threadIdx.x, sub = tid % G, grp = tid / G;
+  const int head = blockIdx.x, v0 = blockIdx.y * COLS, D = p.dim, DV = p.vdim;
+  constexpr int STAGE = SC_ROWS * (STRIDE + COLS);
   const int n_tiles = (m + SC_ROWS - 1) / SC_ROWS;
   if (tid == 0) {
     for (int i = 0; i < n_stages; ++i) mbar_init(smem_u32(&bars[i]), 1);
@@ -285,15 +317,15 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(const scan_rows<T> p, 
   __syncthreads();
   pdl_launch_dependents();
   pdl_wait();
-  const float* rows = p.packed + (size_t)head * m * z.stride;
-  const float* vals = p.packed_v + ((size_t)head * z.blocks + blockIdx.y) * m * z.cols;
+  const float* rows = p.packed + (size_t)head * m * STRIDE;
+  const float* vals = p.packed_v + ((size_t)head * z.blocks + blockIdx.y) * m * COLS;
   auto fetch = [&](int tile) {
     const int s = tile % n_stages, nr = min(SC_ROWS, m - tile * SC_ROWS);
-    const uint32_t bar = smem_u32(&bars[s]), dst = smem_u32(sm + s * stage_floats);
-    const uint32_t b0 = (uint32_t)(nr * z.stride) * 4, b1 = (uint32_t)(nr * z.cols) * 4;
+    const uint32_t bar = smem_u32(&bars[s]), dst = smem_u32(sm + s * STAGE);
+    const uint32_t b0 = (uint32_t)(nr * STRIDE) * 4, b1 = (uint32_t)(nr * COLS) * 4;
     mbar_arrive_expect_tx(bar, b0 + b1);
-    bulk_g2s(dst, rows + (size_t)tile * SC_ROWS * z.stride, b0, bar);
-    bulk_g2s(dst + SC_ROWS * z.stride * 4, vals + (size_t)tile * SC_ROWS * z.cols, b1, bar);
+    bulk_g2s(dst, rows + (size_t)tile * SC_ROWS * STRIDE, b0, bar);
+    bulk_g2s(dst + SC_ROWS * STRIDE * 4, vals + (size_t)tile * SC_ROWS * COLS, b1, bar);
   };
   if (tid == 0)
     for (int t = 0; t < n_stages && t < n_tiles; ++t) fetch(t);
@@ -310,48 +342,81 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(const scan_rows<T> p, 
     }
   const float dec = WKV ? 0.f : p.decay[head];
   const bool odd = sub & 1;
-  const int my_col = c0 + (odd ? 1 : 0);
-  float* out = p.out + head * DV + my_col;
-  const bool writes = sub < 2 && my_col < DV;
+
+  // one row: updates the state, leaves this lane's share of both columns' results in o
+  auto advance = [&](const float* row, const float* val, float (&o)[SC_NC]) {
+    const float2 v = *reinterpret_cast<const float2*>(val);
+    o[0] = o[1] = 0.f;
+#pragma unroll
+    for (int c4 = 0; c4 < KC / 4; ++c4) {
+      const int at = c4 * 4 * G + 4 * sub;
+      const float4 q4 = *reinterpret_cast<const float4*>(row + at), k4 = *reinterpret_cast<const float4*>(row + DIMP + at);
+      float4 w4 = make_float4(dec, dec, dec, dec);
+      if (WKV) w4 = *reinterpret_cast<const float4*>(row + 2 * DIMP + at);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int c = c4 * 4 + e;
+        const float q = reinterpret_cast<const float*>(&q4)[e], k = reinterpret_cast<const float*>(&k4)[e], w = reinterpret_cast<const float*>(&w4)[e];
+        if (WKV) {
+          o[0] = fmaf(q, S[0][c], o[0]);
+          o[1] = fmaf(q, S[1][c], o[1]);
+        }
+        S[0][c] = fmaf(w, S[0][c], k * v.x);
+        S[1][c] = fmaf(w, S[1][c], k * v.y);
+        if (!WKV) {
+          o[0] = fmaf(q, S[0][c], o[0]);
+          o[1] = fmaf(q, S[1][c], o[1]);
+        }
+      }
+    }
+  };
   for (int tile = 0; tile < n_tiles; ++tile) {
     const int s = tile % n_stages, nr = min(SC_ROWS, m - tile * SC_ROWS);
-    const bool ok = mbar_wait(smem_u32(&bars[s]), (uint32_t)(tile / n_stages) & 1u, p.err, DEV_ERR_FULL_WAIT);
-    const float* rs = sm + s * stage_floats;
-    const float* vs = rs + SC_ROWS * z.stride + grp * SC_NC;
-    if (ok) {
-#pragma unroll 4
-      for (int r = 0; r < nr; ++r) {
-        const float* row = rs + r * z.stride;
-        const float2 v = *reinterpret_cast<const float2*>(vs + r * z.cols);
-        float o0 = 0.f, o1 = 0.f;
+    mbar_wait(smem_u32(&bars[s]), (uint32_t)(tile / n_stages) & 1u, p.err, DEV_ERR_FULL_WAIT);  // (expired: the error word is set, results are not used)
+    const float* rs = sm + s * STAGE;
+    const float* vs = rs + SC_ROWS * STRIDE + grp * SC_NC;
+    float* out = p.out + (size_t)tile * SC_ROWS * p.ldo + head * DV;
+    int r = 0;
+#pragma unroll 1
+    for (; r + RB <= nr; r += RB) {
+      float o[RB][SC_NC];
 #pragma unroll
-        for (int c4 = 0; c4 < KC / 4; ++c4) {
-          const int at = c4 * 4 * G + 4 * sub;
-          const float4 q4 = *reinterpret_cast<const float4*>(row + at), k4 = *reinterpret_cast<const float4*>(row + z.dimp + at);
-          float4 w4 = make_float4(dec, dec, dec, dec);
-          if (WKV) w4 = *reinterpret_cast<const float4*>(row + 2 * z.dimp + at);
+      for (int b = 0; b < RB; ++b) advance(rs + (r + b) * STRIDE, vs + (r + b) * COLS, o[b]);
+      // lanes exchange halves: bit 0 of `sub` keeps one column, bit 1 one row of a pair, bit 2 one pair
+      float x[RB];
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int c = c4 * 4 + e;
-            const float q = reinterpret_cast<const float*>(&q4)[e], k = reinterpret_cast<const float*>(&k4)[e], w = reinterpret_cast<const float*>(&w4)[e];
-            if (WKV) {
-              o0 = fmaf(q, S[0][c], o0);
-              o1 = fmaf(q, S[1][c], o1);
-              S[0][c] = fmaf(w, S[0][c], k * v.x);
-              S[1][c] = fmaf(w, S[1][c], k * v.y);
-            } else {
-              S[0][c] = fmaf(w, S[0][c], k * v.x);
-              S[1][c] = fmaf(w, S[1][c], k * v.y);
-              o0 = fmaf(q, S[0][c], o0);
-              o1 = fmaf(q, S[1][c], o1);
-            }
-          }
+      for (int b = 0; b < RB; ++b) x[b] = (odd ? o[b][1] : o[b][0]) + __shfl_xor_sync(0xffffffffu, odd ? o[b][0] : o[b][1], 1);
+      if (G >= 4) {
+        const bool up = sub & 2;
+#pragma unroll
+        for (int b = 0; b < RB / 2; ++b) x[b] = (up ? x[2 * b + 1] : x[2 * b]) + __shfl_xor_sync(0xffffffffu, up ? x[2 * b] : x[2 * b + 1], 2);
+      }
+      if (G >= 8) {
+        const bool up = sub & 4;
+        x[0] = (up ? x[1] : x[0]) + __shfl_xor_sync(0xffffffffu, up ? x[0] : x[1], 4);
+      }
+#pragma unroll
+      for (int y = 8; y < G; y <<= 1) x[0] += __shfl_xor_sync(0xffffffffu, x[0], y);
+      if (sub < SPREAD && c0 + (sub & 1) < DV) {
+#pragma unroll
+        for (int e = 0; e < KEEP; ++e) {
+          const int b = G >= 8 ? ((sub >> 1) & 1) + 2 * ((sub >> 2) & 1) : G >= 4 ? ((sub >> 1) & 1) + 2 * e : e;
+          float y = x[e];
+          if (WKV) y = fmaf(rs[(r + b) * STRIDE + STRIDE - 4], vs[(r + b) * COLS + (sub & 1)], y);
+          out[(size_t)(r + b) * p.ldo + c0 + (sub & 1)] = y;
         }
-        // even lanes go on with column 0, odd lanes with column 1
-        float o = (odd ? o1 : o0) + __shfl_xor_sync(0xffffffffu, odd ? o0 : o1, 1);
-        for (int x = 2; x < G; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
-        if (WKV) o = fmaf(row[z.stride - 4], odd ? v.y : v.x, o);
-        if (writes) out[(size_t)(tile * SC_ROWS + r) * p.ldo] = o;
+      }
+    }
+#pragma unroll 1
+    for (; r < nr; ++r) {
+      float o[SC_NC];
+      advance(rs + r * STRIDE, vs + r * COLS, o);
+      float y = (odd ? o[1] : o[0]) + __shfl_xor_sync(0xffffffffu, odd ? o[0] : o[1], 1);
+#pragma unroll
+      for (int b = 2; b < G; b <<= 1) y += __shfl_xor_sync(0xffffffffu, y, b);
+      if (sub < 2 && c0 + sub < DV) {
+        if (WKV) y = fmaf(rs[r * STRIDE + STRIDE - 4], vs[r * COLS + sub], y);
+        out[(size_t)r * p.ldo + c0 + sub] = y;
       }
     }
     __syncthreads();  // the stage may be overwritten
@@ -366,21 +431,33 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(const scan_rows<T> p, 
     }
 }
 
-template <typename T, int KC, bool WKV>
-int launch_scan_one(const scan_rows<T>& p, const scan_shape& z, int m, int pos0, cudaStream_t stream) {
+template <int KC, int G, bool WKV>
+int launch_scan_shape(const scan_args& a, const scan_shape& z, int heads, int m, int pos0, cudaStream_t stream) {
   const size_t stage = (size_t)SC_ROWS * (z.stride + z.cols) * sizeof(float);
   const int n_stages = (int)std::min<size_t>(SC_MAX_STAGES, (200 * 1024) / stage);
-  LCU_REQUIRE(z.G <= 32 && n_stages >= 1, "scan: head size %d", p.dim);
   static bool attr_done[16] = {};
   int dev = 0;
   LCU_CUDA(cudaGetDevice(&dev));
   if (dev < 16 && !attr_done[dev]) {
-    LCU_CUDA(cudaFuncSetAttribute((scan_kernel<T, KC, WKV>), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    LCU_CUDA(cudaFuncSetAttribute((scan_kernel<KC, G, WKV>), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     attr_done[dev] = true;
   }
-  LCU_CUDA(launch_after(scan_prepare_kernel<T, WKV>, dim3(m, (p.heads + 3) / 4), dim3(128), 0, stream, p, z, m, pos0));
-  LCU_CUDA(launch_after(scan_kernel<T, KC, WKV>, dim3(p.heads, z.blocks), dim3(SC_THREADS), stage * n_stages, stream, p, z, m, pos0, n_stages));
+  LCU_CUDA(launch_after(scan_kernel<KC, G, WKV>, dim3(heads, z.blocks), dim3(SC_THREADS), stage * n_stages, stream, a, z, m, pos0, n_stages));
   return LCU_OK;
+}
+
+template <bool WKV>
+int launch_scan_kernel(const scan_args& a, const scan_shape& z, int heads, int m, int pos0, cudaStream_t stream) {
+#define LCU_SCAN(KC, GG) if (z.kc == KC && z.G == GG) return launch_scan_shape<KC, GG, WKV>(a, z, heads, m, pos0, stream)
+  LCU_SCAN(4, 2);
+  LCU_SCAN(4, 4);
+  LCU_SCAN(8, 4);
+  LCU_SCAN(8, 8);
+  LCU_SCAN(8, 16);
+  LCU_SCAN(8, 32);
+  LCU_SCAN(16, 32);
+#undef LCU_SCAN
+  LCU_REQUIRE(false, "scan: head size %d", a.dim);
 }
 
 // ------------------------------------------------------------------ one token, all branches
@@ -605,11 +682,11 @@ int launch_window_attention(const attn_rows<T>& p, int m, int pos0, cudaStream_t
 template <typename T>
 int launch_scan(const scan_rows<T>& p, bool wkv, int m, int pos0, cudaStream_t stream) {
   const scan_shape z = scan_shape_of(p.dim, p.vdim, wkv);
-#define LCU_SCAN(KC) return wkv ? launch_scan_one<T, KC, true>(p, z, m, pos0, stream) : launch_scan_one<T, KC, false>(p, z, m, pos0, stream)
-  if (z.kc == 4) LCU_SCAN(4);
-  if (z.kc == 8) LCU_SCAN(8);
-  LCU_SCAN(16);
-#undef LCU_SCAN
+  const dim3 grid((m + SP_ROWS - 1) / SP_ROWS, (p.heads + 7) / 8);
+  if (wkv) LCU_CUDA(launch_after(scan_prepare_kernel<T, true>, grid, dim3(256), 0, stream, p, z, m, pos0));
+  else LCU_CUDA(launch_after(scan_prepare_kernel<T, false>, grid, dim3(256), 0, stream, p, z, m, pos0));
+  const scan_args a{p.packed, p.packed_v, p.decay, p.state, p.out, p.dim, p.vdim, p.ldo, p.err};
+  return wkv ? launch_scan_kernel<true>(a, z, p.heads, m, pos0, stream) : launch_scan_kernel<false>(a, z, p.heads, m, pos0, stream);
 }
 
 void scan_scratch(int heads, int dim, int vdim, bool wkv, size_t rows, size_t* packed_floats, size_t* value_floats) {

@@ -166,34 +166,45 @@ int launch_hyper_one(const hyper_params<T>& p, int n_rows, cudaStream_t stream) 
 }
 
 // ------------------------------------------------------------------ token shift
-// V elements per thread and step (width a multiple of V)
+// A thread keeps V columns (width a multiple of V) and their mu over TS_ROWS rows.
+constexpr int TS_ROWS = 8, TS_MIX = 5;
 template <typename T, int V>
-__global__ void __launch_bounds__(256) token_shift_kernel(const T* h, int ldh, T* prev, const float* mu, T* mix, size_t mix_stride, int n_mix, int m,
-                                                          int width, int pos0) {
-  struct __align__(V * sizeof(T) >= 16 ? 16 : sizeof(T)) pack { T e[V]; };
+__global__ void __launch_bounds__(128) token_shift_kernel(const T* h, int ldh, T* prev, const float* mu, T* mix, size_t mix_stride, int m, int width,
+                                                          int pos0) {
+  struct __align__(V * sizeof(T)) pack { T e[V]; };
   pdl_launch_dependents();
   pdl_wait();
-  const int r = blockIdx.x;
-  for (int c = threadIdx.x * V; c < width; c += 256 * V) {
+  const int c = (blockIdx.x * 128 + threadIdx.x) * V, r0 = blockIdx.y * TS_ROWS, r1 = min(m, r0 + TS_ROWS);
+  if (c >= width) return;
+  float mv[TS_MIX][V];
+#pragma unroll
+  for (int i = 0; i < TS_MIX; ++i)
+#pragma unroll
+    for (int e = 0; e < V; ++e) mv[i][e] = mu[(size_t)i * width + c + e];
+  pack pv;
+  if (r0 > 0) {
+    pv = *reinterpret_cast<const pack*>(h + (size_t)(r0 - 1) * ldh + c);
+  } else {
+    pv = *reinterpret_cast<const pack*>(prev + c);
+    if (pos0 == 0)
+#pragma unroll
+      for (int e = 0; e < V; ++e) pv.e[e] = from_f<T>(0.f);
+    *reinterpret_cast<pack*>(prev + c) = *reinterpret_cast<const pack*>(h + (size_t)(m - 1) * ldh + c);  // (only row 0 touches prev)
+  }
+#pragma unroll 2
+  for (int r = r0; r < r1; ++r) {
     const pack hv = *reinterpret_cast<const pack*>(h + (size_t)r * ldh + c);
-    pack pv;
-    if (r > 0) {
-      pv = *reinterpret_cast<const pack*>(h + (size_t)(r - 1) * ldh + c);
-    } else {
-      pv = *reinterpret_cast<const pack*>(prev + c);
-      if (pos0 == 0)
-        for (int e = 0; e < V; ++e) pv.e[e] = from_f<T>(0.f);
-      *reinterpret_cast<pack*>(prev + c) = *reinterpret_cast<const pack*>(h + (size_t)(m - 1) * ldh + c);  // (only row 0 touches prev)
-    }
-    for (int i = 0; i < n_mix; ++i) {
+#pragma unroll
+    for (int i = 0; i < TS_MIX; ++i) {
       pack o;
 #pragma unroll
       for (int e = 0; e < V; ++e) {
         const float hf = to_f(hv.e[e]);
-        o.e[e] = from_f<T>(fmaf(to_f(pv.e[e]) - hf, mu[(size_t)i * width + c + e], hf));
+        o.e[e] = from_f<T>(fmaf(to_f(pv.e[e]) - hf, mv[i][e], hf));
       }
       *reinterpret_cast<pack*>(mix + i * mix_stride + (size_t)r * ldh + c) = o;
     }
+    pv = hv;
   }
 }
 
@@ -206,7 +217,9 @@ __global__ void rotation_table_kernel(float2* table, int n_pos, int half, double
 }
 
 // ------------------------------------------------------------------ wkv decays
-constexpr int WD_ROWS = 32;
+// A thread forms CH neighbouring channels of WD_ROWS rows (CH 4: whole 16-byte vectors of the matrix).
+constexpr int WD_ROWS = 16;
+template <int CH>
 __global__ void __launch_bounds__(128) wkv_decay_kernel(float* w, size_t head_stride, size_t row_stride, const float* low, int ld_low, const float* w2t,
                                                         const float* w0, int rank, int heads, int dim, int m) {
   extern __shared__ __align__(16) float th[];  // [WD_ROWS][rank rounded up to 4]
@@ -218,80 +231,112 @@ __global__ void __launch_bounds__(128) wkv_decay_kernel(float* w, size_t head_st
     th[i] = r < nr && j < rank ? tanhf(low[(size_t)(r0 + r) * ld_low + j]) : 0.f;
   }
   __syncthreads();
-  const int ch = blockIdx.x * 128 + threadIdx.x;
+  const int ch = (blockIdx.x * 128 + threadIdx.x) * CH;
   if (ch >= channels) return;
-  float acc[WD_ROWS];
-  const float z0 = w0[ch];
+  float acc[WD_ROWS][CH];
 #pragma unroll
-  for (int r = 0; r < WD_ROWS; ++r) acc[r] = z0;
+  for (int r = 0; r < WD_ROWS; ++r)
+#pragma unroll
+    for (int c = 0; c < CH; ++c) acc[r][c] = w0[ch + c];
+#pragma unroll 2
   for (int j = 0; j < rank; j += 4) {
-    float a[4];
+    float a[4][CH];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) a[e] = j + e < rank ? w2t[(size_t)(j + e) * channels + ch] : 0.f;
+    for (int e = 0; e < 4; ++e) {
+      const float* src = w2t + (size_t)(j + e) * channels + ch;
+      if (CH == 4) {
+        const float4 v = j + e < rank ? *reinterpret_cast<const float4*>(src) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int c = 0; c < CH; ++c) a[e][c] = reinterpret_cast<const float*>(&v)[c];
+      } else {
+        a[e][0] = j + e < rank ? src[0] : 0.f;
+      }
+    }
 #pragma unroll
     for (int r = 0; r < WD_ROWS; ++r) {
       const float4 t = *reinterpret_cast<const float4*>(th + r * rp + j);
-      acc[r] = fmaf(a[3], t.w, fmaf(a[2], t.z, fmaf(a[1], t.y, fmaf(a[0], t.x, acc[r]))));
+#pragma unroll
+      for (int c = 0; c < CH; ++c) acc[r][c] = fmaf(a[3][c], t.w, fmaf(a[2][c], t.z, fmaf(a[1][c], t.y, fmaf(a[0][c], t.x, acc[r][c]))));
     }
   }
-  const int head = ch / dim, d = ch - head * dim;
+  const int head = ch / dim, d = ch - head * dim;  // (CH 4: the head size is a multiple of 4)
   float* out = w + head * head_stride + r0 * row_stride + d;
 #pragma unroll
   for (int r = 0; r < WD_ROWS; ++r)
-    if (r < nr) out[r * row_stride] = expf(-expf(acc[r]));
+    if (r < nr) {
+      __align__(16) float y[CH];
+#pragma unroll
+      for (int c = 0; c < CH; ++c) y[c] = expf(-expf(acc[r][c]));
+      if (CH == 4) *reinterpret_cast<float4*>(out + r * row_stride) = *reinterpret_cast<const float4*>(y);
+      else out[r * row_stride] = y[0];
+    }
 }
 
 // ------------------------------------------------------------------ normalised, gated heads (one warp per row and head)
-// VEC 4: head sizes that are multiples of 4 with aligned rows, up to 512; VEC 1: anything
-template <typename T, int VEC>
+// LPH lanes share one (row, head), N vectors of VEC elements each; a group takes HG_ITEMS of them, loads first.  VEC 4: head
+// sizes that are multiples of 4 with aligned rows; VEC 1: anything.
+constexpr int HG_ITEMS = 4;
+template <typename T, int VEC, int LPH, int N>
 __global__ void __launch_bounds__(256) head_gate_kernel(T* out, int ldo, const float* o, int ld_raw, const T* g, int ldg, const float* norm, int heads,
                                                         int vdim, float eps, float out_scale, int m) {
+  constexpr int GROUPS = 256 / LPH, I = N > 1 ? 1 : HG_ITEMS;
   pdl_launch_dependents();
   pdl_wait();
-  const int idx = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (idx >= m * heads) return;
-  const int r = idx / heads, hd = idx - r * heads;
-  constexpr int N = 512 / (32 * VEC);  // vectors per lane
-  const float* x = o + (size_t)r * ld_raw + hd * vdim;
-  const T* gr = g + (size_t)r * ldg + hd * vdim;
-  __align__(16) float xv[N][VEC];
-  __align__(16) T gv[N][VEC];
-  float ss = 0.f;
+  const int grp = threadIdx.x / LPH, sub = threadIdx.x % LPH, total = m * heads;
+  const int first = blockIdx.x * GROUPS * I + grp;
+  __align__(16) float xv[I][N][VEC];
+  __align__(16) T gv[I][N][VEC];
 #pragma unroll
-  for (int n = 0; n < N; ++n) {
-    const int j = (n * 32 + lane) * VEC;
-    if (j < vdim) {
-      if (VEC == 4) {
-        *reinterpret_cast<float4*>(xv[n]) = *reinterpret_cast<const float4*>(x + j);
-        if (sizeof(T) == 2) *reinterpret_cast<uint2*>(gv[n]) = *reinterpret_cast<const uint2*>(gr + j);
-        else *reinterpret_cast<uint4*>(gv[n]) = *reinterpret_cast<const uint4*>(gr + j);
-      } else {
-        xv[n][0] = x[j];
-        gv[n][0] = gr[j];
+  for (int i = 0; i < I; ++i) {
+    const int idx = first + i * GROUPS, r = idx / heads, hd = idx - r * heads;
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      const int j = (n * LPH + sub) * VEC;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) xv[i][n][e] = 0.f;
+      if (idx < total && j < vdim) {
+        const float* x = o + (size_t)r * ld_raw + hd * vdim + j;
+        const T* gr = g + (size_t)r * ldg + hd * vdim + j;
+        if (VEC == 4) {
+          *reinterpret_cast<float4*>(xv[i][n]) = *reinterpret_cast<const float4*>(x);
+          if (sizeof(T) == 2) *reinterpret_cast<uint2*>(gv[i][n]) = *reinterpret_cast<const uint2*>(gr);
+          else *reinterpret_cast<uint4*>(gv[i][n]) = *reinterpret_cast<const uint4*>(gr);
+        } else {
+          xv[i][n][0] = x[0];
+          gv[i][n][0] = gr[0];
+        }
       }
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) ss = fmaf(xv[n][e], xv[n][e], ss);
     }
   }
-  ss = warp_sum(ss);
-  const float inv = 1.0f / sqrtf(ss / (float)vdim + eps);
 #pragma unroll
-  for (int n = 0; n < N; ++n) {
-    const int j = (n * 32 + lane) * VEC;
-    if (j < vdim) {
-      __align__(16) T y[VEC];
+  for (int i = 0; i < I; ++i) {
+    float ss = 0.f;
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) {
-        float v = xv[n][e] * inv;
-        if (norm) v *= norm[hd * vdim + j + e];
-        y[e] = from_f<T>(v * silu_f(to_f(gv[n][e])) * out_scale);
-      }
-      T* dst = out + (size_t)r * ldo + hd * vdim + j;
-      if (VEC == 4) {
-        if (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(y);
-        else *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(y);
-      } else {
-        dst[0] = y[0];
+    for (int n = 0; n < N; ++n)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss = fmaf(xv[i][n][e], xv[i][n][e], ss);
+#pragma unroll
+    for (int x = LPH / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+    const float inv = 1.0f / sqrtf(ss / (float)vdim + eps);
+    const int idx = first + i * GROUPS, r = idx / heads, hd = idx - r * heads;
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      const int j = (n * LPH + sub) * VEC;
+      if (idx < total && j < vdim) {
+        __align__(16) T y[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          float v = xv[i][n][e] * inv;
+          if (norm) v *= norm[hd * vdim + j + e];
+          y[e] = from_f<T>(v * silu_f(to_f(gv[i][n][e])) * out_scale);
+        }
+        T* dst = out + (size_t)r * ldo + hd * vdim + j;
+        if (VEC == 4) {
+          if (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(y);
+          else *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(y);
+        } else {
+          dst[0] = y[0];
+        }
       }
     }
   }
@@ -409,8 +454,10 @@ int launch_hyper_rows(const hyper_params<T>& p, int n_rows, cudaStream_t stream)
 template <typename T>
 int launch_token_shift(const T* h, int ldh, T* prev, const float* mu, T* mix, size_t mix_stride, int n_mix, int m, int width, int pos0,
                        cudaStream_t stream) {
-  if (width % 8 == 0) LCU_CUDA(launch_after(token_shift_kernel<T, 8>, dim3(m), dim3(256), 0, stream, h, ldh, prev, mu, mix, mix_stride, n_mix, m, width, pos0));
-  else LCU_CUDA(launch_after(token_shift_kernel<T, 1>, dim3(m), dim3(256), 0, stream, h, ldh, prev, mu, mix, mix_stride, n_mix, m, width, pos0));
+  LCU_REQUIRE(n_mix == TS_MIX, "token_shift: %d mixes", n_mix);
+  const dim3 grid((width + 511) / 512, (m + TS_ROWS - 1) / TS_ROWS);
+  if (width % 4 == 0) LCU_CUDA(launch_after(token_shift_kernel<T, 4>, grid, dim3(128), 0, stream, h, ldh, prev, mu, mix, mix_stride, m, width, pos0));
+  else LCU_CUDA(launch_after(token_shift_kernel<T, 1>, dim3((width + 127) / 128, grid.y), dim3(128), 0, stream, h, ldh, prev, mu, mix, mix_stride, m, width, pos0));
   return LCU_OK;
 }
 
@@ -425,9 +472,11 @@ int launch_wkv_decay(float* w, size_t head_stride, size_t row_stride, const floa
                      int dim, int m, cudaStream_t stream) {
   const size_t smem = (size_t)WD_ROWS * round_up(rank, 4) * 4;
   LCU_REQUIRE(smem <= 160 * 1024, "wkv_decay: rank %d", rank);
-  if (smem > 48 * 1024) LCU_CUDA(cudaFuncSetAttribute(wkv_decay_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  LCU_CUDA(launch_after(wkv_decay_kernel, dim3((heads * dim + 127) / 128, (m + WD_ROWS - 1) / WD_ROWS), dim3(128), smem, stream, w, head_stride, row_stride, low,
-                        ld_low, w2t, w0, rank, heads, dim, m));
+  const bool vec = dim % 4 == 0 && ((uintptr_t)w & 15) == 0 && ((uintptr_t)w2t & 15) == 0 && head_stride % 4 == 0 && row_stride % 4 == 0;
+  auto kernel = vec ? wkv_decay_kernel<4> : wkv_decay_kernel<1>;
+  if (smem > 48 * 1024) LCU_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  LCU_CUDA(launch_after(kernel, dim3((heads * dim / (vec ? 4 : 1) + 127) / 128, (m + WD_ROWS - 1) / WD_ROWS), dim3(128), smem, stream, w, head_stride,
+                        row_stride, low, ld_low, w2t, w0, rank, heads, dim, m));
   return LCU_OK;
 }
 
@@ -435,11 +484,17 @@ template <typename T>
 int launch_head_gate(T* out, int ldo, const float* o, int ld_raw, const T* g, int ldg, const float* norm, int heads, int vdim, float eps,
                      float out_scale, int m, cudaStream_t stream) {
   LCU_REQUIRE(vdim <= 512, "head_gate: head size %d", vdim);
-  const dim3 grid((unsigned)ceil_div((size_t)m * heads, 8));
   const size_t al = 4 * sizeof(T) - 1;
   const bool vec = vdim % 4 == 0 && ldo % 4 == 0 && ldg % 4 == 0 && ld_raw % 4 == 0 && (((uintptr_t)out | (uintptr_t)g) & al) == 0 && ((uintptr_t)o & 15) == 0;
-  if (vec) LCU_CUDA(launch_after(head_gate_kernel<T, 4>, grid, dim3(256), 0, stream, out, ldo, o, ld_raw, g, ldg, norm, heads, vdim, eps, out_scale, m));
-  else LCU_CUDA(launch_after(head_gate_kernel<T, 1>, grid, dim3(256), 0, stream, out, ldo, o, ld_raw, g, ldg, norm, heads, vdim, eps, out_scale, m));
+  const size_t total = (size_t)m * heads;
+#define LCU_GATE(VEC, LPH, N)                                                                                                                     \
+  LCU_CUDA(launch_after(head_gate_kernel<T, VEC, LPH, N>, dim3((unsigned)ceil_div(total, (256 / LPH) * (N > 1 ? 1 : HG_ITEMS))), dim3(256), 0, stream, \
+                        out, ldo, o, ld_raw, g, ldg, norm, heads, vdim, eps, out_scale, m))
+  if (!vec) LCU_GATE(1, 32, 16);
+  else if (vdim <= 64) LCU_GATE(4, 16, 1);
+  else if (vdim <= 128) LCU_GATE(4, 32, 1);
+  else LCU_GATE(4, 32, 4);
+#undef LCU_GATE
   return LCU_OK;
 }
 
