@@ -1,6 +1,6 @@
 // Attention over a sliding window and pooled blocks for several rows, bfloat16 caches, on warp-level tensor-core tiles.
 //
-// One CTA takes 128 query rows of one head (8 warps of 16 rows) and walks the visible keys in tiles of 64: first the block
+// One CTA takes 64 query rows of one head (4 warps of 16 rows) and walks the visible keys in tiles of 64: first the block
 // means any of its rows sees, then the tokens from the first row's window start to the last row.  Keys and values come in
 // by asynchronous copies into two alternating stages; scores and the running softmax (maximum and sum per row) are
 // binary32, probabilities enter the second product as bfloat16.  Head sizes up to 128; rows of the caches are padded to
@@ -13,7 +13,7 @@
 namespace lcu {
 namespace {
 
-constexpr int WA_Q = 128, WA_K = 64, WA_THREADS = 256;
+constexpr int WA_Q = 64, WA_K = 64, WA_THREADS = 128;
 constexpr float LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ void copy16_or_zero(uint32_t dst, const void* src, bool valid) {
@@ -37,7 +37,7 @@ __device__ __forceinline__ uint32_t pack2(float a, float b) {
 }
 
 template <int HD>
-__global__ void __launch_bounds__(WA_THREADS, HD == 64 ? 2 : 1) window_mma_kernel(const attn_rows<__nv_bfloat16> p, int m, int pos0) {
+__global__ void __launch_bounds__(WA_THREADS, HD == 64 ? 4 : 3) window_mma_kernel(const attn_rows<__nv_bfloat16> p, int m, int pos0) {
   using T = __nv_bfloat16;
   constexpr int LDS = HD + 8, TILE = WA_K * LDS, CPR = HD / 8;
   extern __shared__ __align__(16) T wa_smem[];  // [2 stages][keys | values]

@@ -218,7 +218,7 @@ struct scan_shape {
 };
 scan_shape scan_shape_of(int dim, int vdim, bool wkv) {
   scan_shape s;
-  s.kc = dim <= 16 ? 4 : dim <= 256 ? 8 : 16;
+  s.kc = dim <= 128 ? 4 : dim <= 256 ? 8 : 16;
   s.G = std::max(2, pow2_at_least((dim + s.kc - 1) / s.kc));
   s.dimp = s.G * s.kc;
   s.cols = SC_THREADS / s.G * SC_NC;
@@ -376,13 +376,8 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(const scan_args p, con
     const float* rs = sm + s * STAGE;
     const float* vs = rs + SC_ROWS * STRIDE + grp * SC_NC;
     float* out = p.out + (size_t)tile * SC_ROWS * p.ldo + head * DV;
-    int r = 0;
-#pragma unroll 1
-    for (; r + RB <= nr; r += RB) {
-      float o[RB][SC_NC];
-#pragma unroll
-      for (int b = 0; b < RB; ++b) advance(rs + (r + b) * STRIDE, vs + (r + b) * COLS, o[b]);
-      // lanes exchange halves: bit 0 of `sub` keeps one column, bit 1 one row of a pair, bit 2 one pair
+    // results of RB rows: lanes exchange halves - bit 0 of `sub` keeps one column, bit 1 one row of a pair, bit 2 one pair
+    auto finish = [&](const float (&o)[RB][SC_NC], int r) {
       float x[RB];
 #pragma unroll
       for (int b = 0; b < RB; ++b) x[b] = (odd ? o[b][1] : o[b][0]) + __shfl_xor_sync(0xffffffffu, odd ? o[b][0] : o[b][1], 1);
@@ -406,6 +401,18 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(const scan_args p, con
           out[(size_t)(r + b) * p.ldo + c0 + (sub & 1)] = y;
         }
       }
+    };
+    int r = 0;
+    if (nr == SC_ROWS) {  // whole tiles: the exchange of one row block runs beside the next block's arithmetic
+      float o[2][RB][SC_NC];
+#pragma unroll
+      for (; r < SC_ROWS; r += RB) {
+        const int cur = (r / RB) & 1;
+#pragma unroll
+        for (int b = 0; b < RB; ++b) advance(rs + (r + b) * STRIDE, vs + (r + b) * COLS, o[cur][b]);
+        if (r > 0) finish(o[cur ^ 1], r - RB);
+      }
+      finish(o[(SC_ROWS / RB - 1) & 1], SC_ROWS - RB);
     }
 #pragma unroll 1
     for (; r < nr; ++r) {
@@ -451,9 +458,9 @@ int launch_scan_kernel(const scan_args& a, const scan_shape& z, int heads, int m
 #define LCU_SCAN(KC, GG) if (z.kc == KC && z.G == GG) return launch_scan_shape<KC, GG, WKV>(a, z, heads, m, pos0, stream)
   LCU_SCAN(4, 2);
   LCU_SCAN(4, 4);
-  LCU_SCAN(8, 4);
-  LCU_SCAN(8, 8);
-  LCU_SCAN(8, 16);
+  LCU_SCAN(4, 8);
+  LCU_SCAN(4, 16);
+  LCU_SCAN(4, 32);
   LCU_SCAN(8, 32);
   LCU_SCAN(16, 32);
 #undef LCU_SCAN

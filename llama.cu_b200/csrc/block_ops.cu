@@ -218,7 +218,7 @@ __global__ void rotation_table_kernel(float2* table, int n_pos, int half, double
 
 // ------------------------------------------------------------------ wkv decays
 // A thread forms CH neighbouring channels of WD_ROWS rows (CH 4: whole 16-byte vectors of the matrix).
-constexpr int WD_ROWS = 16;
+constexpr int WD_ROWS = 8;
 template <int CH>
 __global__ void __launch_bounds__(128) wkv_decay_kernel(float* w, size_t head_stride, size_t row_stride, const float* low, int ld_low, const float* w2t,
                                                         const float* w0, int rank, int heads, int dim, int m) {
