@@ -566,6 +566,7 @@ __device__ void step_recurrence(const step_branch<T>& b, int head, int rank, int
     if (ng > 1) {  // groups of threads share the rank
       float a = 0.f;
       if (grp < ng)
+#pragma unroll 8
         for (int j = grp; j < b.rank; j += ng) a = fmaf(b.w2t[(size_t)j * ch_all + head * D + c0], lows[j], a);
       part[tid] = a;
       __syncthreads();
@@ -624,16 +625,56 @@ __device__ void step_recurrence(const step_branch<T>& b, int head, int rank, int
   cluster_sync();
 }
 
+// lines of the caches, states and weights this CTA will read, requested while the kernel before it ends
+template <typename T>
+__device__ __forceinline__ void step_lines(const step_branch<T>& b, int head, int rank, const int* pos_ptr) {
+  const int tid = threadIdx.x;
+  if (b.kind == BRANCH_WINDOW_ATTN) {
+    const attn_rows<T>& p = b.attn;
+    const int pos = min(*(volatile const int*)pos_ptr, p.cache.ctx_len - 1);  // (may be the step before's: only lines are asked for)
+    int lo, blocks;
+    window_of(pos, p.window, p.pool, lo, blocks);
+    const int kvh = head / (p.heads / p.kv_heads), total = blocks + pos + 1 - lo;
+    const int t0 = (int)((long long)total * rank / ST_CLUSTER), n = (int)((long long)total * (rank + 1) / ST_CLUSTER) - t0;
+    constexpr int LINE = 128 / sizeof(T);
+    const int lk = (p.cache.ldk + LINE - 1) / LINE, lv = (p.cache.ldv + LINE - 1) / LINE;
+    for (int i = tid; i < n * (lk + lv); i += MX_THREADS) {
+      const int t = t0 + i / (lk + lv), l = i % (lk + lv);
+      const bool pooled = t < blocks, key = l < lk;
+      const size_t row = pooled ? (size_t)kvh * p.cache.n_blocks + t : (size_t)kvh * p.cache.ctx_len + lo + t - blocks;
+      const T* base = key ? (pooled ? p.cache.kp : p.cache.k) : (pooled ? p.cache.vp : p.cache.v);
+      l2_line(base + row * (key ? p.cache.ldk : p.cache.ldv) + (key ? l : l - lk) * LINE);
+    }
+  } else {
+    const scan_rows<T>& p = b.scan;
+    const int v0 = p.vdim * rank / ST_CLUSTER, nv = p.vdim * (rank + 1) / ST_CLUSTER - v0;
+    if (nv > 0)
+      for (int i = tid; i < p.dim; i += MX_THREADS) l2_line(p.state + ((size_t)head * p.dim + i) * p.vdim + v0);
+    if (b.kind == BRANCH_WKV) {
+      const int per = (p.dim + 31) / 32;
+      for (int i = tid; i < b.rank * per; i += MX_THREADS)
+        l2_line(b.w2t + (size_t)(i / per) * p.heads * p.dim + head * p.dim + min(32 * (i % per), p.dim - 1));
+      if (tid < per) {
+        l2_line(b.w0 + head * p.dim + 32 * tid);
+        l2_line(p.u + head * p.dim + 32 * tid);
+        l2_line(b.norm + head * p.dim + 32 * tid);
+      }
+    }
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(MX_THREADS) mixer_step_kernel(const __grid_constant__ mixer_step<T> p) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[MX_THREADS / 32];
   pdl_launch_dependents();
-  pdl_wait();
   const int cl = blockIdx.x / ST_CLUSTER, rank = blockIdx.x % ST_CLUSTER;
   const int bi = p.n_branches > 1 && cl >= p.b[1].first ? 1 : 0;
   const step_branch<T>& b = p.b[bi];
-  const int head = cl - b.first, pos = *p.pos;
+  const int head = cl - b.first;
+  step_lines(b, head, rank, p.pos);
+  pdl_wait();
+  const int pos = *p.pos;
   if (b.kind == BRANCH_WINDOW_ATTN) step_attention(b, head, rank, pos, sm, red);
   else if (b.kind == BRANCH_RETENTION) step_recurrence<T, false>(b, head, rank, pos, sm, red);
   else step_recurrence<T, true>(b, head, rank, pos, sm, red);

@@ -9,8 +9,10 @@ namespace lcu {
 namespace {
 
 // ------------------------------------------------------------------ embedding
-template <typename T>
-__global__ void __launch_bounds__(256) block_embed_kernel(const embed_params<T> p) {
+// V: elements per thread and step (rows a multiple of V)
+template <typename T, int V>
+__global__ void __launch_bounds__(512) block_embed_kernel(const embed_params<T> p) {
+  struct __align__(V * sizeof(T)) pack { T e[V]; };
   pdl_launch_dependents();
   pdl_wait();
   const int r = blockIdx.x;
@@ -28,15 +30,24 @@ __global__ void __launch_bounds__(256) block_embed_kernel(const embed_params<T> 
   const T* e = p.table + (size_t)tok * p.width;
   const T* b = p.buckets > 0 ? p.bigram + (size_t)s_row * p.width : nullptr;
   float* x = p.xs + (size_t)r * p.streams * p.width;
-  for (int c = threadIdx.x; c < p.width; c += 256) {
-    float v = to_f(e[c]) * p.scale;
-    if (b) v += to_f(b[c]);
-    for (int s = 0; s < p.streams; ++s) x[(size_t)s * p.width + c] = v;
+  for (int c = threadIdx.x * V; c < p.width; c += 512 * V) {
+    const pack ev = *reinterpret_cast<const pack*>(e + c);
+    pack bv = {};
+    if (b) bv = *reinterpret_cast<const pack*>(b + c);
+    __align__(16) float v[V];
+#pragma unroll
+    for (int k = 0; k < V; ++k) v[k] = b ? fmaf(to_f(ev.e[k]), p.scale, to_f(bv.e[k])) : to_f(ev.e[k]) * p.scale;
+    for (int s = 0; s < p.streams; ++s) {
+      float* dst = x + (size_t)s * p.width + c;
+      if (V == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(v);
+      else dst[0] = v[0];
+    }
   }
 }
 
 // ------------------------------------------------------------------ hyper-connected residual + norm
 constexpr int HY_THREADS = 256;
+constexpr int HY_MIX = 5;       // inputs of a token-shifted mixer
 constexpr int HY_CLUSTER = 8;  // CTAs that share one row when there is only one
 
 // SM: room for the streams (p.streams <= SM); CL: CTAs per row
@@ -47,6 +58,14 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int i_row = blockIdx.x / CL, rank = blockIdx.x % CL;
   pdl_launch_dependents();
+  if (CL > 1) {  // a single row: what the columns' last step needs from the weights is on its way while the kernel before ends
+    const int first = min(p.width, rank * per), n = min(p.width, first + per) - first;
+    for (int i = 32 * tid; i < n; i += 32 * HY_THREADS) {
+      l2_line(p.norm_w + first + i);
+      if (p.mix)
+        for (int k = 0; k < p.n_mix; ++k) l2_line(p.mu + (size_t)k * p.width + first + i);
+    }
+  }
   pdl_wait();
   const int row = p.rows ? p.rows[i_row] : i_row;
   const int S = p.streams, W = p.width;
@@ -143,7 +162,11 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
     h[c] = hv;
     if (p.mix) {
       const float hf = to_f(hv), d = (start ? 0.f : to_f(p.prev[c])) - hf;
-      for (int i = 0; i < p.n_mix; ++i) p.mix[i * p.mix_stride + c] = from_f<T>(fmaf(d, p.mu[(size_t)i * W + c], hf));
+      float mu[HY_MIX];
+#pragma unroll
+      for (int i = 0; i < HY_MIX; ++i) mu[i] = p.mu[(size_t)i * W + c];
+#pragma unroll
+      for (int i = 0; i < HY_MIX; ++i) p.mix[i * p.mix_stride + c] = from_f<T>(fmaf(d, mu[i], hf));
       p.prev[c] = hv;
     }
   }
@@ -433,7 +456,8 @@ __global__ void __launch_bounds__(256) matmul_f32_tile_kernel(float* out, const 
 
 template <typename T>
 int launch_block_embed(const embed_params<T>& p, cudaStream_t stream) {
-  LCU_CUDA(launch_after(block_embed_kernel<T>, dim3(p.m), dim3(256), 0, stream, p));
+  if (p.width % 4 == 0) LCU_CUDA(launch_after(block_embed_kernel<T, 4>, dim3(p.m), dim3(512), 0, stream, p));
+  else LCU_CUDA(launch_after(block_embed_kernel<T, 1>, dim3(p.m), dim3(512), 0, stream, p));
   return LCU_OK;
 }
 
@@ -441,7 +465,7 @@ template <typename T>
 int launch_hyper_rows(const hyper_params<T>& p, int n_rows, cudaStream_t stream) {
   if (n_rows < 1) return LCU_OK;
   LCU_REQUIRE(p.streams >= 1 && p.streams <= 8, "hyper_rows: %d streams", p.streams);
-  LCU_REQUIRE(p.mix == nullptr || n_rows == 1, "hyper_rows: the token shift is fused for a single row only");
+  LCU_REQUIRE(p.mix == nullptr || (n_rows == 1 && p.n_mix == HY_MIX), "hyper_rows: the token shift is fused for a single row of %d inputs", HY_MIX);
 #define LCU_HYPER(SM) \
   return n_rows == 1 ? launch_hyper_one<T, SM, HY_CLUSTER>(p, n_rows, stream) : launch_hyper_one<T, SM, 1>(p, n_rows, stream)
   if (p.streams == 1) LCU_HYPER(1);

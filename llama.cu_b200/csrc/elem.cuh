@@ -17,6 +17,10 @@ __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return
 
 __host__ __device__ __forceinline__ int round_up_dev(int a, int b) { return (a + b - 1) / b * b; }
 
+// asks for the line of an address in L2 (no register, nothing to wait for); may run ahead of the kernel before this one,
+// whatever that kernel still writes: only the line is fetched, the value is read later
+__device__ __forceinline__ void l2_line(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 
 // launch of a kernel whose CTAs work in clusters of `cluster` (1: plain), as a programmatic dependent of the kernel before it
