@@ -3,8 +3,9 @@
 // One CTA takes 64 query rows of one head (4 warps of 16 rows) and walks the visible keys in tiles of 64: first the block
 // means any of its rows sees, then the tokens from the first row's window start to the last row.  Keys and values come in
 // by asynchronous copies into two alternating stages; scores and the running softmax (maximum and sum per row) are
-// binary32, probabilities enter the second product as bfloat16.  Head sizes up to 128; rows of the caches are padded to
-// multiples of 8 with zeros, smaller heads are zero-filled to the tile width in shared memory.
+// binary32, probabilities enter the second product as bfloat16.  Keys may come in two parts (a head's own and one that all
+// heads share); up to 256 key and 128 value columns.  Rows in memory are padded to multiples of 8 with zeros, smaller heads
+// are zero-filled to the tile width in shared memory.
 #include <math_constants.h>
 
 #include "block_ops.cuh"
@@ -36,18 +37,22 @@ __device__ __forceinline__ uint32_t pack2(float a, float b) {
   return *reinterpret_cast<const uint32_t*>(&h);
 }
 
-template <int HD>
-__global__ void __launch_bounds__(WA_THREADS, HD == 64 ? 4 : 3) window_mma_kernel(const attn_rows<__nv_bfloat16> p, int m, int pos0) {
+// HK, HV: columns of the key (both parts) and value tiles
+template <int HK, int HV>
+__global__ void __launch_bounds__(WA_THREADS, HK == 64 ? 4 : HK == 128 ? 3 : 2) window_mma_kernel(const attn_rows<__nv_bfloat16> p, int m, int pos0) {
   using T = __nv_bfloat16;
-  constexpr int LDS = HD + 8, TILE = WA_K * LDS, CPR = HD / 8;
+  constexpr int LDK = HK + 8, LDV = HV + 8, STAGE = WA_K * (LDK + LDV), CK = HK / 8, CV = HV / 8;
   extern __shared__ __align__(16) T wa_smem[];  // [2 stages][keys | values]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c = lane & 3;
   // row tiles in descending order (the last ones see the most keys), heads of a key/value group next to each other
   const int head = blockIdx.x, q0 = (gridDim.y - 1 - blockIdx.y) * WA_Q;
   const int kvh = head / (p.heads / p.kv_heads);
   const int ldk = p.cache.ldk, ldv = p.cache.ldv;
-  const T* kc = p.cache.k + (size_t)kvh * p.cache.ctx_len * ldk;
-  const T* vc = p.cache.v + (size_t)kvh * p.cache.ctx_len * ldv;
+  const T* kc = p.cache.k + kvh * p.cache.k_head;
+  const T* vc = p.cache.v + kvh * p.cache.v_head;
+  // columns of a staged row: the first key part (padded to 8), the second, zeros
+  const int k_cols = (p.dim + 7) / 8 * 8, v_cols = (p.vdim + 7) / 8 * 8, k2_end = k_cols + (p.key2 ? (p.dim2 + 7) / 8 * 8 : 0);
+  const int q_cols = p.key2 ? k2_end : p.dim;
   const T* kp = p.cache.kp + (size_t)kvh * p.cache.n_blocks * ldk;
   const T* vp = p.cache.vp + (size_t)kvh * p.cache.n_blocks * ldv;
   pdl_launch_dependents();
@@ -64,18 +69,18 @@ __global__ void __launch_bounds__(WA_THREADS, HD == 64 ? 4 : 3) window_mma_kerne
 
   // query fragments (16 rows x HD per warp): rows g and g + 8
   const int r_lo = q0 + warp * 16 + g, r_hi = r_lo + 8;
-  uint32_t qa[HD / 16][4];
+  uint32_t qa[HK / 16][4];
   {
     auto pair = [&](int r, int d) {
-      const T* q = p.q + (size_t)r * p.ld + head * p.dim + d;
+      const T* q = p.q + (size_t)r * p.ld + head * p.q_head + d;
       const T zero = __float2bfloat16(0.f);
       __nv_bfloat162 h;
-      h.x = r < m && d < p.dim ? q[0] : zero;
-      h.y = r < m && d + 1 < p.dim ? q[1] : zero;
+      h.x = r < m && d < q_cols ? q[0] : zero;
+      h.y = r < m && d + 1 < q_cols ? q[1] : zero;
       return *reinterpret_cast<const uint32_t*>(&h);
     };
 #pragma unroll
-    for (int ks = 0; ks < HD / 16; ++ks) {
+    for (int ks = 0; ks < HK / 16; ++ks) {
       const int d = ks * 16 + 2 * c;
       qa[ks][0] = pair(r_lo, d);
       qa[ks][1] = pair(r_hi, d);
@@ -89,25 +94,33 @@ __global__ void __launch_bounds__(WA_THREADS, HD == 64 ? 4 : 3) window_mma_kerne
   const int warp_first = pos0 + q0 + warp * 16, warp_last = warp_first + 15;
 
   auto stage_tile = [&](int tile, int stage) {
-    T* ks = wa_smem + (size_t)stage * 2 * TILE;
-    T* vs = ks + TILE;
+    T* ks = wa_smem + (size_t)stage * STAGE;
+    T* vs = ks + WA_K * LDK;
     const bool pooled = tile < pool_tiles;
     const int t0 = pooled ? tile * WA_K : lo + (tile - pool_tiles) * WA_K, end = pooled ? n_blocks : last_pos + 1;
     const T *kb = pooled ? kp : kc, *vb = pooled ? vp : vc;
-    for (int i = tid; i < WA_K * CPR; i += WA_THREADS) {
-      const int r = i / CPR, ch = (i % CPR) * 8;
+    const int shift = pooled ? 0 : p.cache.first;
+    for (int i = tid; i < WA_K * CK; i += WA_THREADS) {
+      const int r = i / CK, ch = (i % CK) * 8;
       const bool live = t0 + r < end;
-      const size_t row = live ? t0 + r : 0;
-      const bool kv = live && ch < ldk, vv = live && ch < ldv;
-      copy16_or_zero(smem_u32(ks + r * LDS + ch), kv ? kb + row * ldk + ch : kb, kv);
-      copy16_or_zero(smem_u32(vs + r * LDS + ch), vv ? vb + row * ldv + ch : vb, vv);
+      const size_t row = live ? t0 + r - shift : 0;
+      const bool second = ch >= k_cols, kv = live && ch < k2_end;
+      const T* src = !kv ? kb : second ? p.key2 + (size_t)(t0 + r - p.first2) * p.ld2 + ch - k_cols : kb + row * ldk + ch;
+      copy16_or_zero(smem_u32(ks + r * LDK + ch), src, kv);
+    }
+    for (int i = tid; i < WA_K * CV; i += WA_THREADS) {
+      const int r = i / CV, ch = (i % CV) * 8;
+      const bool live = t0 + r < end;
+      const size_t row = live ? t0 + r - shift : 0;
+      const bool vv = live && ch < v_cols;
+      copy16_or_zero(smem_u32(vs + r * LDV + ch), vv ? vb + row * ldv + ch : vb, vv);
     }
     cp_async_commit();
   };
 
-  float o[HD / 8][4];
+  float o[HV / 8][4];
 #pragma unroll
-  for (int j = 0; j < HD / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  for (int j = 0; j < HV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
   float mx_lo = -CUDART_INF_F, mx_hi = -CUDART_INF_F, sum_lo = 0.f, sum_hi = 0.f;
   const float scale2 = p.scale * LOG2E;
 
@@ -125,17 +138,17 @@ __global__ void __launch_bounds__(WA_THREADS, HD == 64 ? 4 : 3) window_mma_kerne
     // nothing of the tile is visible to this warp's rows
     const bool skip = pooled ? t0 >= blocks_of(warp_last) : (t0 > warp_last || t0 + WA_K - 1 < warp_first + 1 - p.window);
     if (!skip) {
-      const T* ks = wa_smem + (size_t)(tile & 1) * 2 * TILE;
-      const T* vs = ks + TILE;
+      const T* ks = wa_smem + (size_t)(tile & 1) * STAGE;
+      const T* vs = ks + WA_K * LDK;
       float s[8][4];
 #pragma unroll
       for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
 #pragma unroll
-      for (int kk = 0; kk < HD / 16; kk += 2) {
+      for (int kk = 0; kk < HK / 16; kk += 2) {
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           uint32_t b0, b1, b2, b3;
-          ldsm_x4(smem_u32(ks + (j * 8 + (lane & 7)) * LDS + kk * 16 + (lane >> 3) * 8), b0, b1, b2, b3);
+          ldsm_x4(smem_u32(ks + (j * 8 + (lane & 7)) * LDK + kk * 16 + (lane >> 3) * 8), b0, b1, b2, b3);
           mma_16816_bf16(s[j], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], b0, b1);
           mma_16816_bf16(s[j], qa[kk + 1][0], qa[kk + 1][1], qa[kk + 1][2], qa[kk + 1][3], b2, b3);
         }
@@ -190,7 +203,7 @@ __global__ void __launch_bounds__(WA_THREADS, HD == 64 ? 4 : 3) window_mma_kerne
       sum_lo = sum_lo * f_lo + ts_lo;  // (this lane's keys; the lanes of a row are added at the end)
       sum_hi = sum_hi * f_hi + ts_hi;
 #pragma unroll
-      for (int j = 0; j < HD / 8; ++j) {
+      for (int j = 0; j < HV / 8; ++j) {
         o[j][0] *= f_lo;
         o[j][1] *= f_lo;
         o[j][2] *= f_hi;
@@ -199,11 +212,11 @@ __global__ void __launch_bounds__(WA_THREADS, HD == 64 ? 4 : 3) window_mma_kerne
 #pragma unroll
       for (int kk = 0; kk < 4; ++kk) {
 #pragma unroll
-        for (int dj = 0; dj < HD / 16; ++dj) {
+        for (int dj = 0; dj < HV / 16; ++dj) {
           const int mrow = kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
           const int mcol = dj * 16 + (lane >> 4) * 8;
           uint32_t b0, b1, b2, b3;
-          ldsm_x4_trans(smem_u32(vs + mrow * LDS + mcol), b0, b1, b2, b3);
+          ldsm_x4_trans(smem_u32(vs + mrow * LDV + mcol), b0, b1, b2, b3);
           mma_16816_bf16(o[2 * dj], pa[kk][0], pa[kk][1], pa[kk][2], pa[kk][3], b0, b1);
           mma_16816_bf16(o[2 * dj + 1], pa[kk][0], pa[kk][1], pa[kk][2], pa[kk][3], b2, b3);
         }
@@ -215,9 +228,22 @@ __global__ void __launch_bounds__(WA_THREADS, HD == 64 ? 4 : 3) window_mma_kerne
   sum_lo += __shfl_xor_sync(0xffffffffu, sum_lo, 2);
   sum_hi += __shfl_xor_sync(0xffffffffu, sum_hi, 1);
   sum_hi += __shfl_xor_sync(0xffffffffu, sum_hi, 2);
-  const float inv_lo = p.out_scale / sum_lo, inv_hi = p.out_scale / sum_hi;
+  float inv_lo = p.out_scale / sum_lo, inv_hi = p.out_scale / sum_hi;
+  if (p.sink) {  // one more term of the denominator, against the larger of it and the row's maximum
+    const float s2 = p.sink[head] * LOG2E;
+    auto with_sink = [&](float mx, float sum) {
+      const float top = fmaxf(mx, s2), f = ex2(mx - top);
+      return p.out_scale * f / (sum * f + ex2(s2 - top));
+    };
+    inv_lo = with_sink(mx_lo, sum_lo);
+    inv_hi = with_sink(mx_hi, sum_hi);
+  }
+  if (p.gate) {
+    if (r_lo < m) inv_lo *= sigmoid_f(to_f(p.gate[(size_t)r_lo * p.ldg + head]));
+    if (r_hi < m) inv_hi *= sigmoid_f(to_f(p.gate[(size_t)r_hi * p.ldg + head]));
+  }
 #pragma unroll
-  for (int j = 0; j < HD / 8; ++j) {
+  for (int j = 0; j < HV / 8; ++j) {
     const int d = j * 8 + 2 * c;
     if (d >= p.vdim) continue;
     T* a = p.out + (size_t)r_lo * p.ldo + head * p.vdim + d;
@@ -234,28 +260,31 @@ __global__ void __launch_bounds__(WA_THREADS, HD == 64 ? 4 : 3) window_mma_kerne
   }
 }
 
-template <int HD>
+template <int HK, int HV>
 int launch_hd(const attn_rows<__nv_bfloat16>& p, int m, int pos0, cudaStream_t stream) {
-  const size_t smem = (size_t)2 * 2 * WA_K * (HD + 8) * 2;
+  const size_t smem = (size_t)2 * WA_K * (HK + HV + 16) * 2;
   static bool attr_done[16] = {};
   int dev = 0;
   LCU_CUDA(cudaGetDevice(&dev));
   if (dev < 16 && !attr_done[dev]) {
-    LCU_CUDA(cudaFuncSetAttribute(window_mma_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    LCU_CUDA(cudaFuncSetAttribute((window_mma_kernel<HK, HV>), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     attr_done[dev] = true;
   }
-  LCU_CUDA(launch_after(window_mma_kernel<HD>, dim3(p.heads, (m + WA_Q - 1) / WA_Q), dim3(WA_THREADS), smem, stream, p, m, pos0));
+  LCU_CUDA(launch_after(window_mma_kernel<HK, HV>, dim3(p.heads, (m + WA_Q - 1) / WA_Q), dim3(WA_THREADS), smem, stream, p, m, pos0));
   return LCU_OK;
 }
 
 }  // namespace
 
-bool window_mma_supported(int dim, int vdim) { return dim <= 128 && vdim <= 128; }
+bool window_mma_supported(int dim, int dim2, int vdim) { return round_up(dim, 8) + round_up(dim2, 8) <= 256 && vdim <= 128; }
 
 int launch_window_mma(const attn_rows<__nv_bfloat16>& p, int m, int pos0, cudaStream_t stream) {
-  LCU_REQUIRE(window_mma_supported(p.dim, p.vdim), "window attention: head size %d x %d", p.dim, p.vdim);
-  if (p.dim <= 64 && p.vdim <= 64) return launch_hd<64>(p, m, pos0, stream);
-  return launch_hd<128>(p, m, pos0, stream);
+  const int dim2 = p.key2 ? p.dim2 : 0, hk = (int)(round_up(p.dim, 8) + round_up(dim2, 8));
+  LCU_REQUIRE(window_mma_supported(p.dim, dim2, p.vdim), "window attention: head size %d + %d x %d", p.dim, dim2, p.vdim);
+  if (hk <= 64 && p.vdim <= 64) return launch_hd<64, 64>(p, m, pos0, stream);
+  if (hk <= 128) return launch_hd<128, 128>(p, m, pos0, stream);
+  if (hk <= 192) return launch_hd<192, 128>(p, m, pos0, stream);
+  return launch_hd<256, 128>(p, m, pos0, stream);
 }
 
 }  // namespace lcu

@@ -48,9 +48,13 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 }
 
 // ------------------------------------------------------------------ attention of one query row and head
+template <typename T>
+__host__ __device__ __forceinline__ int query_cols(const attn_rows<T>& p) {
+  return (p.dim + 7) / 8 * 8 + (p.key2 ? (p.dim2 + 7) / 8 * 8 : 0);
+}
 // `rank` of `C` CTAs takes a slice of the visible keys.  The row's own key and value come from `cur_k` / `cur_v` (shared
-// memory copies) when given, else from the cache.  Leaves max, sum and the unnormalised value row in res[0], res[1],
-// res[2 ..].  Shared memory: q [ldk], scores [slice], part [PART_FLOATS].
+// memory copies) when given, else from the cache.  q_row null: q holds the query already.  Leaves max, sum and the
+// unnormalised value row in res[0], res[1], res[2 ..].  Shared memory: q [query_cols], scores [slice], part [PART_FLOATS].
 template <typename T>
 __device__ void attend_slice(const attn_rows<T>& p, const T* q_row, int head, int pos, int rank, int C, const T* cur_k, const T* cur_v, float* q,
                              float* sc, float* part, float* red, float* res) {
@@ -58,29 +62,31 @@ __device__ void attend_slice(const attn_rows<T>& p, const T* q_row, int head, in
   const int tid = threadIdx.x;
   const int kvh = head / (p.heads / p.kv_heads);
   const int ldk = p.cache.ldk, ldv = p.cache.ldv;
-  const T* kc = p.cache.k + (size_t)kvh * p.cache.ctx_len * ldk;
-  const T* vc = p.cache.v + (size_t)kvh * p.cache.ctx_len * ldv;
+  const int k_cols = (p.dim + 7) / 8 * 8, v_cols = (p.vdim + 7) / 8 * 8, q_cols = query_cols(p);
+  const T* kc = p.cache.k + kvh * p.cache.k_head;
+  const T* vc = p.cache.v + kvh * p.cache.v_head;
   const T* kp = p.cache.kp + (size_t)kvh * p.cache.n_blocks * ldk;
   const T* vp = p.cache.vp + (size_t)kvh * p.cache.n_blocks * ldv;
   int lo, blocks;
   window_of(pos, p.window, p.pool, lo, blocks);
   const int total = blocks + pos + 1 - lo;
   const int t0 = (int)((long long)total * rank / C), n = (int)((long long)total * (rank + 1) / C) - t0;
-  for (int d = tid; d < ldk; d += MX_THREADS) q[d] = d < p.dim ? to_f(q_row[head * p.dim + d]) : 0.f;
+  if (q_row)
+    for (int d = tid; d < q_cols; d += MX_THREADS) q[d] = d < p.dim || p.key2 ? to_f(q_row[head * p.q_head + d]) : 0.f;
   __syncthreads();
   auto key_at = [&](int t) -> const T* {
     if (t < blocks) return kp + (size_t)t * ldk;
     const int j = lo + t - blocks;
-    return cur_k && j == pos ? cur_k : kc + (size_t)j * ldk;
+    return cur_k && j == pos ? cur_k : kc + (size_t)(j - p.cache.first) * ldk;
   };
   auto value_at = [&](int t) -> const T* {
     if (t < blocks) return vp + (size_t)t * ldv;
     const int j = lo + t - blocks;
-    return cur_v && j == pos ? cur_v : vc + (size_t)j * ldv;
+    return cur_v && j == pos ? cur_v : vc + (size_t)(j - p.cache.first) * ldv;
   };
   // scores: lpk lanes per key
   {
-    const int lpk = min(32, pow2_at_least((ldk + VEC - 1) / VEC)), groups = MX_THREADS / lpk, grp = tid / lpk, sub = tid % lpk;
+    const int lpk = min(32, pow2_at_least((k_cols + VEC - 1) / VEC)), groups = MX_THREADS / lpk, grp = tid / lpk, sub = tid % lpk;
     constexpr int U = 4;
     const int rounds = (n + groups * U - 1) / (groups * U);  // (the same for every lane: the shuffles below are warp-wide)
     for (int rd = 0; rd < rounds; ++rd) {
@@ -91,10 +97,18 @@ __device__ void attend_slice(const attn_rows<T>& p, const T* q_row, int head, in
         const int t = (rd * U + u) * groups + grp;
         if (t < n) {
           const T* k = key_at(t0 + t);
-          for (int d = sub * VEC; d < ldk; d += lpk * VEC) {
+          for (int d = sub * VEC; d < k_cols; d += lpk * VEC) {
             const uint4 raw = *reinterpret_cast<const uint4*>(k + d);
 #pragma unroll
             for (int e = 0; e < VEC; ++e) s[u] = fmaf(q[d + e], to_f(reinterpret_cast<const T*>(&raw)[e]), s[u]);
+          }
+          if (p.key2) {
+            const T* k2 = p.key2 + (size_t)(lo + t0 + t - blocks - p.first2) * p.ld2 - k_cols;
+            for (int d = k_cols + sub * VEC; d < q_cols; d += lpk * VEC) {
+              const uint4 raw = *reinterpret_cast<const uint4*>(k2 + d);
+#pragma unroll
+              for (int e = 0; e < VEC; ++e) s[u] = fmaf(q[d + e], to_f(reinterpret_cast<const T*>(&raw)[e]), s[u]);
+            }
           }
         }
       }
@@ -118,11 +132,11 @@ __device__ void attend_slice(const attn_rows<T>& p, const T* q_row, int head, in
   }
   sum = block_sum(sum, red);  // (its barriers also publish the exponentials)
   // values: lpv lanes per row of values, groups of them walk the keys
-  const int lpv = min(32, pow2_at_least((ldv + VEC - 1) / VEC)), groups = MX_THREADS / lpv, grp = tid / lpv, sub = tid % lpv;
-  for (int d0 = 0; d0 < ldv; d0 += lpv * VEC) {
+  const int lpv = min(32, pow2_at_least((v_cols + VEC - 1) / VEC)), groups = MX_THREADS / lpv, grp = tid / lpv, sub = tid % lpv;
+  for (int d0 = 0; d0 < v_cols; d0 += lpv * VEC) {
     const int d = d0 + sub * VEC;
     float acc[VEC] = {};
-    if (d < ldv) {
+    if (d < v_cols) {
 #pragma unroll 4
       for (int t = grp; t < n; t += groups) {
         const uint4 raw = *reinterpret_cast<const uint4*>(value_at(t0 + t) + d);
@@ -157,11 +171,16 @@ __global__ void __launch_bounds__(MX_THREADS) window_rows_kernel(const attn_rows
   pdl_wait();
   const int head = blockIdx.x, r = blockIdx.y;
   float* q = sm;
-  float* part = q + p.cache.ldk;
+  float* part = q + query_cols(p);
   float* res = part + PART_FLOATS;
   float* sc = res + 2 + round_up_dev(p.vdim + 2, 4);
   attend_slice(p, p.q + (size_t)r * p.ld, head, pos0 + r, 0, 1, (const T*)nullptr, (const T*)nullptr, q, sc, part, red, res);
-  const float inv = p.out_scale / res[1];
+  float inv = p.out_scale / res[1];
+  if (p.sink) {
+    const float top = fmaxf(res[0], p.sink[head]), f = expf(res[0] - top);
+    inv = p.out_scale * f / (res[1] * f + expf(p.sink[head] - top));
+  }
+  if (p.gate) inv *= sigmoid_f(to_f(p.gate[(size_t)r * p.ldg + head]));
   for (int d = threadIdx.x; d < p.vdim; d += MX_THREADS) p.out[(size_t)r * p.ldo + head * p.vdim + d] = from_f<T>(res[2 + d] * inv);
 }
 
@@ -518,7 +537,12 @@ __device__ void step_attention(const step_branch<T>& b, int head, int rank, int 
     f[r] = m > -CUDART_INF_F ? expf(m - mx) : 0.f;
     if (f[r] > 0.f) sum += f[r] * ld_dsmem_f32(mapa(smem_u32(res + 1), r));
   }
-  const float inv = p.out_scale / sum;
+  float inv = p.out_scale / sum;
+  if (p.sink) {
+    const float top = fmaxf(mx, p.sink[head]), g = expf(mx - top);
+    inv = p.out_scale * g / (sum * g + expf(p.sink[head] - top));
+  }
+  if (p.gate) inv *= sigmoid_f(to_f(p.gate[head]));
   const int d1 = p.vdim * (rank + 1) / ST_CLUSTER;
   for (int d = p.vdim * rank / ST_CLUSTER + tid; d < d1; d += MX_THREADS) {
     float v = 0.f;
@@ -526,6 +550,130 @@ __device__ void step_attention(const step_branch<T>& b, int head, int rank, int 
     for (int r = 0; r < ST_CLUSTER; ++r)
       if (f[r] > 0.f) v += f[r] * ld_dsmem_f32(mapa(smem_u32(res + 2 + d), r));
     b.out[head * p.vdim + d] = from_f<T>(v * inv);
+  }
+  cluster_sync();
+}
+
+// Latent attention of one token and head without forming keys or values: the query is taken through the head's key matrix
+// once (the CTAs share its columns), so that a key is a cache row and the result a sum of cache rows, which the head's value
+// matrix turns into the output (the CTAs share its rows).  All of it in binary32 but for the cache rows.
+template <typename T>
+size_t latent_step_floats(const latent_rows<T>& p) {
+  return 3 * (size_t)p.cache.ld + round_up(p.dim, 8) + p.cache.rot + 2 + round_up(p.kv_rank + 2, 4) + PART_FLOATS;
+}
+template <typename T>
+__device__ void step_latent(const step_branch<T>& b, int head, int rank, int pos, float* sm, float* red) {
+  const latent_rows<T>& p = b.latent;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int ld = p.cache.ld, rp = p.cache.rot, kp = round_up_dev(p.dim, 8), rotp = ld - rp, vp = round_up_dev(p.vdim, 8), half = p.rot_dims >> 1;
+  struct __align__(16) vec8 { T e[8]; };
+  T* cur = reinterpret_cast<T*>(sm);  // [ld] the token's row as the cache will hold it
+  float* q = sm + ld;                 // [ld] query against cache rows
+  float* oc = q + ld;                 // [rp] sum of cache rows
+  float* qh = oc + rp;                // [kp] query against the head's unrotated keys
+  float* part = qh + kp;
+  float* res = part + PART_FLOATS;
+  float* sc = res + 2 + round_up_dev(p.kv_rank + 2, 4);
+  const T* q_row = p.q + (size_t)head * (kp + rotp);
+  float ss = 0.f;
+  for (int d = tid; d < rp; d += MX_THREADS) {
+    const float x = d < p.kv_rank ? to_f(p.c[d]) : 0.f;
+    oc[d] = x;
+    ss = fmaf(x, x, ss);
+  }
+  for (int d = tid; d < kp; d += MX_THREADS) qh[d] = to_f(q_row[d]);
+  for (int d = tid; d < rotp; d += MX_THREADS) {
+    float kv = d < p.rot_dim ? to_f(p.k[d]) : 0.f, qv = to_f(q_row[kp + d]);
+    if (d < p.rot_dims) {
+      const float2 cs = p.rope[(size_t)pos * half + (d >> 1)];
+      const float sn = d & 1 ? cs.y : -cs.y;
+      kv = kv * cs.x + to_f(p.k[d ^ 1]) * sn;
+      qv = qv * cs.x + to_f(q_row[kp + (d ^ 1)]) * sn;
+    }
+    cur[rp + d] = from_f<T>(kv);
+    q[rp + d] = qv;
+  }
+  ss = block_sum(ss, red);
+  const float inv_c = 1.0f / sqrtf(ss / (float)p.kv_rank + p.eps);
+  for (int d = tid; d < rp; d += MX_THREADS) cur[d] = from_f<T>(d < p.kv_rank ? oc[d] * inv_c * p.norm[d] : 0.f);
+  __syncthreads();
+  if (head == 0 && rank == 0)
+    for (int d = tid; d < ld; d += MX_THREADS) p.cache.rows[(size_t)pos * ld + d] = cur[d];
+  // this CTA's columns of the query against latents, in vectors of 8
+  const int vecs = rp >> 3, v0 = vecs * rank / ST_CLUSTER, nv = vecs * (rank + 1) / ST_CLUSTER - v0;
+  if (nv > 0) {
+    const int ng = min(MX_THREADS / nv, 32), grp = tid / nv, j = tid - grp * nv;
+    if (grp < ng) {
+      float acc[8] = {};
+      const T* w = b.up + (size_t)head * kp * b.ld_up + (v0 + j) * 8;
+#pragma unroll 4
+      for (int d = grp; d < p.dim; d += ng) {
+        const vec8 x = *reinterpret_cast<const vec8*>(w + (size_t)d * b.ld_up);
+        const float qd = qh[d];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] = fmaf(qd, to_f(x.e[e]), acc[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) part[(grp * nv + j) * 8 + e] = acc[e];
+    }
+    __syncthreads();
+    for (int i = tid; i < nv * 8; i += MX_THREADS) {
+      float a = 0.f;
+      for (int g = 0; g < ng; ++g) a += part[g * nv * 8 + i];
+      q[v0 * 8 + i] = a;
+    }
+  }
+  cluster_sync();
+  for (int i = tid; i < rp; i += MX_THREADS) {
+    const int owner = ((i >> 3) * ST_CLUSTER + ST_CLUSTER - 1) / vecs;  // whose vectors hold column i
+    if (owner != rank) q[i] = ld_dsmem_f32(mapa(smem_u32(q + i), owner));
+  }
+  attn_rows<T> a{};
+  a.cache.k = a.cache.v = p.cache.rows;
+  a.cache.ldk = a.cache.ldv = ld;
+  a.heads = a.kv_heads = 1;
+  a.dim = ld;
+  a.vdim = p.kv_rank;
+  a.window = p.window;
+  a.scale = b.attn.scale;
+  attend_slice(a, (const T*)nullptr, 0, pos, rank, ST_CLUSTER, cur, cur, q, sc, part, red, res);
+  cluster_sync();
+  float mx = b.attn.sink ? b.attn.sink[head] : -CUDART_INF_F, sum = 0.f, f[ST_CLUSTER];
+#pragma unroll
+  for (int r = 0; r < ST_CLUSTER; ++r) {
+    f[r] = ld_dsmem_f32(mapa(smem_u32(res), r));
+    mx = fmaxf(mx, f[r]);
+  }
+#pragma unroll
+  for (int r = 0; r < ST_CLUSTER; ++r) {
+    f[r] = f[r] > -CUDART_INF_F ? expf(f[r] - mx) : 0.f;
+    sum = fmaf(f[r], ld_dsmem_f32(mapa(smem_u32(res + 1), r)), sum);
+  }
+  if (b.attn.sink) sum += expf(b.attn.sink[head] - mx);
+  float out_scale = b.attn.out_scale / sum;
+  if (b.attn.gate) out_scale *= sigmoid_f(to_f(b.attn.gate[head]));
+  for (int d = tid; d < rp; d += MX_THREADS) {
+    float v = 0.f;
+    if (d < p.kv_rank) {
+#pragma unroll
+      for (int r = 0; r < ST_CLUSTER; ++r)
+        if (f[r] > 0.f) v = fmaf(f[r], ld_dsmem_f32(mapa(smem_u32(res + 2 + d), r)), v);
+    }
+    oc[d] = v;
+  }
+  __syncthreads();
+  const int j1 = p.vdim * (rank + 1) / ST_CLUSTER;
+  for (int j = p.vdim * rank / ST_CLUSTER + warp; j < j1; j += MX_THREADS / 32) {
+    const T* w = b.up + ((size_t)b.up_v + (size_t)head * vp + j) * b.ld_up;
+    float v = 0.f;
+#pragma unroll 2
+    for (int d = lane * 8; d < rp; d += 256) {
+      const vec8 x = *reinterpret_cast<const vec8*>(w + d);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v = fmaf(oc[d + e], to_f(x.e[e]), v);
+    }
+    v = warp_sum(v);
+    if (lane == 0) b.out[head * p.vdim + j] = from_f<T>(v * out_scale);
   }
   cluster_sync();
 }
@@ -645,6 +793,23 @@ __device__ __forceinline__ void step_lines(const step_branch<T>& b, int head, in
       const T* base = key ? (pooled ? p.cache.kp : p.cache.k) : (pooled ? p.cache.vp : p.cache.v);
       l2_line(base + row * (key ? p.cache.ldk : p.cache.ldv) + (key ? l : l - lk) * LINE);
     }
+  } else if (b.kind == BRANCH_LATENT_ATTN) {
+    const latent_rows<T>& p = b.latent;
+    const int pos = min(*(volatile const int*)pos_ptr, p.cache.ctx_len - 1);
+    int lo, blocks;
+    window_of(pos, p.window, 0, lo, blocks);
+    constexpr int LINE = 128 / sizeof(T);
+    const int ld = p.cache.ld, rp = p.cache.rot, kp = round_up_dev(p.dim, 8), vp = round_up_dev(p.vdim, 8), total = pos + 1 - lo;
+    // the head's matrices: this CTA's columns of the first, rows of the second
+    const int c0 = (rp >> 3) * rank / ST_CLUSTER * 8, c1 = (rp >> 3) * (rank + 1) / ST_CLUSTER * 8, lc = (c1 - c0 + LINE - 1) / LINE;
+    for (int i = tid; i < p.dim * lc; i += MX_THREADS)
+      l2_line(b.up + ((size_t)head * kp + i / lc) * b.ld_up + min(c0 + i % lc * LINE, rp - 1));
+    const int j0 = p.vdim * rank / ST_CLUSTER, j1 = p.vdim * (rank + 1) / ST_CLUSTER, lr = (rp + LINE - 1) / LINE;
+    for (int i = tid; i < (j1 - j0) * lr; i += MX_THREADS) l2_line(b.up + ((size_t)b.up_v + (size_t)head * vp + j0 + i / lr) * b.ld_up + i % lr * LINE);
+    // the heads share the cache rows of this CTA's slice
+    const int t0 = (int)((long long)total * rank / ST_CLUSTER), n = (int)((long long)total * (rank + 1) / ST_CLUSTER) - t0;
+    const int lk = (ld + LINE - 1) / LINE, heads = p.heads;
+    for (int i = tid + MX_THREADS * head; i < n * lk; i += MX_THREADS * heads) l2_line(p.cache.rows + (size_t)(lo + t0 + i / lk) * ld + min(i % lk * LINE, ld - 1));
   } else {
     const scan_rows<T>& p = b.scan;
     const int v0 = p.vdim * rank / ST_CLUSTER, nv = p.vdim * (rank + 1) / ST_CLUSTER - v0;
@@ -676,13 +841,14 @@ __global__ void __launch_bounds__(MX_THREADS) mixer_step_kernel(const __grid_con
   pdl_wait();
   const int pos = *p.pos;
   if (b.kind == BRANCH_WINDOW_ATTN) step_attention(b, head, rank, pos, sm, red);
+  else if (b.kind == BRANCH_LATENT_ATTN) step_latent(b, head, rank, pos, sm, red);
   else if (b.kind == BRANCH_RETENTION) step_recurrence<T, false>(b, head, rank, pos, sm, red);
   else step_recurrence<T, true>(b, head, rank, pos, sm, red);
 }
 
 template <typename T>
 size_t attention_smem(const attn_rows<T>& p, int keys, bool step) {
-  return ((step ? p.cache.ldk + p.cache.ldv : 0) + p.cache.ldk + PART_FLOATS + 2 + round_up(p.vdim + 2, 4) + keys + 8) * sizeof(float);
+  return ((step ? p.cache.ldk + p.cache.ldv : 0) + query_cols(p) + PART_FLOATS + 2 + round_up(p.vdim + 2, 4) + keys + 8) * sizeof(float);
 }
 template <typename T>
 int most_keys(const attn_rows<T>& p, int last_pos) {
@@ -712,7 +878,7 @@ int launch_window_append(const attn_rows<T>& p, int m, int pos0, cudaStream_t st
 template <typename T>
 int launch_window_attention(const attn_rows<T>& p, int m, int pos0, cudaStream_t stream) {
   if constexpr (sizeof(T) == 2)
-    if (window_mma_mode() && window_mma_supported(p.dim, p.vdim)) return launch_window_mma(p, m, pos0, stream);
+    if (window_mma_mode() && window_mma_supported(p.dim, p.key2 ? p.dim2 : 0, p.vdim)) return launch_window_mma(p, m, pos0, stream);
   const int keys = most_keys(p, pos0 + m - 1);
   const size_t smem = attention_smem(p, keys, false);
   LCU_REQUIRE(smem <= 220 * 1024, "window attention: %d visible keys", keys);
@@ -755,6 +921,7 @@ int launch_mixer_step(const mixer_step<T>& p, int ctx_len, cudaStream_t stream) 
   for (int i = 0; i < p.n_branches; ++i) {
     const step_branch<T>& b = p.b[i];
     if (b.kind == BRANCH_WINDOW_ATTN) smem = std::max(smem, attention_smem(b.attn, most_keys(b.attn, ctx_len - 1) / ST_CLUSTER + 2, true));
+    else if (b.kind == BRANCH_LATENT_ATTN) smem = std::max(smem, (latent_step_floats(b.latent) + std::min(b.latent.window, ctx_len) / ST_CLUSTER + 8) * sizeof(float));
     else smem = std::max(smem, (3 * (size_t)b.scan.dim + MX_THREADS + b.rank + 8) * sizeof(float));
   }
   LCU_REQUIRE(smem <= 220 * 1024, "mixer step: %zu bytes of shared memory", smem);

@@ -32,14 +32,29 @@ int block_model::create(std::unique_ptr<block_model>& out, const block_spec& spe
     mat(m->head, m->n_vocab_pad, m->k_width);
     vec(m->final_norm, W);
     vec(m->ones, S);
+    vec(m->zeros, S * S);
+    if (spec.loop_input) {
+      m->k_loop = pad_k(2 * W);
+      mat(m->loop_in, m->n_width, m->k_loop);
+    }
+    const hyper_weights plain{m->ones, m->ones, m->ones};  // (one stream: the plain sum)
+    auto residual = [&](hyper_weights& hc, float*& post, float*& scale) {
+      if (spec.sandwich) {
+        hc = plain;
+        vec(post, W);
+        vec(scale, W);
+        return;
+      }
+      vec(hc.in, S);
+      vec(hc.out, S);
+      vec(hc.mix, S * S);
+    };
     for (size_t i = 0; i < m->layers.size(); ++i) {
       const layer_spec& ls = spec.layers[i];
       block_layer& L = m->layers[i];
       L.branches.assign(ls.branches.size(), branch_weights{});
       vec(L.norm1, W);
-      vec(L.hc1.in, S);
-      vec(L.hc1.out, S);
-      vec(L.hc1.mix, S * S);
+      residual(L.hc1, L.norm1b, L.scale1);
       int rows = 0, cols = 0;
       for (size_t b = 0; b < ls.branches.size(); ++b) {
         const branch_spec& bs = ls.branches[b];
@@ -48,6 +63,22 @@ int block_model::create(std::unique_ptr<block_model>& out, const block_spec& spe
         cols += bs.out_cols();
         if (bs.kind == BRANCH_WKV) continue;
         bw.q = rows;
+        if (bs.kind == BRANCH_LATENT_ATTN) {
+          rows += bs.heads * (bs.dim_pad() + bs.rot_pad());
+          bw.k = rows;
+          rows += bs.rank_pad();
+          bw.v = rows;
+          rows += bs.rot_pad();
+          bw.g = rows;
+          rows += round_up(bs.heads, 8);
+          vec(bw.sink, bs.heads);
+          vec(bw.latent_norm, bs.kv_rank);
+          bw.up_v = bs.heads * bs.dim_pad();
+          bw.up_rows = pad_rows(bw.up_v + bs.heads * bs.vdim_pad());
+          bw.up_k = pad_k(bs.kv_rank);
+          mat(bw.up, bw.up_rows, bw.up_k);
+          continue;
+        }
         rows += bs.heads * bs.dim;
         bw.k = rows;
         rows += bs.kv_heads * bs.dim;
@@ -79,10 +110,18 @@ int block_model::create(std::unique_ptr<block_model>& out, const block_spec& spe
       mat(L.out, m->n_width, L.out_k);
       if (ls.ff > 0) {
         vec(L.norm2, W);
-        vec(L.hc2.in, S);
-        vec(L.hc2.out, S);
-        vec(L.hc2.mix, S * S);
+        residual(L.hc2, L.norm2b, L.scale2);
         L.ff_pad = pad_k(ls.ff);
+        if (ls.experts > 0) {
+          expert_weights& x = L.experts;
+          x.router_rows = pad_rows(ls.experts);
+          x.gate_up_stride = 2 * (size_t)L.ff_pad * m->k_width;
+          x.down_stride = (size_t)m->n_width * L.ff_pad;
+          mat(x.router, x.router_rows, m->k_width);
+          mat(x.gate_up, ls.experts * 2 * (size_t)L.ff_pad, m->k_width);
+          mat(x.down, ls.experts * (size_t)m->n_width, L.ff_pad);
+          continue;
+        }
         mat(L.gate_up, 2 * (size_t)L.ff_pad, m->k_width);
         mat(L.down, m->n_width, L.ff_pad);
       }
@@ -136,6 +175,9 @@ std::vector<block_model::slot> block_model::slots() const {
     s.optional = optional;
     out.push_back(s);
   };
+  auto grouped = [&](int group, int stride, int split = 1 << 30, int gap = 0) {  // of the matrix just listed
+    out.back().groups = row_groups{group, stride, split, gap};
+  };
   auto hyper = [&](const std::string& name, const hyper_weights& h) {
     const bool plain = S == 1;  // a single stream without tensors of its own is the plain residual sum
     vec(name + ".in", h.in, 1, S, slot::MEAN, false, plain);
@@ -144,12 +186,19 @@ std::vector<block_model::slot> block_model::slots() const {
   };
   mat("embed", embed, 0, 0, W, spec.vocab, W);
   if (spec.buckets > 0) mat("bigram", bigram, 0, 0, W, spec.buckets + 1, W);
+  if (spec.loop_input) mat("loop.in", loop_in, 0, 0, k_loop, W, 2 * W);
+  const slot::fill_t norm_fill = spec.sandwich ? slot::ONES : slot::ZEROS;
   for (size_t i = 0; i < layers.size(); ++i) {
     const layer_spec& ls = spec.layers[i];
     const block_layer& L = layers[i];
     const std::string l = "l" + std::to_string(i) + ".", mx = l + "mix.";
-    vec(l + "norm1", L.norm1, 1, W, slot::ZEROS);
-    hyper(l + "hc1", L.hc1);
+    vec(l + "norm1", L.norm1, 1, W, norm_fill);
+    if (spec.sandwich) {
+      vec(l + "norm1b", L.norm1b, 1, W, slot::ONES);
+      vec(l + "ls1", L.scale1, 1, W, slot::ONES);
+    } else {
+      hyper(l + "hc1", L.hc1);
+    }
     for (size_t b = 0; b < ls.branches.size(); ++b) {
       const branch_spec& bs = ls.branches[b];
       const branch_weights& bw = L.branches[b];
@@ -164,6 +213,19 @@ std::vector<block_model::slot> block_model::slots() const {
         vec(p + "w0", L.w0, 1, ch, slot::UNIFORM);
         vec(p + "u", L.u, bs.heads, bs.dim, slot::UNIFORM);
         vec(p + "norm", L.head_norm, 1, ch, slot::ONES);
+      } else if (bs.kind == BRANCH_LATENT_ATTN) {
+        const int dk = bs.dim + bs.rot_dim;
+        mat(p + "q", L.proj, bw.q, 0, k_width, bs.heads * dk, W);
+        grouped(dk, bs.dim_pad() + bs.rot_pad(), bs.dim, bs.dim_pad() - bs.dim);
+        mat(p + "dkv", L.proj, bw.k, 0, k_width, bs.kv_rank + bs.rot_dim, W);
+        grouped(bs.kv_rank + bs.rot_dim, 0, bs.kv_rank, bs.rank_pad() - bs.kv_rank);
+        vec(p + "dkv.norm", bw.latent_norm, 1, bs.kv_rank, slot::ONES);
+        mat(p + "uk", bw.up, 0, 0, bw.up_k, bs.heads * bs.dim, bs.kv_rank);
+        grouped(bs.dim, bs.dim_pad());
+        mat(p + "uv", bw.up, bw.up_v, 0, bw.up_k, bs.heads * bs.vdim, bs.kv_rank);
+        grouped(bs.vdim, bs.vdim_pad());
+        vec(p + "sink", bw.sink, 1, bs.heads, slot::ZEROS);
+        mat(p + "g", L.proj, bw.g, 0, k_width, bs.heads, W);
       } else {
         mat(p + "q", L.proj, bw.q, 0, k_width, bs.heads * bs.dim, W);
         mat(p + "k", L.proj, bw.k, 0, k_width, bs.kv_heads * bs.dim, W);
@@ -173,14 +235,33 @@ std::vector<block_model::slot> block_model::slots() const {
       mat(p + "o", L.out, 0, bw.out_col, L.out_k, W, ch);
     }
     if (ls.ff > 0) {
-      vec(l + "norm2", L.norm2, 1, W, slot::ZEROS);
-      hyper(l + "hc2", L.hc2);
+      vec(l + "norm2", L.norm2, 1, W, norm_fill);
+      if (spec.sandwich) {
+        vec(l + "norm2b", L.norm2b, 1, W, slot::ONES);
+        vec(l + "ls2", L.scale2, 1, W, slot::ONES);
+      } else {
+        hyper(l + "hc2", L.hc2);
+      }
+      if (ls.experts > 0) {
+        const expert_weights& x = L.experts;
+        constexpr int G = EXPERT_GATE_BLOCK;
+        mat(l + "mlp.router", x.router, 0, 0, k_width, ls.experts, W);
+        for (int e = 0; e < ls.experts; ++e) {
+          const std::string n = l + "mlp.e" + std::to_string(e);
+          mat(n + ".gate", (char*)x.gate_up + e * x.gate_up_stride * es, 0, 0, k_width, ls.ff, W);
+          grouped(G, 2 * G);
+          mat(n + ".up", (char*)x.gate_up + e * x.gate_up_stride * es, G, 0, k_width, ls.ff, W);
+          grouped(G, 2 * G);
+          mat(n + ".down", (char*)x.down + e * x.down_stride * es, 0, 0, L.ff_pad, W, ls.ff);
+        }
+        continue;
+      }
       mat(l + "mlp.gate", L.gate_up, 0, 0, k_width, ls.ff, W);
       mat(l + "mlp.up", L.gate_up, L.ff_pad, 0, k_width, ls.ff, W);
       mat(l + "mlp.down", L.down, 0, 0, L.ff_pad, W, ls.ff);
     }
   }
-  vec("final.norm", final_norm, 1, W, slot::ZEROS);
+  vec("final.norm", final_norm, 1, W, norm_fill);
   mat("head", head, 0, 0, k_width, spec.vocab, W);
   return out;
 }
@@ -223,8 +304,8 @@ int block_model::fill_synthetic(uint64_t seed, float scale) {
     rc = launch_synth_fill(tmp, n, seed, fnv1a64(s.name.c_str()), scale, 0, 0);
     if (!rc) rc = launch_half_to_f32(wide, tmp, n, 0);
     if (!rc)
-      rc = s.f32 ? launch_place<float>((float*)s.dst, s.ld, wide, PLACE_F32, s.rows, s.cols, s.transpose, 0)
-                 : launch_place<__nv_bfloat16>((__nv_bfloat16*)s.dst, s.ld, wide, PLACE_F32, s.rows, s.cols, s.transpose, 0);
+      rc = s.f32 ? launch_place<float>((float*)s.dst, s.ld, wide, PLACE_F32, s.rows, s.cols, s.transpose, 0, s.groups)
+                 : launch_place<__nv_bfloat16>((__nv_bfloat16*)s.dst, s.ld, wide, PLACE_F32, s.rows, s.cols, s.transpose, 0, s.groups);
   }
   e = cudaDeviceSynchronize();
   cudaFree(tmp);
@@ -282,8 +363,8 @@ int block_model::load(std::unique_ptr<block_model>& out, const std::string& dir,
       const place_source src = t->dtype == "F32" ? PLACE_F32 : PLACE_BF16;
       rc = loader.copy_file(file.path, tmp, t->bytes, t->offset, file.file_bytes);
       if (!rc)
-        rc = s.f32 ? launch_place<float>((float*)s.dst, s.ld, tmp, src, s.rows, s.cols, s.transpose, loader.stream)
-                   : launch_place<__nv_bfloat16>((__nv_bfloat16*)s.dst, s.ld, tmp, src, s.rows, s.cols, s.transpose, loader.stream);
+        rc = s.f32 ? launch_place<float>((float*)s.dst, s.ld, tmp, src, s.rows, s.cols, s.transpose, loader.stream, s.groups)
+                   : launch_place<__nv_bfloat16>((__nv_bfloat16*)s.dst, s.ld, tmp, src, s.rows, s.cols, s.transpose, loader.stream, s.groups);
     }
     if (rc) break;
   }

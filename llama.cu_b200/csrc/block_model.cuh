@@ -1,6 +1,7 @@
 // Block models on the device: weights of a block_spec in one arena, and the loader of a config.json + model.safetensors
 // directory.
 #pragma once
+#include "block_ops.cuh"
 #include "block_spec.cuh"
 #include "runtime.cuh"
 
@@ -18,12 +19,27 @@ struct hyper_weights {
   float *in = nullptr, *out = nullptr, *mix = nullptr;
 };
 struct branch_weights {
-  int q = 0, k = 0, v = 0, g = 0;  // columns of the branch's parts in a row of the stacked projection
+  int q = 0, k = 0, v = 0, g = 0;  // columns of the branch's parts in a row of the stacked projection (latent attention: k is
+                                   // the latent, v the shared key part that is rotated)
   int out_col = 0;                 // first column of its output in the mixer's output row
   float* decay = nullptr;          // retention
+  float* sink = nullptr;           // attention: per head
+  // latent attention: norm of the latent; [keys of all heads; values of all heads] from it, heads padded to 16-byte vectors
+  float* latent_norm = nullptr;
+  void* up = nullptr;
+  int up_rows = 0, up_v = 0, up_k = 0;  // rows, first value row, row length
+};
+// feed-forward with several experts: expert e's matrices are `gate_up_stride` / `down_stride` elements after expert 0's, in
+// gate_up blocks of EXPERT_GATE_BLOCK gate rows alternate with the blocks of the same up rows
+constexpr int EXPERT_GATE_BLOCK = 32;
+struct expert_weights {
+  void *router = nullptr, *gate_up = nullptr, *down = nullptr;
+  int router_rows = 0;
+  size_t gate_up_stride = 0, down_stride = 0;
 };
 struct block_layer {
   float *norm1 = nullptr, *norm2 = nullptr;
+  float *norm1b = nullptr, *norm2b = nullptr, *scale1 = nullptr, *scale2 = nullptr;  // of a sublayer's result
   hyper_weights hc1, hc2;
   std::vector<branch_weights> branches;
   // branches that read the row itself: one stacked projection
@@ -40,6 +56,7 @@ struct block_layer {
   // feed-forward: [gate; up] and down
   void *gate_up = nullptr, *down = nullptr;
   int ff_pad = 0;
+  expert_weights experts;  // (instead of gate_up and down)
 };
 
 struct block_model : model_base {
@@ -49,6 +66,9 @@ struct block_model : model_base {
   int k_width = 0, n_width = 0, n_vocab_pad = 0;  // padded input / output width, padded vocabulary
   void *embed = nullptr, *bigram = nullptr, *head = nullptr;
   float *final_norm = nullptr, *ones = nullptr;   // ones: [streams], the sum of the streams as an input vector
+  float* zeros = nullptr;                         // [streams * streams]
+  void* loop_in = nullptr;                        // [n_width][k_loop]
+  int k_loop = 0;                                 // padded length of a [residual; embedding] row
   std::vector<block_layer> layers;
 
   const char* family() const override { return spec.architecture.c_str(); }
@@ -72,6 +92,7 @@ struct block_model : model_base {
     int ld = 0;
     bool f32 = false;         // kept in binary32
     bool transpose = false;
+    row_groups groups;        // where rows go
     enum fill_t { MATRIX, ZEROS, ONES, IDENTITY, MEAN, UNIFORM } fill = MATRIX;  // synthetic values
     bool optional = false;    // may be missing: the synthetic values stand
   };

@@ -42,6 +42,12 @@ __global__ void __launch_bounds__(512) block_embed_kernel(const embed_params<T> 
       if (V == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(v);
       else dst[0] = v[0];
     }
+    if (p.copy) {
+      pack o;
+#pragma unroll
+      for (int k = 0; k < V; ++k) o.e[k] = from_f<T>(v[k]);
+      *reinterpret_cast<pack*>(p.copy + (size_t)r * p.ld_copy + c) = o;
+    }
   }
 }
 
@@ -50,18 +56,25 @@ constexpr int HY_THREADS = 256;
 constexpr int HY_MIX = 5;       // inputs of a token-shifted mixer
 constexpr int HY_CLUSTER = 8;  // CTAs that share one row when there is only one
 
-// SM: room for the streams (p.streams <= SM); CL: CTAs per row
-template <typename T, int SM, int CL>
+// SM: room for the streams (p.streams <= SM); CL: CTAs per row; PRE: y is gathered and normed first
+template <typename T, int SM, int CL, bool PRE>
 __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_params<T> p, const int per) {
-  extern __shared__ float u_row[];  // this CTA's columns of u
-  __shared__ float s_red[HY_THREADS / 32], s_part;
+  extern __shared__ __align__(16) float u_row[];  // this CTA's columns of u (PRE: first of y), then a router's partial sums
+  __shared__ float s_red[2][HY_THREADS / 32], s_part[2];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int i_row = blockIdx.x / CL, rank = blockIdx.x % CL;
   pdl_launch_dependents();
   if (CL > 1) {  // a single row: what the columns' last step needs from the weights is on its way while the kernel before ends
     const int first = min(p.width, rank * per), n = min(p.width, first + per) - first;
+    if (p.router) {
+      constexpr int LINE = 128 / sizeof(T);
+      const int lines = (n + LINE - 1) / LINE;
+      for (int i = tid; i < p.experts * lines; i += HY_THREADS) l2_line(p.router + (size_t)(i / lines) * p.ld_router + first + i % lines * LINE);
+    }
     for (int i = 32 * tid; i < n; i += 32 * HY_THREADS) {
-      l2_line(p.norm_w + first + i);
+      if (p.norm_w) l2_line(p.norm_w + first + i);
+      if (PRE && p.post_w) l2_line(p.post_w + first + i);
+      if (PRE && p.post_scale) l2_line(p.post_scale + first + i);
       if (p.mix)
         for (int k = 0; k < p.n_mix; ++k) l2_line(p.mu + (size_t)k * p.width + first + i);
     }
@@ -79,7 +92,53 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
     for (int t = 0; t < SM; ++t) mix[s][t] = p.y && s < S && t < S ? p.up_mix[s * S + t] : 0.f;
   }
   float* x = p.xs + (size_t)row * S * W;
-  const float* y = p.y ? p.y + (size_t)row * p.ldy : nullptr;
+  const float* y = p.y ? p.y + (PRE && p.y_rows ? 0 : (size_t)row * p.ldy) : nullptr;
+  auto row_total = [&](float v, int which) {  // over the CTA's threads, then the row's CTAs
+    v = warp_sum(v);
+    if (lane == 0) s_red[which][warp] = v;
+    __syncthreads();
+    float t = 0.f;
+#pragma unroll
+    for (int w = 0; w < HY_THREADS / 32; ++w) t += s_red[which][w];
+    if (CL > 1) {
+      if (tid == 0) s_part[which] = t;
+      cluster_sync();
+      t = 0.f;
+#pragma unroll
+      for (int r = 0; r < CL; ++r) t += ld_dsmem_f32(mapa(smem_u32(&s_part[which]), r));
+    }
+    return t;
+  };
+  float inv_y = 1.f;
+  if (PRE && y) {  // (a thread reads back only columns it has written itself)
+    const int* yr = p.y_rows ? p.y_rows + (size_t)row * p.n_y : nullptr;
+    const int pieces = yr ? p.n_y : 1;
+    float sy = 0.f;
+    if ((W & 3) == 0) {
+      for (int c = c0 + 4 * tid; c < c1; c += 4 * HY_THREADS) {
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int k = 0; k < pieces; ++k) {
+          const float4 v = *reinterpret_cast<const float4*>(y + (yr ? (size_t)yr[k] * p.ldy : 0) + c);
+          a = make_float4(a.x + v.x, a.y + v.y, a.z + v.z, a.w + v.w);
+        }
+        *reinterpret_cast<float4*>(u_row + c - c0) = a;
+        sy = fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(a.z, a.z, fmaf(a.w, a.w, sy))));
+      }
+    } else {
+      for (int c = c0 + tid; c < c1; c += HY_THREADS) {
+        float a = 0.f;
+        for (int k = 0; k < pieces; ++k) a += y[(yr ? (size_t)yr[k] * p.ldy : 0) + c];
+        u_row[c - c0] = a;
+        sy = fmaf(a, a, sy);
+      }
+    }
+    if (p.post_w) inv_y = 1.0f / sqrtf(row_total(sy, 0) / (float)W + p.eps);
+  }
+  auto y_at = [&](int c, float v) {  // PRE: the column's part in the sum
+    if (!PRE || !p.post_w) return v;
+    v *= inv_y * p.post_w[c];
+    return p.post_scale ? v * p.post_scale[c] : v;
+  };
   float ss = 0.f;
   auto column = [&](float (&v)[SM], float yv) {  // new streams in v, returns u
     if (y) {
@@ -104,7 +163,8 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
       float4 xv[SM];
 #pragma unroll
       for (int s = 0; s < SM; ++s) xv[s] = s < S ? *reinterpret_cast<const float4*>(x + (size_t)s * W + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-      const float4 yv = y ? *reinterpret_cast<const float4*>(y + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      float4 yv = y ? *reinterpret_cast<const float4*>(PRE ? u_row + c - c0 : y + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      if (PRE && y) yv = make_float4(y_at(c, yv.x), y_at(c + 1, yv.y), y_at(c + 2, yv.z), y_at(c + 3, yv.w));
       float4 u;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
@@ -129,7 +189,7 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
       float v[SM];
 #pragma unroll
       for (int s = 0; s < SM; ++s) v[s] = s < S ? x[(size_t)s * W + c] : 0.f;
-      const float u = column(v, y ? y[c] : 0.f);
+      const float u = column(v, y ? y_at(c, PRE ? u_row[c - c0] : y[c]) : 0.f);
       u_row[c - c0] = u;
       ss = fmaf(u, u, ss);
       if (y && p.store) {
@@ -139,27 +199,15 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
       }
     }
   }
-  ss = warp_sum(ss);
-  if (lane == 0) s_red[warp] = ss;
-  __syncthreads();
-  float total = 0.f;
-#pragma unroll
-  for (int w = 0; w < HY_THREADS / 32; ++w) total += s_red[w];
-  if (CL > 1) {
-    if (tid == 0) s_part = total;
-    cluster_sync();
-    total = 0.f;
-#pragma unroll
-    for (int r = 0; r < CL; ++r) total += ld_dsmem_f32(mapa(smem_u32(&s_part), r));
-  }
-  const float inv = 1.0f / sqrtf(total / (float)W + p.eps);
+  const float inv = 1.0f / sqrtf(row_total(ss, 1) / (float)W + p.eps);
   T* h = p.h + (size_t)i_row * p.ldh;
   const bool start = p.mix && *p.pos == 0;
   for (int c = c0 + tid; c < c1; c += HY_THREADS) {
     const float u = u_row[c - c0];
     if (p.u_out) p.u_out[(size_t)i_row * W + c] = u;
-    const T hv = from_f<T>(u * inv * (1.0f + p.norm_w[c]));
+    const T hv = from_f<T>(p.norm_w ? u * inv * (p.norm_base + p.norm_w[c]) : u);
     h[c] = hv;
+    if (CL > 1 && p.router) u_row[c - c0] = to_f(hv);
     if (p.mix) {
       const float hf = to_f(hv), d = (start ? 0.f : to_f(p.prev[c])) - hf;
       float mu[HY_MIX];
@@ -170,22 +218,58 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
       p.prev[c] = hv;
     }
   }
+  if (CL > 1 && p.router) {  // z = router . h: this CTA's columns of every expert, then the sum over the CTAs in rank 0
+    __syncthreads();
+    float* z = u_row + per;
+    for (int e = warp; e < p.experts; e += HY_THREADS / 32) {
+      const T* w = p.router + (size_t)e * p.ld_router + c0;
+      float a = 0.f;
+      if ((W & 3) == 0) {
+        struct __align__(4 * sizeof(T)) pack { T e[4]; };
+#pragma unroll 4
+        for (int c = 4 * lane; c < c1 - c0; c += 128) {
+          const pack wv = *reinterpret_cast<const pack*>(w + c);
+          const float4 hv = *reinterpret_cast<const float4*>(u_row + c);
+          a = fmaf(to_f(wv.e[0]), hv.x, fmaf(to_f(wv.e[1]), hv.y, fmaf(to_f(wv.e[2]), hv.z, fmaf(to_f(wv.e[3]), hv.w, a))));
+        }
+      } else {
+        for (int c = lane; c < c1 - c0; c += 32) a = fmaf(to_f(w[c]), u_row[c], a);
+      }
+      a = warp_sum(a);
+      if (lane == 0) z[e] = a;
+    }
+    cluster_sync();
+    if (rank == 0) {
+      for (int e = tid; e < p.experts; e += HY_THREADS) {
+        float a = 0.f;
+#pragma unroll
+        for (int r = 0; r < CL; ++r) a += ld_dsmem_f32(mapa(smem_u32(z + e), r));
+        z[p.experts + e] = a;
+      }
+      __syncthreads();
+      if (warp == 0)
+        pick_largest(z + p.experts, p.experts, p.top, [&](int k, int e, float v) {
+          p.pick[k] = e;
+          p.pick_weight[k] = sigmoid_f(v);
+        });
+    }
+  }
   if (CL > 1) cluster_sync();  // nobody leaves while its partial sum may still be read
 }
 
-template <typename T, int SM, int CL>
+template <typename T, int SM, int CL, bool PRE>
 int launch_hyper_one(const hyper_params<T>& p, int n_rows, cudaStream_t stream) {
   const int per = (int)round_up(ceil_div(p.width, CL), 4);
-  const size_t smem = (size_t)per * sizeof(float);
+  const size_t smem = ((size_t)per + (p.router ? 2 * p.experts : 0)) * sizeof(float);
   LCU_REQUIRE(smem <= 200 * 1024, "hyper_rows: a row of %d does not fit in shared memory", p.width);
   static bool attr_done[16] = {};
   int dev = 0;
   LCU_CUDA(cudaGetDevice(&dev));
   if (dev < 16 && !attr_done[dev]) {
-    LCU_CUDA(cudaFuncSetAttribute((hyper_rows_kernel<T, SM, CL>), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    LCU_CUDA(cudaFuncSetAttribute((hyper_rows_kernel<T, SM, CL, PRE>), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     attr_done[dev] = true;
   }
-  return launch_clustered(hyper_rows_kernel<T, SM, CL>, n_rows * CL, CL, HY_THREADS, smem, stream, p, per);
+  return launch_clustered(hyper_rows_kernel<T, SM, CL, PRE>, n_rows * CL, CL, HY_THREADS, smem, stream, p, per);
 }
 
 // ------------------------------------------------------------------ token shift
@@ -366,7 +450,7 @@ __global__ void __launch_bounds__(256) head_gate_kernel(T* out, int ldo, const f
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256) gate_rows_kernel(T* out, const T* ab, int m, int f) {
+__global__ void __launch_bounds__(256) gate_rows_kernel(T* out, const T* ab, int m, int f, const float* row_scale, int block) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int V = 16 / sizeof(T);
@@ -374,18 +458,21 @@ __global__ void __launch_bounds__(256) gate_rows_kernel(T* out, const T* ab, int
   const int fv = f / V;
   if (i >= (size_t)m * fv) return;
   const size_t r = i / fv, jv = i - r * fv;
-  const uint4 av = reinterpret_cast<const uint4*>(ab + r * 2 * f)[jv], bv = reinterpret_cast<const uint4*>(ab + r * 2 * f + f)[jv];
+  const size_t j = jv * V, ja = block ? j / block * 2 * block + j % block : j, jb = ja + (block ? block : f);
+  const uint4 av = *reinterpret_cast<const uint4*>(ab + r * 2 * f + ja), bv = *reinterpret_cast<const uint4*>(ab + r * 2 * f + jb);
+  const float s = row_scale ? row_scale[r] : 1.0f;
   __align__(16) T o[V];
 #pragma unroll
-  for (int e = 0; e < V; ++e) o[e] = from_f<T>(silu_f(to_f(reinterpret_cast<const T*>(&av)[e])) * to_f(reinterpret_cast<const T*>(&bv)[e]));
+  for (int e = 0; e < V; ++e) o[e] = from_f<T>(silu_f(s * to_f(reinterpret_cast<const T*>(&av)[e])) * (s * to_f(reinterpret_cast<const T*>(&bv)[e])));
   reinterpret_cast<uint4*>(out + r * f)[jv] = *reinterpret_cast<const uint4*>(o);
 }
 
 template <typename T>
-__global__ void place_kernel(T* dst, int ld, const void* src, int f32, int rows, int cols, int transpose) {
+__global__ void place_kernel(T* dst, int ld, const void* src, int f32, int rows, int cols, int transpose, const row_groups g) {
   const size_t n = (size_t)rows * cols;
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
-    const size_t r = i / cols, c = i - r * cols;
+    const size_t from = i / cols, c = i - from * cols, w = from % g.group;
+    const size_t r = from / g.group * g.stride + w + (w >= g.split ? g.gap : 0);
     const float v = f32 ? reinterpret_cast<const float*>(src)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(src)[i]);
     dst[transpose ? c * ld + r : r * ld + c] = from_f<T>(v);
   }
@@ -417,12 +504,20 @@ __global__ void __launch_bounds__(256) matmul_f32_few_kernel(float* out, const f
   }
 }
 // 64 x 64 tiles, 4 x 4 results per thread
-__global__ void __launch_bounds__(256) matmul_f32_tile_kernel(float* out, const float* x, int ldx, const float* w, int m, int N, int K) {
+__global__ void __launch_bounds__(256) matmul_f32_tile_kernel(float* out, const float* x, int ldx, const float* w, int m, int N, int K, const int4* tiles,
+                                                              const int* n_tiles) {
   __shared__ float xs[16][68], ws[16][68];
   pdl_launch_dependents();
   pdl_wait();
-  const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4, n0 = blockIdx.x * 64;
+  int m0 = blockIdx.y * 64;
+  if (tiles) {
+    if ((int)blockIdx.y >= *n_tiles) return;
+    const int4 t = tiles[blockIdx.y];
+    m0 = t.x;
+    m = t.y;
+    w += (size_t)t.z * N * K;
+  }
   float acc[4][4] = {};
   const int lr = tid >> 2, lk = (tid & 3) * 4;  // loader: row of the tile, four k
   for (int k0 = 0; k0 < K; k0 += 16) {
@@ -466,11 +561,14 @@ int launch_hyper_rows(const hyper_params<T>& p, int n_rows, cudaStream_t stream)
   if (n_rows < 1) return LCU_OK;
   LCU_REQUIRE(p.streams >= 1 && p.streams <= 8, "hyper_rows: %d streams", p.streams);
   LCU_REQUIRE(p.mix == nullptr || (n_rows == 1 && p.n_mix == HY_MIX), "hyper_rows: the token shift is fused for a single row of %d inputs", HY_MIX);
-#define LCU_HYPER(SM) \
-  return n_rows == 1 ? launch_hyper_one<T, SM, HY_CLUSTER>(p, n_rows, stream) : launch_hyper_one<T, SM, 1>(p, n_rows, stream)
-  if (p.streams == 1) LCU_HYPER(1);
-  if (p.streams == 2) LCU_HYPER(2);
-  if (p.streams <= 4) LCU_HYPER(4);
+  LCU_REQUIRE(p.router == nullptr || n_rows == 1, "hyper_rows: experts are picked for a single row");
+  const bool pre = p.y && (p.post_w || p.y_rows);
+#define LCU_HYPER(SM)                                                                                                                        \
+  if (pre) return n_rows == 1 ? launch_hyper_one<T, SM, HY_CLUSTER, true>(p, n_rows, stream) : launch_hyper_one<T, SM, 1, true>(p, n_rows, stream); \
+  return n_rows == 1 ? launch_hyper_one<T, SM, HY_CLUSTER, false>(p, n_rows, stream) : launch_hyper_one<T, SM, 1, false>(p, n_rows, stream)
+  if (p.streams == 1) { LCU_HYPER(1); }
+  if (p.streams == 2) { LCU_HYPER(2); }
+  if (p.streams <= 4) { LCU_HYPER(4); }
   LCU_HYPER(8);
 #undef LCU_HYPER
 }
@@ -523,17 +621,17 @@ int launch_head_gate(T* out, int ldo, const float* o, int ld_raw, const T* g, in
 }
 
 template <typename T>
-int launch_gate_rows(T* out, const T* ab, int m, int f, cudaStream_t stream) {
-  LCU_REQUIRE(f % 8 == 0, "gate_rows: rows of %d elements are not 16-byte vectors", f);
-  LCU_CUDA(launch_after(gate_rows_kernel<T>, dim3((unsigned)ceil_div((size_t)m * f * sizeof(T) / 16, 256)), dim3(256), 0, stream, out, ab, m, f));
+int launch_gate_rows(T* out, const T* ab, int m, int f, cudaStream_t stream, const float* row_scale, int block) {
+  LCU_REQUIRE(f % 8 == 0 && block % 8 == 0 && (block == 0 || f % block == 0), "gate_rows: rows of %d elements (blocks of %d) are not 16-byte vectors", f, block);
+  LCU_CUDA(launch_after(gate_rows_kernel<T>, dim3((unsigned)ceil_div((size_t)m * f * sizeof(T) / 16, 256)), dim3(256), 0, stream, out, ab, m, f, row_scale, block));
   return LCU_OK;
 }
 
 template <typename T>
-int launch_place(T* dst, int ld, const void* src, place_source type, int rows, int cols, bool transpose, cudaStream_t stream) {
+int launch_place(T* dst, int ld, const void* src, place_source type, int rows, int cols, bool transpose, cudaStream_t stream, const row_groups& groups) {
   const size_t n = (size_t)rows * cols;
   if (n == 0) return LCU_OK;
-  place_kernel<T><<<(unsigned)std::min<size_t>(ceil_div(n, 256), 148 * 16), 256, 0, stream>>>(dst, ld, src, type == PLACE_F32, rows, cols, transpose);
+  place_kernel<T><<<(unsigned)std::min<size_t>(ceil_div(n, 256), 148 * 16), 256, 0, stream>>>(dst, ld, src, type == PLACE_F32, rows, cols, transpose, groups);
   LCU_CUDA(cudaGetLastError());
   return LCU_OK;
 }
@@ -541,7 +639,14 @@ int launch_place(T* dst, int ld, const void* src, place_source type, int rows, i
 int launch_matmul_f32(float* out, const float* x, int ldx, const float* w, int m, int N, int K, cudaStream_t stream) {
   LCU_REQUIRE(m >= 1 && K % 16 == 0 && ldx % 4 == 0, "matmul_f32: unsupported shape m=%d K=%d", m, K);
   if (m <= MF_ROWS) LCU_CUDA(launch_after(matmul_f32_few_kernel, dim3((N + 7) / 8, 1), dim3(256), 0, stream, out, x, ldx, w, m, N, K));
-  else LCU_CUDA(launch_after(matmul_f32_tile_kernel, dim3((N + 63) / 64, (m + 63) / 64), dim3(256), 0, stream, out, x, ldx, w, m, N, K));
+  else LCU_CUDA(launch_after(matmul_f32_tile_kernel, dim3((N + 63) / 64, (m + 63) / 64), dim3(256), 0, stream, out, x, ldx, w, m, N, K, (const int4*)nullptr,
+                             (const int*)nullptr));
+  return LCU_OK;
+}
+int launch_matmul_f32_grouped(float* out, const float* x, int ldx, const float* w, int N, int K, const int4* tiles, const int* n_tiles, int most_tiles,
+                              cudaStream_t stream) {
+  LCU_REQUIRE(most_tiles >= 1 && K % 16 == 0 && ldx % 4 == 0, "matmul_f32: unsupported shape of %d tiles, K=%d", most_tiles, K);
+  LCU_CUDA(launch_after(matmul_f32_tile_kernel, dim3((N + 63) / 64, most_tiles), dim3(256), 0, stream, out, x, ldx, w, 0, N, K, tiles, n_tiles));
   return LCU_OK;
 }
 
@@ -550,8 +655,8 @@ int launch_matmul_f32(float* out, const float* x, int ldx, const float* w, int m
   template int launch_hyper_rows<T>(const hyper_params<T>&, int, cudaStream_t);                                                      \
   template int launch_token_shift<T>(const T*, int, T*, const float*, T*, size_t, int, int, int, int, cudaStream_t);                 \
   template int launch_head_gate<T>(T*, int, const float*, int, const T*, int, const float*, int, int, float, float, int, cudaStream_t); \
-  template int launch_gate_rows<T>(T*, const T*, int, int, cudaStream_t);                                                            \
-  template int launch_place<T>(T*, int, const void*, place_source, int, int, bool, cudaStream_t);
+  template int launch_gate_rows<T>(T*, const T*, int, int, cudaStream_t, const float*, int);                                                            \
+  template int launch_place<T>(T*, int, const void*, place_source, int, int, bool, cudaStream_t, const row_groups&);
 LCU_BLOCK_OPS(__nv_bfloat16)
 LCU_BLOCK_OPS(float)
 

@@ -66,6 +66,32 @@ int read_window_attention(const json_value& m, branch_spec& b) {
   return LCU_OK;
 }
 
+int read_rotation(const json_value& m, branch_spec& b, int most) {
+  const json_value *rot = nullptr, *base = nullptr;
+  SPEC_TRY(need(m, "rot", json_value::OBJECT, &rot));
+  SPEC_TRY(need_int(*rot, "dims", &b.rot_dims));
+  SPEC_TRY(need(*rot, "base", json_value::NUMBER, &base));
+  b.rot_base = base->number;
+  LCU_REQUIRE(b.rot_dims % 2 == 0 && b.rot_dims <= most, "config.json: %d rotated dimensions of %d", b.rot_dims, most);
+  return LCU_OK;
+}
+
+int read_latent_attention(const json_value& m, branch_spec& b) {
+  b.kind = BRANCH_LATENT_ATTN;
+  SPEC_TRY(need_int(m, "heads", &b.heads));
+  b.kv_heads = b.heads;
+  SPEC_TRY(need_int(m, "dim", &b.dim));
+  SPEC_TRY(need_int(m, "vdim", &b.vdim));
+  SPEC_TRY(need_int(m, "kv_rank", &b.kv_rank));
+  SPEC_TRY(need_int(m, "rot_dim", &b.rot_dim));
+  SPEC_TRY(need_float(m, "scale", &b.score_scale));
+  const json_value* mask = nullptr;
+  SPEC_TRY(need(m, "mask", json_value::OBJECT, &mask));
+  SPEC_TRY(need_int(*mask, "size", &b.window));
+  b.sink = b.head_gate = true;
+  return read_rotation(m, b, b.rot_dim);
+}
+
 int read_retention(const json_value& m, branch_spec& b) {
   b.kind = BRANCH_RETENTION;
   SPEC_TRY(need_int(m, "heads", &b.heads));
@@ -73,13 +99,7 @@ int read_retention(const json_value& m, branch_spec& b) {
   SPEC_TRY(need_int(m, "dim", &b.dim));
   b.vdim = b.dim;
   if (m.get("vdim")) SPEC_TRY(need_int(m, "vdim", &b.vdim));
-  if (const json_value* rot = m.get("rot")) {
-    SPEC_TRY(need_int(*rot, "dims", &b.rot_dims));
-    const json_value* base = nullptr;
-    SPEC_TRY(need(*rot, "base", json_value::NUMBER, &base));
-    b.rot_base = base->number;
-    LCU_REQUIRE(b.rot_dims % 2 == 0 && b.rot_dims <= b.dim, "config.json: %d rotated dimensions of %d", b.rot_dims, b.dim);
-  }
+  if (m.get("rot")) SPEC_TRY(read_rotation(m, b, b.dim));
   const json_value* decay = nullptr;
   SPEC_TRY(need(m, "decay", json_value::ARRAY, &decay));
   LCU_REQUIRE((int)decay->items.size() == b.heads, "config.json: %zu decays for %d heads", decay->items.size(), b.heads);
@@ -118,6 +138,16 @@ int read_mlp(const json_value& layer, layer_spec& l) {
   const json_value* mlp = layer.get("mlp");
   if (!mlp) return LCU_OK;
   const json_value* kind = mlp->get("kind");
+  if (kind && kind->text == "moe") {
+    const json_value *router = nullptr, *expert = nullptr;
+    SPEC_TRY(need(*mlp, "router", json_value::OBJECT, &router));
+    SPEC_TRY(need_int(*router, "experts", &l.experts));
+    SPEC_TRY(need_int(*router, "top", &l.top));
+    LCU_REQUIRE(l.experts <= MAX_EXPERTS, "config.json: %d experts (up to %d)", l.experts, MAX_EXPERTS);
+    LCU_REQUIRE(l.top <= l.experts && l.top <= MAX_TOP, "config.json: top %d of %d experts (up to %d)", l.top, l.experts, MAX_TOP);
+    SPEC_TRY(need(*mlp, "expert", json_value::OBJECT, &expert));
+    return need_int(*expert, "ff", &l.ff);
+  }
   LCU_REQUIRE(!kind || kind->text == "dense", "config.json: feed-forward kind '%s' is not known", kind->text.c_str());
   return need_int(*mlp, "ff", &l.ff);
 }
@@ -132,10 +162,14 @@ int read_runs(const json_value& c, block_spec& s) {
     SPEC_TRY(need_int(*loop, "times", &times, 0));
     LCU_REQUIRE(start <= stop && stop <= n, "config.json: loop over layers %d..%d of %d", start, stop, n);
   }
-  for (int i = 0; i < start; ++i) s.runs.push_back(i);
+  auto add = [&](int layer, bool first) {
+    s.runs.push_back(layer);
+    s.pass_start.push_back(first);
+  };
+  for (int i = 0; i < start; ++i) add(i, false);
   for (int t = 0; t < times; ++t)
-    for (int i = start; i < stop; ++i) s.runs.push_back(i);
-  for (int i = stop; i < n; ++i) s.runs.push_back(i);
+    for (int i = start; i < stop; ++i) add(i, i == start);
+  for (int i = stop; i < n; ++i) add(i, false);
   return LCU_OK;
 }
 
@@ -174,8 +208,31 @@ int read_filulix(const json_value& c, block_spec& s) {
   return read_runs(c, s);
 }
 
+// Zibovik: latent attention with a sink and gated heads, mixture of experts; norms before and after every sublayer, its
+// result scaled channel by channel; looped layers that start every pass from the residual and the embedding.
+int read_zibovik(const json_value& c, block_spec& s) {
+  SPEC_TRY(read_stack(c, s));
+  s.sandwich = true;
+  s.loop_input = c.get("loop") != nullptr;
+  const json_value* layers = nullptr;
+  SPEC_TRY(need(c, "layers", json_value::ARRAY, &layers));
+  for (auto& jl : layers->items) {
+    layer_spec l;
+    const json_value *type = nullptr, *mixer = nullptr;
+    SPEC_TRY(need(jl, "type", json_value::STRING, &type));
+    SPEC_TRY(need(jl, "mixer", json_value::OBJECT, &mixer));
+    LCU_REQUIRE(type->text == "latent_attention", "config.json: mixer type '%s' is not known", type->text.c_str());
+    l.branches.resize(1);
+    SPEC_TRY(read_latent_attention(*mixer, l.branches[0]));
+    SPEC_TRY(read_mlp(jl, l));
+    s.layers.push_back(std::move(l));
+  }
+  return read_runs(c, s);
+}
+
 const architecture ARCHITECTURES[] = {
     {"Filulix", read_filulix},
+    {"Zibovik", read_zibovik},
 };
 
 }  // namespace
@@ -208,6 +265,7 @@ int read_block_config(const std::string& text, block_spec& out) {
   for (auto& l : out.layers)
     for (auto& b : l.branches) {
       LCU_REQUIRE(b.dim <= 512 && b.vdim <= 512, "config.json: head size %d x %d (up to 512)", b.dim, b.vdim);
+      LCU_REQUIRE(b.kv_rank <= 2048 && b.rot_dim <= 512, "config.json: latent of %d with %d rotated dimensions (up to 2048 and 512)", b.kv_rank, b.rot_dim);
       LCU_REQUIRE(b.kind != BRANCH_WKV || l.branches.size() == 1, "config.json: a wkv mixer does not share its layer");
     }
   return LCU_OK;

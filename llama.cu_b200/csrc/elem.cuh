@@ -1,6 +1,7 @@
 // Element conversions, the gate function and the clustered launch shared by the block-model kernels.
 #pragma once
 #include <cuda_bf16.h>
+#include <math_constants.h>
 
 #include "common.cuh"
 
@@ -22,6 +23,37 @@ __host__ __device__ __forceinline__ int round_up_dev(int a, int b) { return (a +
 __device__ __forceinline__ void l2_line(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+
+// the `top` largest of z[0 .. n-1] (ties: the lower index) by one warp, in descending order: emit(k, index, value); z is used up
+template <typename F>
+__device__ __forceinline__ void pick_largest(float* z, int n, int top, F emit) {
+  const int lane = threadIdx.x & 31;
+  for (int k = 0; k < top; ++k) {
+    float best = -CUDART_INF_F;
+    int at = n;
+    for (int e = lane; e < n; e += 32)
+      if (z[e] > best) {
+        best = z[e];
+        at = e;
+      }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float b = __shfl_xor_sync(0xffffffffu, best, o);
+      const int a = __shfl_xor_sync(0xffffffffu, at, o);
+      if (a < n && (at >= n || b > best || (b == best && a < at))) {
+        best = b;
+        at = a;
+      }
+    }
+    if (at >= n) at = 0;  // (no value compares: not a number everywhere)
+    if (lane == 0) {
+      emit(k, at, best);
+      z[at] = -CUDART_INF_F;
+    }
+    __syncwarp();
+  }
+}
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 // launch of a kernel whose CTAs work in clusters of `cluster` (1: plain), as a programmatic dependent of the kernel before it
 template <typename... KP, typename... Args>

@@ -75,6 +75,21 @@ __device__ __forceinline__ void store_row_piece<float>(float* o, const float (&a
     reinterpret_cast<float4*>(o)[i] = v;
   }
 }
+// 32 columns of the gate and of the up part, both times the row's weight: silu(s a) * (s b)
+__device__ __forceinline__ void gate_piece(float (&a)[32], const float (&b)[32], float s) {
+#pragma unroll
+  for (int i = 0; i < 32; ++i) {
+    const float z = s * a[i];
+    a[i] = silu_of_half(z) * (s * b[i]);
+  }
+}
+// row groups (gemm_groups) as the kernels take them; mode 0: one matrix for all rows
+struct group_args {
+  const int4* tiles = nullptr;
+  const int* n_tiles = nullptr;
+  const float* row_scale = nullptr;
+};
+constexpr int GM_NONE = 0, GM_PLAIN = 1, GM_GATED = 2;
 __device__ __forceinline__ void st_dsmem_f4(uint32_t addr, float a, float b, float c, float d) {
   asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "f"(a), "f"(b), "f"(c), "f"(d) : "memory");
 }
@@ -85,10 +100,12 @@ __device__ __forceinline__ void st_dsmem_f4(uint32_t addr, float a, float b, flo
 // r BN / S: every CTA pushes its fp32 partials of the columns it does not own into the owner's shared
 // memory (distributed shared memory), one cluster barrier, and the owner adds them in rank order.
 // T: operand type (__half or __nv_bfloat16); TO: output type (T, or float for results that feed a 32-bit sum).
-template <typename T, typename TO, int BN, int S>
+// GM: row groups - blockIdx.y is a tile of the table, the CTA leaves with nothing done past its end.
+template <typename T, typename TO, int BN, int S, int GM = GM_NONE>
 __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                                                                 TO* out, int m, int N, int K, float beta, int nstages, int a_box_rows,
-                                                                int kbs, int* err) {
+                                                                int kbs, int* err, const group_args ga) {
+  static_assert(GM != GM_GATED || (S == 1 && BN % 64 == 0), "gate and up columns meet in one CTA");
   // A stage holds the activation box (a_box_rows rows, 2 to 16 KB) and the BN weight rows.  The MMA reads 128 operand rows
   // from the box's address: with a short box the rest comes from whatever follows in the ring, reaches output rows >= m
   // only, and those are never stored.  Short prompts so get up to 12 stages of weights in flight instead of 6.
@@ -115,9 +132,11 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const __grid_con
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int rank = S > 1 ? (int)cluster_ctarank() : 0;
-  const int n0 = (blockIdx.x / S) * BN, m0 = blockIdx.y * BM;
+  const int n0 = (blockIdx.x / S) * BN;
+  int m0 = blockIdx.y * BM, n_w = n0;  // first row, first weight row
   const int groups = (K / BK + kbs - 1) / kbs;  // (k-blocks past K in the last group arrive as zeros)
-  const int kb0 = rank * groups / S, nk = (rank + 1) * groups / S - kb0;  // this CTA's groups of k-blocks
+  const int kb0 = rank * groups / S;
+  int nk = (rank + 1) * groups / S - kb0;  // this CTA's groups of k-blocks
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < nstages; ++i) {
@@ -138,6 +157,17 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const __grid_con
   const uint32_t tmem_base = *tmem_slot;
   pdl_launch_dependents();
   pdl_wait();  // everything above ran under the previous kernel's tail; nothing before this line touches global memory
+  if (GM != GM_NONE) {
+    if ((int)blockIdx.y < *ga.n_tiles) {
+      const int4 t = ga.tiles[blockIdx.y];
+      m0 = t.x;
+      m = t.y;
+      n_w += t.z * N;
+    } else {  // (every CTA of a cluster has the same tile)
+      m0 = m = 0;
+      nk = 0;
+    }
+  }
 
   float own[S == 1 ? 1 : CPR][32];  // epilogue warps: this CTA's partial of the columns it owns
   bool go = false;
@@ -151,7 +181,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const __grid_con
         const uint32_t dst = base + (uint32_t)s * STAGE;
         mbar_arrive_expect_tx(full, STAGE);
         tma_load_3d(dst, &map_a, 0, m0, (kb0 + kb) * kbs, full);
-        tma_load_3d(dst + (uint32_t)kbs * A_BYTES, &map_b, 0, n0, (kb0 + kb) * kbs, full);
+        tma_load_3d(dst + (uint32_t)kbs * A_BYTES, &map_b, 0, n_w, (kb0 + kb) * kbs, full);
       }
     }
   } else if (warp == 1) {
@@ -179,9 +209,26 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const __grid_con
     const int trow = quad * 32 + lane;  // row of the tile = TMEM lane
     const bool ok = mbar_wait(smem_u32(&bars[2 * MAXS]), 0, err, DEV_ERR_TMEM_WAIT);
     tc_fence_after();
-    go = __all_sync(0xffffffffu, ok && *(volatile int*)err == 0);  // warp-uniform: tcgen05.ld is .aligned
+    go = __all_sync(0xffffffffu, ok && nk > 0 && *(volatile int*)err == 0);  // warp-uniform: tcgen05.ld is .aligned
     if (S > 1) asm volatile("barrier.cluster.wait.aligned;" ::: "memory");  // every CTA of the cluster is running
-    if (go) {
+    if (GM == GM_GATED && go) {
+      const float s = m0 + trow < m && ga.row_scale ? ga.row_scale[m0 + trow] : 1.f;
+#pragma unroll
+      for (int c = 0; c < BN / 32; c += 2) {
+        uint32_t ra[32], rb[32];
+        tc_ld_32x32(tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(c * 32), ra);
+        tc_ld_32x32(tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(c * 32 + 32), rb);
+        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+        float a[32], b[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          a[i] = __uint_as_float(ra[i]);
+          b[i] = __uint_as_float(rb[i]);
+        }
+        gate_piece(a, b, s);
+        if (m0 + trow < m && n0 + c * 32 < N) store_row_piece(out + (size_t)(m0 + trow) * (N / 2) + n0 / 2 + c * 16, a, 0.f);
+      }
+    } else if (go) {
 #pragma unroll
       for (int c = 0; c < BN / 32; ++c) {
         uint32_t r[32];
@@ -275,10 +322,10 @@ __device__ __forceinline__ void mbar_arrive_cluster(uint32_t bar_cluster_addr) {
   asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(bar_cluster_addr) : "memory");
 }
 
-template <typename T, typename TO, int BN>  // weight rows per pair tile: 128 or 256
+template <typename T, typename TO, int BN, int GM = GM_NONE>  // weight rows per pair tile: 128 or 256; row groups as above
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TC_THREADS, 1)
     gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, TO* out, int m, int N, int K,
-                        float beta, int nstages, int tiles_m, int n_tiles, int kbs, int* err) {
+                        float beta, int nstages, int tiles_m, int n_tiles, int kbs, int* err, const group_args ga) {
   // (a stage is kbs k-blocks, one three-dimensional tensor copy per operand, as in the one-SM kernel)
   constexpr uint32_t A_BYTES = BM * BK * 2, B_BYTES = (BN / 2) * BK * 2;
   const uint32_t STAGE = (uint32_t)kbs * (A_BYTES + B_BYTES);
@@ -317,14 +364,23 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TC_THREADS, 1)
   const uint32_t tmem_base = *tmem_slot;
   pdl_launch_dependents();
   pdl_wait();  // everything above ran under the previous kernel's tail; nothing before this line touches global memory
+  if (GM != GM_NONE) {
+    tiles_m = *ga.n_tiles;
+    n_tiles = tiles_m * (N / BN);
+  }
 
   if (warp == 0) {
     if (lane == 0) {  // ---- TMA producer (both CTAs)
       int it = 0;
       bool ok = true;
       for (int t = cluster_id; t < n_tiles && ok; t += n_clusters) {
-        const int m0 = (t % tiles_m) * (2 * BM) + (int)rank * BM;
-        const int n0 = (t / tiles_m) * BN + (int)rank * (BN / 2);
+        int m0 = (t % tiles_m) * (2 * BM) + (int)rank * BM;
+        int n0 = (t / tiles_m) * BN + (int)rank * (BN / 2);
+        if (GM != GM_NONE) {
+          const int4 tile = ga.tiles[t % tiles_m];
+          m0 = tile.x + (int)rank * BM;
+          n0 += tile.z * N;
+        }
         for (int kb = 0; kb < nk; kb += kbs, ++it) {  // (k-blocks past K arrive as zeros)
           const int s = it % nstages;
           const uint32_t ph = (uint32_t)(it / nstages) & 1u;
@@ -375,14 +431,36 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TC_THREADS, 1)
     for (int t = cluster_id; t < n_tiles && go; t += n_clusters, ++ti) {
       const int b = ti & 1;
       const uint32_t acc_ph = (uint32_t)(ti >> 1) & 1u;
-      const int row = (t % tiles_m) * (2 * BM) + (int)rank * BM + quad * 32 + lane;
+      int row = (t % tiles_m) * (2 * BM) + (int)rank * BM + quad * 32 + lane;
       const int n0 = (t / tiles_m) * BN;
+      float s = 1.f;
+      if (GM != GM_NONE) {
+        const int4 tile = ga.tiles[t % tiles_m];
+        row = tile.x + (int)rank * BM + quad * 32 + lane;
+        m = tile.y;
+        if (GM == GM_GATED && row < m && ga.row_scale) s = ga.row_scale[row];
+      }
       const bool ok = mbar_wait(smem_u32(&bars[16 + b]), acc_ph, err, DEV_ERR_TMEM_WAIT);
       tc_fence_after();
       go = __all_sync(0xffffffffu, ok && *(volatile int*)err == 0);
       if (!go) break;
 #pragma unroll 1
-      for (int c = 0; c < BN; c += 32) {
+      for (int c = 0; GM == GM_GATED && c < BN; c += 64) {
+        uint32_t ra[32], rb[32];
+        tc_ld_32x32(tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(b * BN + c), ra);
+        tc_ld_32x32(tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(b * BN + c + 32), rb);
+        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+        float a[32], bb[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          a[i] = __uint_as_float(ra[i]);
+          bb[i] = __uint_as_float(rb[i]);
+        }
+        gate_piece(a, bb, s);
+        if (row < m) store_row_piece(out + (size_t)row * (N / 2) + (n0 + c) / 2, a, 0.f);
+      }
+#pragma unroll 1
+      for (int c = 0; GM != GM_GATED && c < BN; c += 32) {
         uint32_t r[32];
         tc_ld_32x32(tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(b * BN + c), r);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -426,10 +504,13 @@ int get_encoder(encode_fn* out) {
   return LCU_OK;
 }
 
-template <typename T, typename TO, int BN, int S>
-int launch_bn(void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream) {
+// tile_m: rows a tile holds at most
+template <typename T, typename TO, int BN, int S, int GM = GM_NONE>
+int launch_bn(void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
+              const gemm_groups* gr = nullptr, int tile_m = 0) {
   CUtensorMap map_a, map_b;
-  const int a_box_rows = m > 64 ? BM : m > 32 ? 64 : m > 16 ? 32 : 16;
+  if (tile_m <= 0) tile_m = m;
+  const int a_box_rows = tile_m > 64 ? BM : tile_m > 32 ? 64 : tile_m > 16 ? 32 : 16;
   constexpr size_t RED = S > 1 ? (size_t)(S - 1) * BM * (BN / S) * 4 : 0;
   // k-blocks per stage: as many as still leave four stages and two stages' worth of work per CTA
   int kbs = tc_kb_per_stage();
@@ -443,7 +524,8 @@ int launch_bn(void* out, const void* lhs, int ldx, const void* w, int m, int N, 
     const uint32_t box_a[3] = {(uint32_t)BK, (uint32_t)a_box_rows, (uint32_t)kbs};
     int rc = tc_encode_map(&map_a, lhs, 3, dims_a, str_a, box_a);
     if (rc) return rc;
-    const uint64_t dims_b[3] = {(uint64_t)BK, (uint64_t)N, (uint64_t)(K / BK)}, str_b[2] = {(uint64_t)K * 2, (uint64_t)BK * 2};
+    const uint64_t n_rows = (uint64_t)N * (GM != GM_NONE ? gr->groups : 1);
+    const uint64_t dims_b[3] = {(uint64_t)BK, n_rows, (uint64_t)(K / BK)}, str_b[2] = {(uint64_t)K * 2, (uint64_t)BK * 2};
     const uint32_t box_b[3] = {(uint32_t)BK, (uint32_t)BN, (uint32_t)kbs};
     rc = tc_encode_map(&map_b, w, 3, dims_b, str_b, box_b, true);
     if (rc) return rc;
@@ -459,11 +541,13 @@ int launch_bn(void* out, const void* lhs, int ldx, const void* w, int m, int N, 
   int dev = 0;
   LCU_CUDA(cudaGetDevice(&dev));
   if (dev < 16 && !attr_done[dev]) {
-    LCU_CUDA(cudaFuncSetAttribute((gemm_tc_kernel<T, TO, BN, S>), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    LCU_CUDA(cudaFuncSetAttribute((gemm_tc_kernel<T, TO, BN, S, GM>), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     attr_done[dev] = true;
   }
   cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(((N + BN - 1) / BN) * S, (m + BM - 1) / BM);
+  cfg.gridDim = dim3(((N + BN - 1) / BN) * S, GM != GM_NONE ? gr->most_tiles : (m + BM - 1) / BM);
+  group_args ga;
+  if (GM != GM_NONE) ga = group_args{gr->tiles, gr->n_tiles, gr->row_scale};
   cfg.blockDim = dim3(TC_THREADS);
   cfg.dynamicSmemBytes = smem;
   cfg.stream = stream;
@@ -483,12 +567,13 @@ int launch_bn(void* out, const void* lhs, int ldx, const void* w, int m, int N, 
   }
   cfg.attrs = attr;
   cfg.numAttrs = n_attr;
-  LCU_CUDA(cudaLaunchKernelEx(&cfg, gemm_tc_kernel<T, TO, BN, S>, map_a, map_b, (TO*)out, m, N, K, beta, nstages, a_box_rows, kbs, err));
+  LCU_CUDA(cudaLaunchKernelEx(&cfg, gemm_tc_kernel<T, TO, BN, S, GM>, map_a, map_b, (TO*)out, m, N, K, beta, nstages, a_box_rows, kbs, err, ga));
   return LCU_OK;
 }
 
-template <typename T, typename TO, int BN>
-int launch_pair(void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream) {
+template <typename T, typename TO, int BN, int GM = GM_NONE>
+int launch_pair(void* out, const void* lhs, int ldx, const void* w, int m, int N, int K, float beta, int* err, cudaStream_t stream,
+                const gemm_groups* gr = nullptr) {
   CUtensorMap map_a, map_b;
   int kbs = sk_kb_per_stage();  // k-blocks per stage and tensor copy
   if (kbs <= 0) kbs = 2;
@@ -498,7 +583,8 @@ int launch_pair(void* out, const void* lhs, int ldx, const void* w, int m, int N
     const uint32_t box_a[3] = {(uint32_t)BK, (uint32_t)BM, (uint32_t)kbs};
     int rc = tc_encode_map(&map_a, lhs, 3, dims_a, str_a, box_a);
     if (rc) return rc;
-    const uint64_t dims_b[3] = {(uint64_t)BK, (uint64_t)N, (uint64_t)(K / BK)}, str_b[2] = {(uint64_t)K * 2, (uint64_t)BK * 2};
+    const uint64_t n_rows = (uint64_t)N * (GM != GM_NONE ? gr->groups : 1);
+    const uint64_t dims_b[3] = {(uint64_t)BK, n_rows, (uint64_t)(K / BK)}, str_b[2] = {(uint64_t)K * 2, (uint64_t)BK * 2};
     const uint32_t box_b[3] = {(uint32_t)BK, (uint32_t)(BN / 2), (uint32_t)kbs};
     rc = tc_encode_map(&map_b, w, 3, dims_b, str_b, box_b, true);
     if (rc) return rc;
@@ -511,14 +597,16 @@ int launch_pair(void* out, const void* lhs, int ldx, const void* w, int m, int N
   int dev = 0;
   LCU_CUDA(cudaGetDevice(&dev));
   if (dev < 16 && !attr_done[dev]) {
-    LCU_CUDA(cudaFuncSetAttribute((gemm_tc_pair_kernel<T, TO, BN>), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    LCU_CUDA(cudaFuncSetAttribute((gemm_tc_pair_kernel<T, TO, BN, GM>), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     attr_done[dev] = true;
   }
-  const int tiles_m = (m + 2 * BM - 1) / (2 * BM), n_tiles = tiles_m * (N / BN);
+  const int tiles_m = GM != GM_NONE ? gr->most_tiles : (m + 2 * BM - 1) / (2 * BM), n_tiles = tiles_m * (N / BN);
+  group_args ga;
+  if (GM != GM_NONE) ga = group_args{gr->tiles, gr->n_tiles, gr->row_scale};
   int clusters = gemv_sm_count() / 2;
   if (clusters > n_tiles) clusters = n_tiles;
-  LCU_CUDA(launch_after(gemm_tc_pair_kernel<T, TO, BN>, dim3(2 * clusters), dim3(TC_THREADS), smem, stream, map_a, map_b, (TO*)out, m, N, K, beta, nstages, tiles_m,
-                        n_tiles, kbs, err));
+  LCU_CUDA(launch_after(gemm_tc_pair_kernel<T, TO, BN, GM>, dim3(2 * clusters), dim3(TC_THREADS), smem, stream, map_a, map_b, (TO*)out, m, N, K, beta, nstages, tiles_m,
+                        n_tiles, kbs, err, ga));
   return LCU_OK;
 }
 
@@ -742,6 +830,28 @@ int launch_gemm_tc(tc_type type, void* out, const void* lhs, int ldx, const void
     case TC_BF16_F32: return launch_gemm_shape<__nv_bfloat16, float>(out, lhs, ldx, w, m, N, K, beta, err, stream, force_bn, force_pair, force_split);
   }
   LCU_REQUIRE(false, "gemm_tc: unknown operand type %d", (int)type);
+}
+
+// rows per tile: whole SM-pair tiles once the groups hold about that many rows each
+int gemm_tc_group_tile(int rows, int groups) { return rows >= 160 * groups ? 2 * BM : BM; }
+
+int launch_gemm_tc_grouped(tc_type type, void* out, const void* lhs, int ldx, const void* w, int rows, int N, int K, bool gated, const gemm_groups& g,
+                           int* err, cudaStream_t stream) {
+  LCU_REQUIRE(type == (gated ? TC_BF16 : TC_BF16_F32), "gemm_tc_grouped: operand type %d", (int)type);
+  LCU_REQUIRE(rows >= 1 && N % 128 == 0 && gemm_tc_supported(rows, N, K, ldx, lhs, w, out), "gemm_tc_grouped: unsupported shape m=%d N=%d K=%d", rows, N, K);
+  LCU_REQUIRE(g.tile_rows == BM || g.tile_rows == 2 * BM, "gemm_tc_grouped: tiles of %d rows", g.tile_rows);
+  using T = __nv_bfloat16;
+  if (g.tile_rows == 2 * BM) {
+    if (gated) {
+      if (N % 256 == 0) return launch_pair<T, T, 256, GM_GATED>(out, lhs, ldx, w, rows, N, K, 0.f, err, stream, &g);
+      return launch_pair<T, T, 128, GM_GATED>(out, lhs, ldx, w, rows, N, K, 0.f, err, stream, &g);
+    }
+    if (N % 256 == 0) return launch_pair<T, float, 256, GM_PLAIN>(out, lhs, ldx, w, rows, N, K, 0.f, err, stream, &g);
+    return launch_pair<T, float, 128, GM_PLAIN>(out, lhs, ldx, w, rows, N, K, 0.f, err, stream, &g);
+  }
+  const int tile_m = std::min(rows, BM);
+  if (gated) return launch_bn<T, T, 128, 1, GM_GATED>(out, lhs, ldx, w, rows, N, K, 0.f, err, stream, &g, tile_m);
+  return launch_bn<T, float, 128, 1, GM_PLAIN>(out, lhs, ldx, w, rows, N, K, 0.f, err, stream, &g, tile_m);
 }
 
 }  // namespace lcu

@@ -25,6 +25,22 @@ inline int launch_gemm_tc(__half* out, const __half* lhs, int ldx, const __half*
   return launch_gemm_tc(TC_F16, out, lhs, ldx, w, m, N, K, beta, err, stream, force_bn, force_pair, force_split);
 }
 
+// Products of several row groups with a matrix each (the experts of a routed feed-forward): rows lie group after group, and a
+// table on the device cuts them into tiles of up to tile_rows rows of one group: {first row, row past the last, group, -}.
+// Group g's matrix is w + g * N * K.  gated: w alternates blocks of 32 gate and 32 up rows, and out[rows][N / 2] =
+// silu(s a) * (s b) with s = row_scale[row] - a row's weight, applied to the expert's input.  out is dense.
+struct gemm_groups {
+  const int4* tiles;
+  const int* n_tiles;       // in device memory
+  int most_tiles;           // bound of *n_tiles
+  int tile_rows;            // 128 or 256 (gemm_tc_group_tile)
+  int groups;
+  const float* row_scale;
+};
+int gemm_tc_group_tile(int rows, int groups);  // for `rows` rows over all groups
+int launch_gemm_tc_grouped(tc_type type, void* out, const void* lhs, int ldx, const void* w, int rows, int N, int K, bool gated, const gemm_groups& g,
+                           int* err, cudaStream_t stream);
+
 // Wide-tile variant with the K loop balanced over the SM pairs (gemm_tc_sk.cu): 256 x tile_n output tiles (tile_n 256 or
 // 512, dividing N), any number of rows.  Partial sums of tiles shared between pairs go through a workspace kept per
 // (device, stream) and are added in a fixed order.

@@ -10,7 +10,7 @@ enum gemv_epilogue : int {
   EPI_SILU = 2      // two matrices w1|w3 interleaved row by row: out[i] = half(silu(half(a_i)) * half(b_i))
 };
 
-constexpr int GEMV_MAX_BATCH = 6;
+constexpr int GEMV_MAX_BATCH = 8;
 
 struct gemv_params {
   // weights: up to three [rows_per_mat][K] matrices that share K; fp16, or u8 with fp16 scales [rows][K/bs]
@@ -66,10 +66,20 @@ struct gemv_batch {
   int rows[GEMV_MAX_BATCH];
   int f32[GEMV_MAX_BATCH];              // output type: 0 bfloat16, 1 binary32
   int first_cta[GEMV_MAX_BATCH + 1];    // filled in by the launch
+  // matrices picked on the device (experts): entry i works on w[i] + choice[i] * choice_bytes
+  const int* choice = nullptr;
+  size_t choice_bytes = 0;
+  bool choice_settled = false;          // `choice` is older than the kernel before this one, which was launched with `hold`
+  const float* gate_scale = nullptr;    // gate epilogue: factor of both parts, per entry
+  int gate_shift = 0;                   // gate epilogue: gate and up rows alternate in blocks of 1 << gate_shift
+  bool hold = false;                    // the next kernel may not start before every CTA of this one sees its predecessor's results
 };
 int launch_gemv_bf16(const gemv_batch& b, int K, int* err, cudaStream_t stream, int pdl);
 // out[f] = bfloat16(silu(w1 . x) * (w3 . x)), w13 = [w1; w3] stacked ([2 f][K])
 int launch_gemv_bf16_gated(void* out, const void* x, const void* w13, int f, int K, int* err, cudaStream_t stream, int pdl);
+// the same for b.n picked matrices w[0] + choice[i] and one input vector b.x[0]: b.out[i][f] = bfloat16(silu(s a) * (s b)),
+// s = gate_scale[i]
+int launch_gemv_bf16_gated_picked(const gemv_batch& b, int f, int K, int* err, cudaStream_t stream, int pdl);
 
 constexpr int TP_EXCHANGES_PER_STEP = 1024;  // bound of the exchange ids of one decode step
 

@@ -24,6 +24,8 @@
 // (reference llama_cu.cu:287-289); the RMSNorm prologue keeps the reference's summation order.
 #include <cuda_bf16.h>
 
+#include <algorithm>
+
 #include "gemv.cuh"
 
 namespace lcu {
@@ -225,16 +227,23 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
   uint8_t* stages = nws + (p.norm_w != nullptr && p.K > 4096 ? (((p.K - 4096) * 2 + 127) & ~127) : 0);  // [NW][sw][STAGE_BYTES]
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  pdl_launch_dependents();
+  if (WT != 3 || !bt.hold) pdl_launch_dependents();
 
   int pairs = (p.n_mats * p.rows_per_mat) >> 1, cta = blockIdx.x, n_ctas = gridDim.x, bi = 0;
-  if (WT == 3 && EPI == EPI_PLAIN) {  // which of the batch's matrices this CTA works on
+  if (WT == 3 && bt.n > 0) {  // which of the batch's matrices this CTA works on
     while (bi + 1 < bt.n && (int)blockIdx.x >= bt.first_cta[bi + 1]) ++bi;
     cta = blockIdx.x - bt.first_cta[bi];
     n_ctas = bt.first_cta[bi + 1] - bt.first_cta[bi];
     pairs = bt.rows[bi] >> 1;
   }
-  auto weights_of = [&](int mat) { return reinterpret_cast<const uint8_t*>(WT == 3 && EPI == EPI_PLAIN ? bt.w[bi] : p.w[mat]); };
+  // (picked matrices: the producer warp reads the choice once it is there, see below)
+  size_t picked = 0;
+  auto weights_of = [&](int mat) { return reinterpret_cast<const uint8_t*>(WT == 3 && bt.n > 0 ? bt.w[bi] : p.w[mat]) + (WT == 3 ? picked : 0); };
+  // row of a matrix in memory: gate and up rows of picked matrices alternate in blocks
+  auto place_of = [&](int mat, int row) {
+    if (WT == 3 && EPI == EPI_SILU && bt.n > 0) return ((row >> bt.gate_shift) << (bt.gate_shift + 1)) + (mat << bt.gate_shift) + (row & ((1 << bt.gate_shift) - 1));
+    return row;
+  };
   const __half* x_row = WT == 3 && EPI == EPI_PLAIN ? reinterpret_cast<const __half*>(bt.x[bi]) : p.x;
   const int pr0 = (int)(((long long)pairs * cta) / n_ctas);
   const int npairs = (int)(((long long)pairs * (cta + 1)) / n_ctas) - pr0;
@@ -260,12 +269,16 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
     // ------------------------------------------------------------ producer
     // (this warp's instruction chain per stage bounds the u8 kernels: shifts, no divisions)
     const uint64_t pol = policy_evict_first();
+    if (WT == 3 && bt.choice != nullptr) {
+      if (!bt.choice_settled) pdl_wait();
+      picked = (size_t)bt.choice[bi] * bt.choice_bytes;
+    }
     if (pf_bytes > 0) {  // L2 look-ahead over the first rows of this CTA
       const int rows_pf = max(1, min(pf_bytes / rowbytes, 2 * npairs));
       for (int r = lane; r < rows_pf; r += 32) {
         int mat, row;
         map_row<EPI>(p, 2 * pr0 + r, mat, row);
-        l2_prefetch(weights_of(mat) + (size_t)row * rowbytes, (uint32_t)rowbytes);
+        l2_prefetch(weights_of(mat) + (size_t)place_of(mat, row) * rowbytes, (uint32_t)rowbytes);
       }
     }
     int slot[NW];
@@ -306,7 +319,7 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
     auto pair_sources = [&](const int pr, const uint8_t*& row_src, const __half*& sc_src) {
       int mat, row;
       map_row<EPI>(p, 2 * pr + (lane & 1), mat, row);
-      row_src = weights_of(mat) + (size_t)row * rowbytes;
+      row_src = weights_of(mat) + (size_t)place_of(mat, row) * rowbytes;
       sc_src = nullptr;
       if (!is16<WT>) {
         int m2, r2;
@@ -360,6 +373,8 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
     cp_async_commit();
   }
   pdl_wait();
+  if (WT == 3 && bt.hold) pdl_launch_dependents();
+  const float gate_scale = WT == 3 && EPI == EPI_SILU && bt.n > 0 ? bt.gate_scale[bi] : 1.0f;
   if (npairs > 0) {
     // Rows that fit the consumers' registers (NVEC vectors per thread: K <= 4096 with four warps) are loaded by the
     // threads themselves and stay in registers for the normalisation.  Longer rows come in as bulk copies of one
@@ -543,7 +558,9 @@ __global__ void __launch_bounds__((NW + 1) * 32, NW == 4 ? 3 : 2) gemv1_kernel(c
           if (bt.f32[bi]) *reinterpret_cast<float2*>(reinterpret_cast<float*>(bt.out[bi]) + vrow) = make_float2(v0, v1);
           else *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(bt.out[bi]) + vrow) = __floats2bfloat162_rn(v0, v1);
         } else {  // the gate on the binary32 sums
-          reinterpret_cast<__nv_bfloat16*>(p.out)[pr] = __float2bfloat16(v0 / (1.0f + expf(-v0)) * v1);
+          __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(bt.n > 0 ? bt.out[bi] : p.out);
+          const float z = gate_scale * v0;
+          o[pr] = __float2bfloat16(z / (1.0f + expf(-z)) * (gate_scale * v1));
         }
         continue;
       }
@@ -764,6 +781,31 @@ int launch_gemv_bf16_gated(void* out, const void* x, const void* w13, int f, int
   int rc = configure(p, gemv_sm_count(), c);
   if (rc) return rc;
   return launch_one<3, EPI_SILU, 4>(p, stream, pdl, c.smem, c.grid, c.sw, c.pf);
+}
+
+int launch_gemv_bf16_gated_picked(const gemv_batch& b, int f, int K, int* err, cudaStream_t stream, int pdl) {
+  LCU_REQUIRE(b.n >= 1 && b.n <= GEMV_MAX_BATCH && b.choice && b.gate_scale, "gemv: %d picked matrices outside 1..%d", b.n, GEMV_MAX_BATCH);
+  LCU_REQUIRE(K > 0 && K % 256 == 0 && f > 0, "gemv: K=%d must be a positive multiple of 256", K);
+  LCU_REQUIRE(f % (1 << b.gate_shift) == 0, "gemv: %d rows in blocks of %d", f, 1 << b.gate_shift);
+  LCU_REQUIRE((((uintptr_t)b.w[0] | (uintptr_t)b.x[0] | b.choice_bytes) & 15) == 0, "gemv: unaligned operand");
+  gemv_params p{};
+  p.n_mats = 2;
+  p.rows_per_mat = f * b.n;
+  p.K = K;
+  p.m = 1;
+  p.x = reinterpret_cast<const __half*>(b.x[0]);
+  p.err = err;
+  gemv1_config c;
+  int rc = configure(p, gemv_sm_count(), c);
+  if (rc) return rc;
+  gemv_batch bt = b;
+  const int per = std::max(1, c.grid / b.n);  // every matrix the same share of the CTAs
+  for (int i = 0; i <= b.n; ++i) bt.first_cta[i] = i * per;
+  for (int i = 0; i < b.n; ++i) {
+    bt.w[i] = b.w[0];
+    bt.rows[i] = 2 * f;
+  }
+  return launch_one<3, EPI_SILU, 4>(p, stream, pdl, c.smem, per * b.n, c.sw, c.pf, bt);
 }
 
 }  // namespace lcu

@@ -69,6 +69,10 @@ def norm_around_zero(x, w, eps):
     return unit_rms(x, eps) * (1 + w)
 
 
+def norm(x, w, eps):
+    return unit_rms(x, eps) * w
+
+
 # ------------------------------------------------------------------ embedding
 def embed(tokens, W, cfg):
     e = cfg["embedding"]
@@ -162,11 +166,72 @@ def wkv(h, W, p, m, eps):
     return o @ W[p + "o"].T
 
 
-MIXERS = {"parallel": parallel, "wkv": wkv}
+def rotate_pairs(x, positions, base, dims):
+    """x [tokens, heads, dim]: dimensions 0 .. dims-1 in the pairing (2i, 2i + 1)."""
+    out = x.copy()
+    for i in range(dims // 2):
+        a = positions * base ** (-2.0 * i / dims)
+        c, s = np.cos(a)[:, None].astype(x.dtype), np.sin(a)[:, None].astype(x.dtype)
+        u, v = x[..., 2 * i], x[..., 2 * i + 1]
+        out[..., 2 * i] = u * c - v * s
+        out[..., 2 * i + 1] = v * c + u * s
+    return out
+
+
+def window_softmax(q, k, v, scale, size, sink=None):
+    """q, k [tokens, heads, dim], v [tokens, heads, vdim]: position i sees i - size + 1 .. i; sink [heads]: one more term
+    exp(sink) of every denominator."""
+    T, H, _ = q.shape
+    out = np.zeros((T, H, v.shape[2]), q.dtype)
+    for i in range(T):
+        lo = max(0, i - size + 1)
+        for hd in range(H):
+            s = k[lo:i + 1, hd] @ q[i, hd] * scale
+            top = s.max() if sink is None else max(s.max(), sink[hd])
+            e = np.exp(s - top)
+            out[i, hd] = e @ v[lo:i + 1, hd] / (e.sum() + (0 if sink is None else np.exp(sink[hd] - top)))
+    return out
+
+
+def latent_attention(h, W, p, m, eps):
+    """Keys and values of every head from one normalised latent per token, and one rotated key part for all heads."""
+    T = h.shape[0]
+    H, D, R, DV, C = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    pos = np.arange(T).astype(np.float64)
+    q = (h @ W[p + "q"].T).reshape(T, H, D + R)
+    down = h @ W[p + "dkv"].T
+    c = norm(down[:, :C], W[p + "dkv.norm"], eps)
+    turn = lambda a: rotate_pairs(a, pos, m["rot"]["base"], m["rot"]["dims"])  # noqa: E731
+    q_rot, k_rot = turn(q[..., D:]), turn(down[:, None, C:])
+    k = np.concatenate([(c @ W[p + "uk"].T).reshape(T, H, D), np.repeat(k_rot, H, axis=1)], axis=2)
+    v = (c @ W[p + "uv"].T).reshape(T, H, DV)
+    o = window_softmax(np.concatenate([q[..., :D], q_rot], axis=2), k, v, m["scale"], m["mask"]["size"], W[p + "sink"])
+    o = o * sigmoid(h @ W[p + "g"].T)[:, :, None]
+    return o.reshape(T, H * DV) @ W[p + "o"].T
+
+
+MIXERS = {"parallel": parallel, "wkv": wkv, "latent_attention": latent_attention}
 
 
 def feed_forward(h, W, p):
     return (silu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
+
+
+def route(h, W, p, top):
+    """(experts, weights) of every token: the `top` largest scores sigmoid(z), which are the weights as they are."""
+    z = h @ W[p + "router"].T
+    pick = np.argsort(-z, axis=1, kind="stable")[:, :top]
+    return pick, sigmoid(np.take_along_axis(z, pick, axis=1))
+
+
+def experts(h, W, p, m):
+    """A weight multiplies its expert's input."""
+    pick, weight = route(h, W, p, m["router"]["top"])
+    out = np.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, w in zip(pick[t], weight[t]):
+            out[t] += feed_forward(w * h[t:t + 1], W, f"{p}e{e}.")[0]
+    return out
 
 
 # ------------------------------------------------------------------ the stack
@@ -186,8 +251,34 @@ def hyper_sublayer(streams, W, hc, fn):
     return np.einsum("st,sxd->txd", W[hc + "mix"], streams) + W[hc + "out"][:, None, None] * y[None]
 
 
+def sandwich_sublayer(x, W, p, n, eps, fn):
+    """Norm before and after the sublayer, the result scaled channel by channel."""
+    return x + W[f"{p}ls{n}"] * norm(fn(norm(x, W[f"{p}norm{n}"], eps)), W[f"{p}norm{n}b"], eps)
+
+
+def forward_sandwich(tokens, cfg, W, dtype=np.float64, layers_out=None):
+    """Logits [tokens, vocab] of a stack of sandwich sublayers in which every pass of the loop starts from a linear map of the
+    residual row beside the embedding row."""
+    W = {k: a.astype(dtype) for k, a in W.items()}
+    eps = cfg["norm"]["eps"]
+    x = x0 = W["embed"][np.asarray(tokens)]
+    runs, loop = layer_runs(cfg), cfg.get("loop")
+    for n, i in enumerate(runs):
+        L, p = cfg["layers"][i], f"l{i}."
+        if loop and loop["start"] <= n < loop["start"] + (loop["stop"] - loop["start"]) * loop["times"] and i == loop["start"]:
+            x = np.concatenate([x, x0], axis=1) @ W["loop.in"].T
+        x = sandwich_sublayer(x, W, p, 1, eps, lambda h: MIXERS[L["type"]](h, W, p + "mix.", L["mixer"], eps))
+        if L.get("mlp"):
+            x = sandwich_sublayer(x, W, p, 2, eps, lambda h: experts(h, W, p + "mlp.", L["mlp"]))
+        if layers_out is not None:
+            layers_out.append(x)
+    return norm(x, W["final.norm"], eps) @ W["head"].T
+
+
 def forward(tokens, cfg, W, dtype=np.float64, layers_out=None):
     """Logits [tokens, vocab] of one whole sequence; layers_out collects the sum of the streams after every layer run."""
+    if cfg["architecture"] == "Zibovik":
+        return forward_sandwich(tokens, cfg, W, dtype, layers_out)
     W = {k: a.astype(dtype) for k, a in W.items()}
     eps = cfg["norm"]["eps"]
     x = embed(np.asarray(tokens), W, cfg).astype(dtype)
