@@ -832,8 +832,15 @@ int launch_gemm_tc(tc_type type, void* out, const void* lhs, int ldx, const void
   LCU_REQUIRE(false, "gemm_tc: unknown operand type %d", (int)type);
 }
 
+int& gemm_tc_group_mode() {
+  static int mode = 0;
+  return mode;
+}
 // rows per tile: whole SM-pair tiles once the groups hold about that many rows each
-int gemm_tc_group_tile(int rows, int groups) { return rows >= 160 * groups ? 2 * BM : BM; }
+int gemm_tc_group_tile(int rows, int groups) {
+  const int mode = gemm_tc_group_mode();
+  return mode == BM || mode == 2 * BM ? mode : rows >= 160 * groups ? 2 * BM : BM;
+}
 
 int launch_gemm_tc_grouped(tc_type type, void* out, const void* lhs, int ldx, const void* w, int rows, int N, int K, bool gated, const gemm_groups& g,
                            int* err, cudaStream_t stream) {

@@ -38,6 +38,7 @@ struct gemm_groups {
   const float* row_scale;
 };
 int gemm_tc_group_tile(int rows, int groups);  // for `rows` rows over all groups
+int& gemm_tc_group_mode();  // 128 / 256 = always that tile, 0 (default) = by the rows per group
 int launch_gemm_tc_grouped(tc_type type, void* out, const void* lhs, int ldx, const void* w, int rows, int N, int K, bool gated, const gemm_groups& g,
                            int* err, cudaStream_t stream);
 

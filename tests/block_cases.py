@@ -85,6 +85,86 @@ def case(seed=0, **kw):
     return cfg, weights(cfg, seed)
 
 
+# ------------------------------------------------------------------ latent attention and experts
+def latent_mixer(heads=3, dim=20, rot_dim=6, vdim=12, kv_rank=28, window=11, base=700.0, scale=None, rot_dims=None):
+    return {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "mask": {"size": window},
+            "rot": {"base": base, "dims": rot_dims or rot_dim}, "scale": scale if scale is not None else 1.5 * (dim + rot_dim) ** -0.5}
+
+
+def latent_config(layers=2, loop=None, vocab=211, width=88, mixer=None, mixers=None, experts=5, top=2, ff=24, mlp_none=(), eps=2e-5, moe=None):
+    """mixers / moe: per-layer changes {layer: {...}} of the common mixer / (experts, top, ff)."""
+    ls = []
+    for i in range(layers):
+        e = {"experts": experts, "top": top, "ff": ff, **((moe or {}).get(i, {}))}
+        ls.append({"type": "latent_attention", "mixer": latent_mixer(**{**(mixer or {}), **((mixers or {}).get(i, {}))}),
+                   "mlp": None if i in mlp_none else {"kind": "moe", "expert": {"ff": e["ff"]}, "router": {"experts": e["experts"], "top": e["top"]}}})
+    cfg = {"architecture": "Zibovik", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": ls}
+    if loop:
+        cfg["loop"] = loop
+    return cfg
+
+
+def latent_weights(cfg, seed=0, clear_routing=True):
+    """Random weights, rounded to bfloat16.  clear_routing: the last channels of the residual hold values that only the
+    embedding writes, a few well separated levels per token, and the routers read nothing else - the choice of experts is never
+    close, whatever rounding does to a row."""
+    rng = np.random.default_rng(seed)
+    w, v = cfg["width"], cfg["vocab"]
+    W = {}
+
+    def mat(name, rows, cols, gain=1.0):
+        W[name] = gain * rng.standard_normal((rows, cols)) / np.sqrt(cols)
+
+    most = max([L["mlp"]["router"]["experts"] for L in cfg["layers"] if L["mlp"]], default=0) if clear_routing else 0
+    assert most < w
+    free = w - most  # channels sublayers may write
+    W["embed"] = rng.standard_normal((v, w))
+    for t in range(v if most else 0):
+        W["embed"][t, free:] = rng.permutation(np.linspace(-2.0, 2.0, most) if most > 1 else [1.0])
+    if cfg.get("loop"):
+        mat("loop.in", w, 2 * w, 1.2)
+        W["loop.in"][free:] = 0
+        for c in range(free, w):
+            W["loop.in"][c, c], W["loop.in"][c, w + c] = 0.75, 0.25
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        H, D, R, DV, C = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+        for n in "12" if L["mlp"] else "1":
+            W[p + "norm" + n] = 0.5 + rng.random(w)
+            W[p + f"norm{n}b"] = 0.5 + rng.random(w)
+            W[p + "ls" + n] = 0.3 + rng.random(w)
+        mat(p + "mix.q", H * (D + R), w)
+        mat(p + "mix.dkv", C + R, w)
+        W[p + "mix.dkv.norm"] = 0.5 + rng.random(C)
+        mat(p + "mix.uk", H * D, C)
+        mat(p + "mix.uv", H * DV, C)
+        W[p + "mix.sink"] = 1.5 + rng.standard_normal(H)
+        mat(p + "mix.g", H, w, 1.5)
+        mat(p + "mix.o", w, H * DV, 2.0)
+        W[p + "mix.o"][free:] = 0
+        if L["mlp"]:
+            E, ff = L["mlp"]["router"]["experts"], L["mlp"]["expert"]["ff"]
+            for e in range(E):
+                mat(p + f"mlp.e{e}.gate", ff, w, 1.5)
+                mat(p + f"mlp.e{e}.up", ff, w, 1.5)
+                mat(p + f"mlp.e{e}.down", w, ff, 2.0)
+                W[p + f"mlp.e{e}.down"][free:] = 0
+            mat(p + "mlp.router", E, w, 2.0)
+            if most:
+                W[p + "mlp.router"][:] = 0
+                W[p + "norm2"][free:] = 1.0
+                for e in range(E):
+                    W[p + "mlp.router"][e, free + e] = 1.5
+    W["final.norm"] = 0.5 + rng.random(w)
+    mat("head", v, w)
+    return {k: (P.to_bf16_bits(a).astype(np.uint32) << 16).view(np.float32).astype(np.float64) for k, a in W.items()}
+
+
+def latent_case(seed=0, clear_routing=True, **kw):
+    cfg = latent_config(**kw)
+    return cfg, latent_weights(cfg, seed, clear_routing)
+
+
 def write(path, cfg, W):
     os.makedirs(path, exist_ok=True)
     with open(os.path.join(path, "config.json"), "w") as f:
