@@ -573,7 +573,8 @@ def tensor_parallel_leg(lcu, n_gpus, K, W):
 
 
 # Block models at the sizes of real layers beside the LLaMA family at equal width, feed-forward and layer count: half of the
-# layers window-and-blocks attention with retention (grouped keys, stacked projection of about 3 x width rows), half wkv.
+# layers window-and-blocks attention with retention (grouped keys, stacked projection of about 3 x width rows), half wkv
+# (Filulix); latent attention with 8 experts of half the feed-forward, two of them per token (Zibovik).
 BLOCK_SIZES = {
     "1024": dict(width=1024, ff=2816, layers=8, heads=8, n_heads_llama=8),
     "2048": dict(width=2048, ff=5632, layers=8, heads=16, n_heads_llama=16),
@@ -595,8 +596,21 @@ def block_config(size, vocab=32000, window=1024, pool=16):
             "layers": [parallel if i % 2 == 0 else wkv for i in range(z["layers"])], "loop": None}
 
 
-def block_leg(lcu, size, K, W, profile=None):
-    """Decode and prompt throughput of a block model and of a LLaMA-shaped fp16 model of the same width, feed-forward, layer
+def latent_config(size, vocab=32000, window=1024, experts=8, top=2):
+    z = BLOCK_SIZES[size]
+    dim, rot = 128, 64
+    layer = {"type": "latent_attention",
+             "mixer": {"heads": z["heads"], "dim": dim, "rot_dim": rot, "vdim": dim, "kv_rank": min(512, z["width"] // 4), "mask": {"size": window},
+                       "rot": {"base": 10000.0, "dims": rot}, "scale": (dim + rot) ** -0.5},
+             "mlp": {"kind": "moe", "expert": {"ff": z["ff"] // top}, "router": {"experts": experts, "top": top}}}
+    return {"architecture": "Zibovik", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6}, "layers": [layer] * z["layers"]}
+
+
+BLOCK_MODELS = {"filulix": block_config, "zibovik": latent_config, "llama": None}
+
+
+def block_leg(lcu, size, K, W, profile=None, models=tuple(BLOCK_MODELS)):
+    """Decode and prompt throughput of the block models and of a LLaMA-shaped fp16 model of the same width, feed-forward, layer
     count and vocabulary, random weights, batch 1: decode as `K` device-chained greedy steps between CUDA events after a
     prompt of 128 and of 1900 tokens, prompts of 512 and 2000 tokens through next_token (host clock, median of 5)."""
     z = BLOCK_SIZES[size]
@@ -604,9 +618,9 @@ def block_leg(lcu, size, K, W, profile=None):
     out = {"size": size, "layers": z["layers"], "width": z["width"], "ff": z["ff"], "data": "synthetic", "steps": K}
     clk = ClockSampler(0)
     clk.start()
-    for name in ("filulix", "llama"):
-        if name == "filulix":
-            model = lcu.Model.from_config(block_config(size), seed=SEED, scale=SCALE)
+    for name in models:
+        if BLOCK_MODELS[name]:
+            model = lcu.Model.from_config(BLOCK_MODELS[name](size), seed=SEED, scale=SCALE)
         else:
             model = lcu.Model.synthetic(dim=z["width"], n_heads=z["n_heads_llama"], n_layers=z["layers"], n_vocab=32000, seed=SEED, scale=SCALE,
                                         multiple_of=256)
@@ -893,7 +907,8 @@ def main():
     ap.add_argument("--pipeline", type=int, default=1, help="single process: split the layers evenly over this many GPUs")
     ap.add_argument("--tp", type=int, default=0, help="single process: only the tensor-parallel leg (65B-shaped u8 model) over this many GPUs")
     ap.add_argument("--blocks", nargs="+", default=None, choices=sorted(BLOCK_SIZES), metavar="WIDTH",
-                    help="only the block-model leg: Filulix beside a LLaMA-shaped model at these widths (1024, 2048, 4096)")
+                    help="only the block-model leg: Filulix, Zibovik and a LLaMA-shaped model at these widths (1024, 2048, 4096)")
+    ap.add_argument("--block-models", nargs="+", default=list(BLOCK_MODELS), choices=sorted(BLOCK_MODELS), help="models of the block-model leg")
     ap.add_argument("--profile", nargs="?", const="decode", default=None, choices=["decode", "prefill"],
                     help="cudaProfilerStart/Stop around the device-chained timed region (decode) or around the prompt pass and GEMM (prefill)")
     args = ap.parse_args()
@@ -904,7 +919,7 @@ def main():
     os.dup2(2, 1)
     if args.blocks:
         lcu = load_package()
-        emit({"blocks": [block_leg(lcu, size, args.steps, args.warmup, args.profile) for size in args.blocks]})
+        emit({"blocks": [block_leg(lcu, size, args.steps, args.warmup, args.profile, args.block_models) for size in args.blocks]})
     elif args.tp > 1:
         lcu = load_package()
         emit({"tensor_parallel": tensor_parallel_leg(lcu, args.tp, args.steps, args.warmup)})

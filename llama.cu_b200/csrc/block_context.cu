@@ -37,7 +37,7 @@ struct run_cache {  // of one layer run
 // a sublayer result in y that the residual has not taken in yet
 struct pending_result {
   const hyper_weights* streams = nullptr;            // null: nothing is pending
-  const float *post = nullptr, *scale = nullptr;     // output norm and channel scale
+  const float* post = nullptr;                       // output norm and channel scale
   const int* pieces = nullptr;                       // rows of y that make up a row's result [row][n_pieces]
   int n_pieces = 0;
 };
@@ -147,7 +147,6 @@ int block_context<T>::residual(hyper_params<T>& p, const pending_result& done, i
     p.up_mix = done.streams->mix;
     p.up_out = done.streams->out;
     p.post_w = done.post;
-    p.post_scale = done.scale;
     p.n_y = done.n_pieces;
   }
   ++launches;
@@ -396,12 +395,28 @@ int block_context<T>::mixer_one(int run) {
     LCU_TRY(product(proj, false, h, K, L.proj, 1, L.proj_rows, K));
   }
   mixer_step<T> st{};
-  st.n_branches = (int)ls.branches.size();
-  LCU_REQUIRE(st.n_branches <= STEP_MAX_BRANCHES, "mixer with %d branches", st.n_branches);
-  for (int i = 0; i < st.n_branches; ++i) {
+  for (int i = 0; i < (int)ls.branches.size(); ++i) {
     const branch_spec& bs = ls.branches[i];
     const branch_weights& bw = L.branches[i];
-    step_branch<T>& b = st.b[i];
+    if (bs.kind == BRANCH_LATENT_ATTN) {
+      latent_step<T> a{};
+      a.rows = latents(run, i, L.proj_rows);
+      a.up = (const T*)bw.up;
+      a.ld_up = bw.up_k;
+      a.up_v = bw.up_v;
+      a.scale = bs.score_scale;
+      a.out_scale = bs.out_scale;
+      a.sink = bs.sink ? bw.sink : nullptr;
+      a.gate = bs.head_gate ? proj + bw.g : nullptr;
+      a.out = cat + bw.out_col;
+      a.pos = gpus[0].state;
+      a.err = err();
+      ++launches;
+      LCU_TRY(launch_latent_step(a, stream()));
+      continue;
+    }
+    LCU_REQUIRE(st.n_branches < STEP_MAX_BRANCHES, "mixer with more than %d branches", STEP_MAX_BRANCHES);
+    step_branch<T>& b = st.b[st.n_branches++];
     b.kind = bs.kind;
     b.first = st.n_clusters;
     st.n_clusters += bs.heads;
@@ -410,15 +425,6 @@ int block_context<T>::mixer_one(int run) {
     b.out = cat + bw.out_col;
     if (bs.kind == BRANCH_WINDOW_ATTN) {
       b.attn = attention(run, i, L.proj_rows);
-    } else if (bs.kind == BRANCH_LATENT_ATTN) {
-      b.latent = latents(run, i, L.proj_rows);
-      b.up = (const T*)bw.up;
-      b.ld_up = bw.up_k;
-      b.up_v = bw.up_v;
-      b.attn.scale = bs.score_scale;
-      b.attn.out_scale = bs.out_scale;
-      b.attn.sink = bs.sink ? bw.sink : nullptr;
-      b.attn.gate = bs.head_gate ? proj + bw.g : nullptr;
     } else {
       b.scan = recurrence(run, i, L.proj_rows);
       if (bs.kind == BRANCH_WKV) {
@@ -433,9 +439,11 @@ int block_context<T>::mixer_one(int run) {
       }
     }
   }
-  st.pos = gpus[0].state;
-  ++launches;
-  LCU_TRY(launch_mixer_step(st, opt.context_len, stream()));
+  if (st.n_branches > 0) {
+    st.pos = gpus[0].state;
+    ++launches;
+    LCU_TRY(launch_mixer_step(st, opt.context_len, stream()));
+  }
   return product(y, true, cat, L.out_k, L.out, 1, m->n_width, L.out_k);
 }
 
@@ -463,7 +471,12 @@ template <typename T>
 int block_context<T>::expert_rows(const layer_spec& ls, const block_layer& L, int rows, pending_result& done) {
   const expert_weights& x = L.experts;
   const int K = m->k_width, f = L.ff_pad, total = rows * ls.top;
-  LCU_TRY(product(z, true, h, K, x.router, rows, x.router_rows, K));
+  if (is_f32<T>() || rows == 1) {
+    LCU_TRY(product(z, true, h, K, x.router, rows, x.router_rows, K));
+  } else {  // (one narrow matrix: K split over clusters fills more SMs than a few tiles of SM pairs)
+    ++launches;
+    LCU_TRY(launch_gemm_tc(TC_BF16_F32, z, h, K, x.router, rows, x.router_rows, K, 0.f, err(), stream(), 0, 0));
+  }
   route_rows<T> r{};
   r.z = z;
   r.ldz = x.router_rows;
@@ -548,18 +561,12 @@ int block_context<T>::layers(int rows, int pos0, pending_result& done) {
     LCU_TRY(hyper(L.hc1, L.norm1, done, rows, step && ls.is_wkv() ? &L : nullptr, runs[run].prev, nullptr, nullptr));
     LCU_TRY(step ? mixer_one((int)run) : mixer_rows((int)run, rows, pos0));
     done = pending_result{&L.hc1};
-    if (sandwich) {
-      done.post = L.norm1b;
-      done.scale = L.scale1;
-    }
+    if (sandwich) done.post = L.norm1b;
     if (ls.ff > 0) {
       const bool fused_pick = step && ls.experts > 0 && !is_f32<T>();
       LCU_TRY(hyper(L.hc2, L.norm2, done, rows, nullptr, nullptr, fused_pick ? &ls : nullptr, &L));
       done = pending_result{&L.hc2};
-      if (sandwich) {
-        done.post = L.norm2b;
-        done.scale = L.scale2;
-      }
+      if (sandwich) done.post = L.norm2b;
       if (fused_pick) LCU_TRY(expert_one(ls, L, done));
       else if (ls.experts > 0) LCU_TRY(expert_rows(ls, L, rows, done));
       else LCU_TRY(feed_forward(L, rows));

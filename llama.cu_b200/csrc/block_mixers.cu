@@ -53,8 +53,8 @@ __host__ __device__ __forceinline__ int query_cols(const attn_rows<T>& p) {
   return (p.dim + 7) / 8 * 8 + (p.key2 ? (p.dim2 + 7) / 8 * 8 : 0);
 }
 // `rank` of `C` CTAs takes a slice of the visible keys.  The row's own key and value come from `cur_k` / `cur_v` (shared
-// memory copies) when given, else from the cache.  q_row null: q holds the query already.  Leaves max, sum and the
-// unnormalised value row in res[0], res[1], res[2 ..].  Shared memory: q [query_cols], scores [slice], part [PART_FLOATS].
+// memory copies) when given, else from the cache.  Leaves max, sum and the unnormalised value row in res[0], res[1],
+// res[2 ..].  Shared memory: q [query_cols], scores [slice], part [PART_FLOATS].
 template <typename T>
 __device__ void attend_slice(const attn_rows<T>& p, const T* q_row, int head, int pos, int rank, int C, const T* cur_k, const T* cur_v, float* q,
                              float* sc, float* part, float* red, float* res) {
@@ -71,8 +71,7 @@ __device__ void attend_slice(const attn_rows<T>& p, const T* q_row, int head, in
   window_of(pos, p.window, p.pool, lo, blocks);
   const int total = blocks + pos + 1 - lo;
   const int t0 = (int)((long long)total * rank / C), n = (int)((long long)total * (rank + 1) / C) - t0;
-  if (q_row)
-    for (int d = tid; d < q_cols; d += MX_THREADS) q[d] = d < p.dim || p.key2 ? to_f(q_row[head * p.q_head + d]) : 0.f;
+  for (int d = tid; d < q_cols; d += MX_THREADS) q[d] = d < p.dim || p.key2 ? to_f(q_row[head * p.q_head + d]) : 0.f;
   __syncthreads();
   auto key_at = [&](int t) -> const T* {
     if (t < blocks) return kp + (size_t)t * ldk;
@@ -554,130 +553,6 @@ __device__ void step_attention(const step_branch<T>& b, int head, int rank, int 
   cluster_sync();
 }
 
-// Latent attention of one token and head without forming keys or values: the query is taken through the head's key matrix
-// once (the CTAs share its columns), so that a key is a cache row and the result a sum of cache rows, which the head's value
-// matrix turns into the output (the CTAs share its rows).  All of it in binary32 but for the cache rows.
-template <typename T>
-size_t latent_step_floats(const latent_rows<T>& p) {
-  return 3 * (size_t)p.cache.ld + round_up(p.dim, 8) + p.cache.rot + 2 + round_up(p.kv_rank + 2, 4) + PART_FLOATS;
-}
-template <typename T>
-__device__ void step_latent(const step_branch<T>& b, int head, int rank, int pos, float* sm, float* red) {
-  const latent_rows<T>& p = b.latent;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int ld = p.cache.ld, rp = p.cache.rot, kp = round_up_dev(p.dim, 8), rotp = ld - rp, vp = round_up_dev(p.vdim, 8), half = p.rot_dims >> 1;
-  struct __align__(16) vec8 { T e[8]; };
-  T* cur = reinterpret_cast<T*>(sm);  // [ld] the token's row as the cache will hold it
-  float* q = sm + ld;                 // [ld] query against cache rows
-  float* oc = q + ld;                 // [rp] sum of cache rows
-  float* qh = oc + rp;                // [kp] query against the head's unrotated keys
-  float* part = qh + kp;
-  float* res = part + PART_FLOATS;
-  float* sc = res + 2 + round_up_dev(p.kv_rank + 2, 4);
-  const T* q_row = p.q + (size_t)head * (kp + rotp);
-  float ss = 0.f;
-  for (int d = tid; d < rp; d += MX_THREADS) {
-    const float x = d < p.kv_rank ? to_f(p.c[d]) : 0.f;
-    oc[d] = x;
-    ss = fmaf(x, x, ss);
-  }
-  for (int d = tid; d < kp; d += MX_THREADS) qh[d] = to_f(q_row[d]);
-  for (int d = tid; d < rotp; d += MX_THREADS) {
-    float kv = d < p.rot_dim ? to_f(p.k[d]) : 0.f, qv = to_f(q_row[kp + d]);
-    if (d < p.rot_dims) {
-      const float2 cs = p.rope[(size_t)pos * half + (d >> 1)];
-      const float sn = d & 1 ? cs.y : -cs.y;
-      kv = kv * cs.x + to_f(p.k[d ^ 1]) * sn;
-      qv = qv * cs.x + to_f(q_row[kp + (d ^ 1)]) * sn;
-    }
-    cur[rp + d] = from_f<T>(kv);
-    q[rp + d] = qv;
-  }
-  ss = block_sum(ss, red);
-  const float inv_c = 1.0f / sqrtf(ss / (float)p.kv_rank + p.eps);
-  for (int d = tid; d < rp; d += MX_THREADS) cur[d] = from_f<T>(d < p.kv_rank ? oc[d] * inv_c * p.norm[d] : 0.f);
-  __syncthreads();
-  if (head == 0 && rank == 0)
-    for (int d = tid; d < ld; d += MX_THREADS) p.cache.rows[(size_t)pos * ld + d] = cur[d];
-  // this CTA's columns of the query against latents, in vectors of 8
-  const int vecs = rp >> 3, v0 = vecs * rank / ST_CLUSTER, nv = vecs * (rank + 1) / ST_CLUSTER - v0;
-  if (nv > 0) {
-    const int ng = min(MX_THREADS / nv, 32), grp = tid / nv, j = tid - grp * nv;
-    if (grp < ng) {
-      float acc[8] = {};
-      const T* w = b.up + (size_t)head * kp * b.ld_up + (v0 + j) * 8;
-#pragma unroll 4
-      for (int d = grp; d < p.dim; d += ng) {
-        const vec8 x = *reinterpret_cast<const vec8*>(w + (size_t)d * b.ld_up);
-        const float qd = qh[d];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] = fmaf(qd, to_f(x.e[e]), acc[e]);
-      }
-#pragma unroll
-      for (int e = 0; e < 8; ++e) part[(grp * nv + j) * 8 + e] = acc[e];
-    }
-    __syncthreads();
-    for (int i = tid; i < nv * 8; i += MX_THREADS) {
-      float a = 0.f;
-      for (int g = 0; g < ng; ++g) a += part[g * nv * 8 + i];
-      q[v0 * 8 + i] = a;
-    }
-  }
-  cluster_sync();
-  for (int i = tid; i < rp; i += MX_THREADS) {
-    const int owner = ((i >> 3) * ST_CLUSTER + ST_CLUSTER - 1) / vecs;  // whose vectors hold column i
-    if (owner != rank) q[i] = ld_dsmem_f32(mapa(smem_u32(q + i), owner));
-  }
-  attn_rows<T> a{};
-  a.cache.k = a.cache.v = p.cache.rows;
-  a.cache.ldk = a.cache.ldv = ld;
-  a.heads = a.kv_heads = 1;
-  a.dim = ld;
-  a.vdim = p.kv_rank;
-  a.window = p.window;
-  a.scale = b.attn.scale;
-  attend_slice(a, (const T*)nullptr, 0, pos, rank, ST_CLUSTER, cur, cur, q, sc, part, red, res);
-  cluster_sync();
-  float mx = b.attn.sink ? b.attn.sink[head] : -CUDART_INF_F, sum = 0.f, f[ST_CLUSTER];
-#pragma unroll
-  for (int r = 0; r < ST_CLUSTER; ++r) {
-    f[r] = ld_dsmem_f32(mapa(smem_u32(res), r));
-    mx = fmaxf(mx, f[r]);
-  }
-#pragma unroll
-  for (int r = 0; r < ST_CLUSTER; ++r) {
-    f[r] = f[r] > -CUDART_INF_F ? expf(f[r] - mx) : 0.f;
-    sum = fmaf(f[r], ld_dsmem_f32(mapa(smem_u32(res + 1), r)), sum);
-  }
-  if (b.attn.sink) sum += expf(b.attn.sink[head] - mx);
-  float out_scale = b.attn.out_scale / sum;
-  if (b.attn.gate) out_scale *= sigmoid_f(to_f(b.attn.gate[head]));
-  for (int d = tid; d < rp; d += MX_THREADS) {
-    float v = 0.f;
-    if (d < p.kv_rank) {
-#pragma unroll
-      for (int r = 0; r < ST_CLUSTER; ++r)
-        if (f[r] > 0.f) v = fmaf(f[r], ld_dsmem_f32(mapa(smem_u32(res + 2 + d), r)), v);
-    }
-    oc[d] = v;
-  }
-  __syncthreads();
-  const int j1 = p.vdim * (rank + 1) / ST_CLUSTER;
-  for (int j = p.vdim * rank / ST_CLUSTER + warp; j < j1; j += MX_THREADS / 32) {
-    const T* w = b.up + ((size_t)b.up_v + (size_t)head * vp + j) * b.ld_up;
-    float v = 0.f;
-#pragma unroll 2
-    for (int d = lane * 8; d < rp; d += 256) {
-      const vec8 x = *reinterpret_cast<const vec8*>(w + d);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) v = fmaf(oc[d + e], to_f(x.e[e]), v);
-    }
-    v = warp_sum(v);
-    if (lane == 0) b.out[head * p.vdim + j] = from_f<T>(v * out_scale);
-  }
-  cluster_sync();
-}
-
 template <typename T, bool WKV>
 __device__ void step_recurrence(const step_branch<T>& b, int head, int rank, int pos, float* sm, float* red) {
   const scan_rows<T>& p = b.scan;
@@ -793,23 +668,6 @@ __device__ __forceinline__ void step_lines(const step_branch<T>& b, int head, in
       const T* base = key ? (pooled ? p.cache.kp : p.cache.k) : (pooled ? p.cache.vp : p.cache.v);
       l2_line(base + row * (key ? p.cache.ldk : p.cache.ldv) + (key ? l : l - lk) * LINE);
     }
-  } else if (b.kind == BRANCH_LATENT_ATTN) {
-    const latent_rows<T>& p = b.latent;
-    const int pos = min(*(volatile const int*)pos_ptr, p.cache.ctx_len - 1);
-    int lo, blocks;
-    window_of(pos, p.window, 0, lo, blocks);
-    constexpr int LINE = 128 / sizeof(T);
-    const int ld = p.cache.ld, rp = p.cache.rot, kp = round_up_dev(p.dim, 8), vp = round_up_dev(p.vdim, 8), total = pos + 1 - lo;
-    // the head's matrices: this CTA's columns of the first, rows of the second
-    const int c0 = (rp >> 3) * rank / ST_CLUSTER * 8, c1 = (rp >> 3) * (rank + 1) / ST_CLUSTER * 8, lc = (c1 - c0 + LINE - 1) / LINE;
-    for (int i = tid; i < p.dim * lc; i += MX_THREADS)
-      l2_line(b.up + ((size_t)head * kp + i / lc) * b.ld_up + min(c0 + i % lc * LINE, rp - 1));
-    const int j0 = p.vdim * rank / ST_CLUSTER, j1 = p.vdim * (rank + 1) / ST_CLUSTER, lr = (rp + LINE - 1) / LINE;
-    for (int i = tid; i < (j1 - j0) * lr; i += MX_THREADS) l2_line(b.up + ((size_t)b.up_v + (size_t)head * vp + j0 + i / lr) * b.ld_up + i % lr * LINE);
-    // the heads share the cache rows of this CTA's slice
-    const int t0 = (int)((long long)total * rank / ST_CLUSTER), n = (int)((long long)total * (rank + 1) / ST_CLUSTER) - t0;
-    const int lk = (ld + LINE - 1) / LINE, heads = p.heads;
-    for (int i = tid + MX_THREADS * head; i < n * lk; i += MX_THREADS * heads) l2_line(p.cache.rows + (size_t)(lo + t0 + i / lk) * ld + min(i % lk * LINE, ld - 1));
   } else {
     const scan_rows<T>& p = b.scan;
     const int v0 = p.vdim * rank / ST_CLUSTER, nv = p.vdim * (rank + 1) / ST_CLUSTER - v0;
@@ -841,7 +699,6 @@ __global__ void __launch_bounds__(MX_THREADS) mixer_step_kernel(const __grid_con
   pdl_wait();
   const int pos = *p.pos;
   if (b.kind == BRANCH_WINDOW_ATTN) step_attention(b, head, rank, pos, sm, red);
-  else if (b.kind == BRANCH_LATENT_ATTN) step_latent(b, head, rank, pos, sm, red);
   else if (b.kind == BRANCH_RETENTION) step_recurrence<T, false>(b, head, rank, pos, sm, red);
   else step_recurrence<T, true>(b, head, rank, pos, sm, red);
 }
@@ -921,7 +778,6 @@ int launch_mixer_step(const mixer_step<T>& p, int ctx_len, cudaStream_t stream) 
   for (int i = 0; i < p.n_branches; ++i) {
     const step_branch<T>& b = p.b[i];
     if (b.kind == BRANCH_WINDOW_ATTN) smem = std::max(smem, attention_smem(b.attn, most_keys(b.attn, ctx_len - 1) / ST_CLUSTER + 2, true));
-    else if (b.kind == BRANCH_LATENT_ATTN) smem = std::max(smem, (latent_step_floats(b.latent) + std::min(b.latent.window, ctx_len) / ST_CLUSTER + 8) * sizeof(float));
     else smem = std::max(smem, (3 * (size_t)b.scan.dim + MX_THREADS + b.rank + 8) * sizeof(float));
   }
   LCU_REQUIRE(smem <= 220 * 1024, "mixer step: %zu bytes of shared memory", smem);

@@ -74,7 +74,7 @@ int block_model::create(std::unique_ptr<block_model>& out, const block_spec& spe
           vec(bw.sink, bs.heads);
           vec(bw.latent_norm, bs.kv_rank);
           bw.up_v = bs.heads * bs.dim_pad();
-          bw.up_rows = pad_rows(bw.up_v + bs.heads * bs.vdim_pad());
+          bw.up_rows = pad_stack(bw.up_v + bs.heads * bs.vdim_pad());
           bw.up_k = pad_k(bs.kv_rank);
           mat(bw.up, bw.up_rows, bw.up_k);
           continue;
@@ -103,7 +103,7 @@ int block_model::create(std::unique_ptr<block_model>& out, const block_spec& spe
         vec(L.u, ch);
         vec(L.head_norm, ch);
       } else {
-        L.proj_rows = pad_rows(rows);
+        L.proj_rows = pad_stack(rows);
         mat(L.proj, L.proj_rows, m->k_width);
       }
       L.out_k = pad_k(cols);
@@ -284,6 +284,16 @@ int block_model::set_default(const slot& s) {
   return LCU_OK;
 }
 
+// every output norm and the channel scale behind it become one factor (products of two bfloat16 values are exact)
+int block_model::fold_scales() {
+  for (auto& L : layers) {
+    if (L.scale1) LCU_TRY(launch_scale_vector(L.norm1b, L.scale1, spec.width, 0));
+    if (L.scale2) LCU_TRY(launch_scale_vector(L.norm2b, L.scale2, spec.width, 0));
+  }
+  LCU_CUDA(cudaDeviceSynchronize());
+  return LCU_OK;
+}
+
 int block_model::fill_synthetic(uint64_t seed, float scale) {
   device_guard g(device);
   size_t most = 0;
@@ -312,7 +322,7 @@ int block_model::fill_synthetic(uint64_t seed, float scale) {
   cudaFree(wide);
   if (rc) return rc;
   LCU_CUDA(e);
-  return LCU_OK;
+  return fold_scales();
 }
 
 int block_model::load(std::unique_ptr<block_model>& out, const std::string& dir, block_dtype dtype) {
@@ -370,6 +380,7 @@ int block_model::load(std::unique_ptr<block_model>& out, const std::string& dir,
   }
   if (!rc) rc = loader.finish();
   cudaFree(tmp);
+  if (!rc) rc = m->fold_scales();
   if (rc) return rc;
   out = std::move(m);
   return LCU_OK;

@@ -13,6 +13,7 @@ enum block_dtype : int { BLOCK_BF16 = 0, BLOCK_F32 = 1 };
 // Matrices are stored [rows][K] with rows padded to a multiple of 128 and K to a multiple of 256 (zeros), so that every
 // size takes the same product kernels; matrices that share an input are stacked.
 constexpr int pad_rows(int n) { return (n + 127) / 128 * 128; }
+constexpr int pad_stack(int n) { return n > 2048 ? (n + 255) / 256 * 256 : pad_rows(n); }  // long stacks: whole tiles of SM pairs
 constexpr int pad_k(int k) { return (k + 255) / 256 * 256; }
 
 struct hyper_weights {
@@ -39,7 +40,8 @@ struct expert_weights {
 };
 struct block_layer {
   float *norm1 = nullptr, *norm2 = nullptr;
-  float *norm1b = nullptr, *norm2b = nullptr, *scale1 = nullptr, *scale2 = nullptr;  // of a sublayer's result
+  float *norm1b = nullptr, *norm2b = nullptr;  // of a sublayer's result, times its channel scale once the weights are in place
+  float *scale1 = nullptr, *scale2 = nullptr;
   hyper_weights hc1, hc2;
   std::vector<branch_weights> branches;
   // branches that read the row itself: one stacked projection
@@ -98,6 +100,7 @@ struct block_model : model_base {
   };
   std::vector<slot> slots() const;
   int set_default(const slot& s);
+  int fold_scales();
 };
 
 }  // namespace lcu

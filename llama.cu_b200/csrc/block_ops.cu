@@ -74,7 +74,6 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
     for (int i = 32 * tid; i < n; i += 32 * HY_THREADS) {
       if (p.norm_w) l2_line(p.norm_w + first + i);
       if (PRE && p.post_w) l2_line(p.post_w + first + i);
-      if (PRE && p.post_scale) l2_line(p.post_scale + first + i);
       if (p.mix)
         for (int k = 0; k < p.n_mix; ++k) l2_line(p.mu + (size_t)k * p.width + first + i);
     }
@@ -109,13 +108,15 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
     }
     return t;
   };
+  constexpr int KEEP = PRE && SM == 1 ? (CL > 1 ? 1 : 4) : 0;  // vectors of the residual row held per thread from the start
+  float4 kept[KEEP > 0 ? KEEP : 1];
   float inv_y = 1.f;
   if (PRE && y) {  // (a thread reads back only columns it has written itself)
     const int* yr = p.y_rows ? p.y_rows + (size_t)row * p.n_y : nullptr;
     const int pieces = yr ? p.n_y : 1;
     float sy = 0.f;
     if ((W & 3) == 0) {
-      for (int c = c0 + 4 * tid; c < c1; c += 4 * HY_THREADS) {
+      auto gather4 = [&](int c) {
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
         for (int k = 0; k < pieces; ++k) {
           const float4 v = *reinterpret_cast<const float4*>(y + (yr ? (size_t)yr[k] * p.ldy : 0) + c);
@@ -123,7 +124,18 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
         }
         *reinterpret_cast<float4*>(u_row + c - c0) = a;
         sy = fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(a.z, a.z, fmaf(a.w, a.w, sy))));
+      };
+#pragma unroll
+      for (int i = 0; i < KEEP; ++i) {  // the residual's columns are on their way meanwhile
+        const int c = c0 + 4 * (tid + i * HY_THREADS);
+        kept[i] = c < c1 ? *reinterpret_cast<const float4*>(x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
       }
+#pragma unroll
+      for (int i = 0; i < KEEP; ++i) {
+        const int c = c0 + 4 * (tid + i * HY_THREADS);
+        if (c < c1) gather4(c);
+      }
+      for (int c = c0 + 4 * (tid + KEEP * HY_THREADS); c < c1; c += 4 * HY_THREADS) gather4(c);
     } else {
       for (int c = c0 + tid; c < c1; c += HY_THREADS) {
         float a = 0.f;
@@ -136,8 +148,7 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
   }
   auto y_at = [&](int c, float v) {  // PRE: the column's part in the sum
     if (!PRE || !p.post_w) return v;
-    v *= inv_y * p.post_w[c];
-    return p.post_scale ? v * p.post_scale[c] : v;
+    return v * (inv_y * p.post_w[c]);
   };
   float ss = 0.f;
   auto column = [&](float (&v)[SM], float yv) {  // new streams in v, returns u
@@ -158,31 +169,42 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
     for (int s = 0; s < SM; ++s) u = fmaf(in[s], v[s], u);
     return u;
   };
-  if ((W & 3) == 0) {  // (per is a multiple of 4: rows and slices start 16-byte aligned)
-    for (int c = c0 + 4 * tid; c < c1; c += 4 * HY_THREADS) {
+  auto columns4 = [&](int c, float4 (&xv)[SM]) {  // (per is a multiple of 4: rows and slices start 16-byte aligned)
+    float4 yv = y ? *reinterpret_cast<const float4*>(PRE ? u_row + c - c0 : y + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (PRE && y) yv = make_float4(y_at(c, yv.x), y_at(c + 1, yv.y), y_at(c + 2, yv.z), y_at(c + 3, yv.w));
+    float4 u;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float v[SM];
+#pragma unroll
+      for (int s = 0; s < SM; ++s) v[s] = reinterpret_cast<const float*>(&xv[s])[e];
+      const float ue = column(v, reinterpret_cast<const float*>(&yv)[e]);
+      reinterpret_cast<float*>(&u)[e] = ue;
+      ss = fmaf(ue, ue, ss);
+#pragma unroll
+      for (int s = 0; s < SM; ++s) reinterpret_cast<float*>(&xv[s])[e] = v[s];
+    }
+    *reinterpret_cast<float4*>(u_row + c - c0) = u;
+    if (y && p.store) {
+#pragma unroll
+      for (int s = 0; s < SM; ++s)
+        if (s < S) *reinterpret_cast<float4*>(x + (size_t)s * W + c) = xv[s];
+    }
+  };
+  if ((W & 3) == 0) {
+    if (y) {
+#pragma unroll
+      for (int i = 0; i < KEEP; ++i) {
+        const int c = c0 + 4 * (tid + i * HY_THREADS);
+        float4 xv[SM] = {kept[i]};
+        if (c < c1) columns4(c, xv);
+      }
+    }
+    for (int c = c0 + 4 * (tid + (y ? KEEP * HY_THREADS : 0)); c < c1; c += 4 * HY_THREADS) {
       float4 xv[SM];
 #pragma unroll
       for (int s = 0; s < SM; ++s) xv[s] = s < S ? *reinterpret_cast<const float4*>(x + (size_t)s * W + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-      float4 yv = y ? *reinterpret_cast<const float4*>(PRE ? u_row + c - c0 : y + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-      if (PRE && y) yv = make_float4(y_at(c, yv.x), y_at(c + 1, yv.y), y_at(c + 2, yv.z), y_at(c + 3, yv.w));
-      float4 u;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        float v[SM];
-#pragma unroll
-        for (int s = 0; s < SM; ++s) v[s] = reinterpret_cast<const float*>(&xv[s])[e];
-        const float ue = column(v, reinterpret_cast<const float*>(&yv)[e]);
-        reinterpret_cast<float*>(&u)[e] = ue;
-        ss = fmaf(ue, ue, ss);
-#pragma unroll
-        for (int s = 0; s < SM; ++s) reinterpret_cast<float*>(&xv[s])[e] = v[s];
-      }
-      *reinterpret_cast<float4*>(u_row + c - c0) = u;
-      if (y && p.store) {
-#pragma unroll
-        for (int s = 0; s < SM; ++s)
-          if (s < S) *reinterpret_cast<float4*>(x + (size_t)s * W + c) = xv[s];
-      }
+      columns4(c, xv);
     }
   } else {
     for (int c = c0 + tid; c < c1; c += HY_THREADS) {
@@ -202,7 +224,25 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
   const float inv = 1.0f / sqrtf(row_total(ss, 1) / (float)W + p.eps);
   T* h = p.h + (size_t)i_row * p.ldh;
   const bool start = p.mix && *p.pos == 0;
-  for (int c = c0 + tid; c < c1; c += HY_THREADS) {
+  if ((W & 3) == 0 && !p.mix) {  // (a thread's own columns)
+    struct __align__(4 * sizeof(T)) pack { T e[4]; };
+#pragma unroll 4
+    for (int c = c0 + 4 * tid; c < c1; c += 4 * HY_THREADS) {
+      const float4 u = *reinterpret_cast<const float4*>(u_row + c - c0);
+      if (p.u_out) *reinterpret_cast<float4*>(p.u_out + (size_t)i_row * W + c) = u;
+      const float4 w = p.norm_w ? *reinterpret_cast<const float4*>(p.norm_w + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      pack o;
+      float4 back;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float ue = reinterpret_cast<const float*>(&u)[e];
+        o.e[e] = from_f<T>(p.norm_w ? ue * inv * (p.norm_base + reinterpret_cast<const float*>(&w)[e]) : ue);
+        reinterpret_cast<float*>(&back)[e] = to_f(o.e[e]);
+      }
+      *reinterpret_cast<pack*>(h + c) = o;
+      if (CL > 1 && p.router) *reinterpret_cast<float4*>(u_row + c - c0) = back;
+    }
+  } else for (int c = c0 + tid; c < c1; c += HY_THREADS) {
     const float u = u_row[c - c0];
     if (p.u_out) p.u_out[(size_t)i_row * W + c] = u;
     const T hv = from_f<T>(p.norm_w ? u * inv * (p.norm_base + p.norm_w[c]) : u);
@@ -632,6 +672,16 @@ int launch_place(T* dst, int ld, const void* src, place_source type, int rows, i
   const size_t n = (size_t)rows * cols;
   if (n == 0) return LCU_OK;
   place_kernel<T><<<(unsigned)std::min<size_t>(ceil_div(n, 256), 148 * 16), 256, 0, stream>>>(dst, ld, src, type == PLACE_F32, rows, cols, transpose, groups);
+  LCU_CUDA(cudaGetLastError());
+  return LCU_OK;
+}
+
+__global__ void scale_vector_kernel(float* dst, const float* src, int n) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) dst[i] *= src[i];
+}
+int launch_scale_vector(float* dst, const float* src, int n, cudaStream_t stream) {
+  scale_vector_kernel<<<(n + 255) / 256, 256, 0, stream>>>(dst, src, n);
   LCU_CUDA(cudaGetLastError());
   return LCU_OK;
 }

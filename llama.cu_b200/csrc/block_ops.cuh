@@ -33,7 +33,7 @@ int launch_block_embed(const embed_params<T>& p, cudaStream_t stream);
 
 // One pass over residual rows between two sublayers:
 //   y <- sum_k y[y_rows[row][k]]                     (optional: a result that lies in pieces)
-//   y <- y / sqrt(mean(y^2) + eps) * post_w * post_scale      (optional: a sublayer's output norm and channel scale)
+//   y <- y / sqrt(mean(y^2) + eps) * post_w          (optional: a sublayer's output norm, its channel scale included)
 //   x_t <- sum_s up_mix[s][t] x_s + up_out[t] y      (the sublayer just computed; skipped when y is null)
 //   u = sum_s in[s] x_s;  h = u / sqrt(mean(u^2) + eps) * (norm_base + norm_w)    (the norm of the next one; without norm_w h = u)
 // and, for a single row, what follows at once: the inputs mix_i = h + (h_prev - h) * mu_i of a token-shifted mixer, with
@@ -49,7 +49,7 @@ struct hyper_params {
   const float* in;
   const float* norm_w;
   float norm_base, eps;
-  const float *post_w, *post_scale;
+  const float* post_w;
   const int* y_rows;     // [rows][n_y]
   int n_y;
   const int* rows;       // row numbers to work on, or null: 0 .. n-1; results are dense
@@ -140,10 +140,27 @@ struct latent_rows {
   int ld_staged;
 };
 // first position that row `pos0` of a pass sees
-inline int window_first(int pos0, int window) { return pos0 + 1 > window ? pos0 + 1 - window : 0; }
+__host__ __device__ inline int window_first(int pos0, int window) { return pos0 + 1 > window ? pos0 + 1 - window : 0; }
 // norm and rotation of m new rows, into the cache; staged[i] = latent of position window_first(pos0) + i
 template <typename T>
 int launch_latent_rows(const latent_rows<T>& p, int m, int pos0, cudaStream_t stream);
+
+// One token in one launch, without forming keys or values: a query goes through its head's key matrix once, so that a key is a
+// cache row and the result a sum of cache rows, which the head's value matrix turns into the output.
+template <typename T>
+struct latent_step {
+  latent_rows<T> rows;   // of the token; staged is not used
+  const T* up;           // [heads * dim_pad | heads * vdim_pad][ld_up]: keys and values of all heads from a latent
+  int ld_up, up_v;       // up_v: first value row
+  float scale, out_scale;
+  const float* sink;     // as attn_rows
+  const T* gate;
+  T* out;                // [heads * vdim]
+  const int* pos;
+  int* err;
+};
+template <typename T>
+int launch_latent_step(const latent_step<T>& p, cudaStream_t stream);
 
 // ---- linear recurrences over rows, per head:
 //   retention: S <- decay S + k v^T, o = S^T q          (k and q rotated, k times kscale)
@@ -184,10 +201,7 @@ template <typename T>
 struct step_branch {
   int kind;               // branch_kind
   int first;              // first cluster of the launch
-  attn_rows<T> attn;      // attention (row pointers: the token's row); latent attention: heads, window, scale, sink, gate
-  latent_rows<T> latent;  // latent attention, with its matrix from latents to keys and values
-  const T* up;            // [heads * dim_pad | heads * vdim_pad][ld_up]
-  int ld_up, up_v;        // up_v: first value row
+  attn_rows<T> attn;      // attention (row pointers: the token's row)
   scan_rows<T> scan;      // recurrences
   const T* g;             // gate projection of the token
   const float* low;       // wkv: input of the decay's second product
@@ -242,6 +256,9 @@ struct row_groups {
 template <typename T>
 int launch_place(T* dst, int ld, const void* src, place_source type, int rows, int cols, bool transpose, cudaStream_t stream,
                  const row_groups& groups = row_groups{});
+
+// dst[i] *= src[i]
+int launch_scale_vector(float* dst, const float* src, int n, cudaStream_t stream);
 
 // ---- binary32 products: out[m][N] = x[m][ldx] . w[N][K]^T
 int launch_matmul_f32(float* out, const float* x, int ldx, const float* w, int m, int N, int K, cudaStream_t stream);

@@ -41,7 +41,7 @@ __global__ void __launch_bounds__(ROUTE_THREADS) route_pick_kernel(const route_r
 template <typename T>
 __global__ void __launch_bounds__(ROUTE_THREADS) route_place_kernel(const route_rows<T> p, int chunks) {
   extern __shared__ int r_sm[];  // first [E]: the chunk's place in every expert's run; size [E]
-  __shared__ int s_at[ROUTE_CHUNK * MAX_TOP];
+  __shared__ int s_at[ROUTE_CHUNK * MAX_TOP], s_pick[ROUTE_CHUNK * MAX_TOP];
   pdl_launch_dependents();
   pdl_wait();
   const int tid = threadIdx.x, E = p.experts, top = p.top;
@@ -49,13 +49,17 @@ __global__ void __launch_bounds__(ROUTE_THREADS) route_place_kernel(const route_
   const int* pick = p.scratch;
   const float* weight = reinterpret_cast<const float*>(p.scratch + (size_t)p.rows * top);
   const int* counts = p.scratch + 2 * (size_t)p.rows * top;
+  const int r0 = blockIdx.x * ROUTE_CHUNK, n = min(ROUTE_CHUNK, p.rows - r0) * top;
+  const size_t at0 = (size_t)r0 * top;
   for (int e = tid; e < 2 * E; e += ROUTE_THREADS) r_sm[e] = 0;
+  for (int i = tid; i < n; i += ROUTE_THREADS) s_pick[i] = pick[at0 + i];
   __syncthreads();
   // (threads that share an expert take chunks in turn)
   const int per = E >= ROUTE_THREADS ? 1 : ROUTE_THREADS / E;
   for (int i = tid; i < E * per; i += ROUTE_THREADS) {
     const int e = i % E, g = i / E;
     int all = 0, before = 0;
+#pragma unroll 4
     for (int c = g; c < chunks; c += per) {
       const int n = counts[(size_t)c * E + e];
       all += n;
@@ -90,22 +94,23 @@ __global__ void __launch_bounds__(ROUTE_THREADS) route_place_kernel(const route_
     if (blockIdx.x == 0 && tid == 0) *p.n_tiles = tiles;
   }
   __syncthreads();
-  const int r0 = blockIdx.x * ROUTE_CHUNK, n = min(ROUTE_CHUNK, p.rows - r0) * top;
   for (int i = tid; i < n; i += ROUTE_THREADS) {  // place of entry i: entries of the chunk before it with the same expert
-    const size_t at0 = (size_t)r0 * top;
-    const int e = pick[at0 + i];
+    const int e = s_pick[i];
     int at = first[e];
-    for (int j = 0; j < i; ++j) at += pick[at0 + j] == e;
+    for (int j = 0; j < i; ++j) at += s_pick[j] == e;
     s_at[i] = at;
     p.at[at0 + i] = at;
     p.weight[at] = weight[at0 + i];
   }
   __syncthreads();
   constexpr int VEC = 16 / sizeof(T);
-  const int vecs = p.cols / VEC;
-  for (int i = tid; i < n * vecs; i += ROUTE_THREADS) {
-    const int j = i / vecs, c = (i - j * vecs) * VEC;
-    *reinterpret_cast<uint4*>(p.packed + (size_t)s_at[j] * p.ldh + c) = *reinterpret_cast<const uint4*>(p.h + (size_t)(r0 + j / top) * p.ldh + c);
+  // a row is read once and written to the places of all its experts
+  const int vecs = p.cols / VEC, rows = n / top;
+#pragma unroll 4
+  for (int i = tid; i < rows * vecs; i += ROUTE_THREADS) {
+    const int r = i / vecs, c = (i - r * vecs) * VEC;
+    const uint4 v = *reinterpret_cast<const uint4*>(p.h + (size_t)(r0 + r) * p.ldh + c);
+    for (int k = 0; k < top; ++k) *reinterpret_cast<uint4*>(p.packed + (size_t)s_at[r * top + k] * p.ldh + c) = v;
   }
 }
 

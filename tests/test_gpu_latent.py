@@ -330,3 +330,21 @@ def test_replay_program(tmp_path, dtype):
         assert f.exists() == bool(len(w))
         if len(w):
             check(np.fromfile(f, np.float32).reshape(len(w), cfg["vocab"]), w, dtype, factor=1.5)
+
+
+@both
+def test_many_chunks_of_keys(run, dtype):  # noqa: F811
+    """A window of more rows than a decode step's buffers hold at once, also with long cache rows."""
+    for mixer in (dict(heads=2, window=3000, kv_rank=48), dict(heads=1, window=1200, kv_rank=700)):
+        cfg, W = B.latent_case(seed=33, layers=1, mlp_none=(0,), mixer=mixer)
+        t = B.tokens(cfg, 1400, 3)
+        want = P.forward(t, cfg, W)
+        check(run(cfg, W, dtype, context_len=1500).feed(t, [1380, 1]), want, dtype)
+
+
+@both
+@pytest.mark.parametrize("heads", [20, 41, 75])
+def test_heads_that_share_a_cluster(run, heads, dtype):  # noqa: F811
+    cfg, W = B.latent_case(seed=heads, layers=1, mlp_none=(0,), mixer=dict(heads=heads, dim=10, rot_dim=4, vdim=9, kv_rank=37))
+    t = B.tokens(cfg, 40, 3)
+    check(run(cfg, W, dtype).feed(t, [1]), P.forward(t, cfg, W), dtype)
