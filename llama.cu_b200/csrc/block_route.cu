@@ -8,6 +8,7 @@ namespace lcu {
 namespace {
 
 constexpr int ROUTE_CHUNK = 16, ROUTE_THREADS = 256, ROUTE_WARPS = ROUTE_THREADS / 32;
+constexpr int ROUTE_SLICES = 8;  // CTAs that share the columns of a chunk's copies
 
 // scratch: pick [rows * top], pick_weight [rows * top] (float), counts [chunks][experts]
 template <typename T>
@@ -38,6 +39,7 @@ __global__ void __launch_bounds__(ROUTE_THREADS) route_pick_kernel(const route_r
   for (int e = tid; e < E; e += ROUTE_THREADS) counts[e] = count[e];
 }
 
+// grid (chunks, slices of the columns); the first slice also writes what the later launches read
 template <typename T>
 __global__ void __launch_bounds__(ROUTE_THREADS) route_place_kernel(const route_rows<T> p, int chunks) {
   extern __shared__ int r_sm[];  // first [E]: the chunk's place in every expert's run; size [E]
@@ -85,13 +87,13 @@ __global__ void __launch_bounds__(ROUTE_THREADS) route_place_kernel(const route_
       const int start = run + ns - n;
       if (e < E) {
         first[e] += start;
-        if (blockIdx.x == 0)
+        if (blockIdx.x == 0 && blockIdx.y == 0)
           for (int j = 0; j < t; ++j) p.tiles[tiles + ts - t + j] = make_int4(start + j * p.tile_rows, min(start + (j + 1) * p.tile_rows, start + n), e, 0);
       }
       run += __shfl_sync(0xffffffffu, ns, 31);
       tiles += __shfl_sync(0xffffffffu, ts, 31);
     }
-    if (blockIdx.x == 0 && tid == 0) *p.n_tiles = tiles;
+    if (blockIdx.x == 0 && blockIdx.y == 0 && tid == 0) *p.n_tiles = tiles;
   }
   __syncthreads();
   for (int i = tid; i < n; i += ROUTE_THREADS) {  // place of entry i: entries of the chunk before it with the same expert
@@ -99,16 +101,17 @@ __global__ void __launch_bounds__(ROUTE_THREADS) route_place_kernel(const route_
     int at = first[e];
     for (int j = 0; j < i; ++j) at += s_pick[j] == e;
     s_at[i] = at;
+    if (blockIdx.y > 0) continue;
     p.at[at0 + i] = at;
     p.weight[at] = weight[at0 + i];
   }
   __syncthreads();
   constexpr int VEC = 16 / sizeof(T);
   // a row is read once and written to the places of all its experts
-  const int vecs = p.cols / VEC, rows = n / top;
+  const int all = p.cols / VEC, first_vec = all * blockIdx.y / gridDim.y, vecs = all * (blockIdx.y + 1) / gridDim.y - first_vec, rows = n / top;
 #pragma unroll 4
   for (int i = tid; i < rows * vecs; i += ROUTE_THREADS) {
-    const int r = i / vecs, c = (i - r * vecs) * VEC;
+    const int r = i / vecs, c = (first_vec + i - r * vecs) * VEC;
     const uint4 v = *reinterpret_cast<const uint4*>(p.h + (size_t)(r0 + r) * p.ldh + c);
     for (int k = 0; k < top; ++k) *reinterpret_cast<uint4*>(p.packed + (size_t)s_at[r * top + k] * p.ldh + c) = v;
   }
@@ -127,7 +130,7 @@ int launch_route(const route_rows<T>& p, cudaStream_t stream) {
   LCU_REQUIRE(p.cols % 8 == 0 && p.ldh % 8 == 0, "route: rows of %d columns are not 16-byte vectors", p.cols);
   const int chunks = (int)ceil_div(p.rows, ROUTE_CHUNK);
   LCU_CUDA(launch_after(route_pick_kernel<T>, dim3(chunks), dim3(ROUTE_THREADS), (ROUTE_WARPS + 1) * (size_t)p.experts * 4, stream, p));
-  LCU_CUDA(launch_after(route_place_kernel<T>, dim3(chunks), dim3(ROUTE_THREADS), 2 * (size_t)p.experts * 4, stream, p, chunks));
+  LCU_CUDA(launch_after(route_place_kernel<T>, dim3(chunks, ROUTE_SLICES), dim3(ROUTE_THREADS), 2 * (size_t)p.experts * 4, stream, p, chunks));
   return LCU_OK;
 }
 

@@ -839,7 +839,7 @@ int& gemm_tc_group_mode() {
 // rows per tile: whole SM-pair tiles once the groups hold about that many rows each
 int gemm_tc_group_tile(int rows, int groups) {
   const int mode = gemm_tc_group_mode();
-  return mode == BM || mode == 2 * BM ? mode : rows >= 160 * groups ? 2 * BM : BM;
+  return mode == BM || mode == 2 * BM ? mode : rows >= 112 * groups ? 2 * BM : BM;
 }
 
 int launch_gemm_tc_grouped(tc_type type, void* out, const void* lhs, int ldx, const void* w, int rows, int N, int K, bool gated, const gemm_groups& g,
