@@ -40,7 +40,8 @@ int lcu_set_matmul_type(int type);
  * "prefill_tc_tile_n", "prefill_tc_pair", "prefill_tc_split", "prefill_tc_sk", "prefill_tc_kb", "prefill_sk_kb" (k-blocks per
  * stage and tensor copy of the one-SM / the pair GEMMs), "prefill_gate_fused", "prefill_u8_deq_min_rows", "prefill_u8_shadow", "prefill_fuse",
  * "prefill_attn_tc", "prefill_attn_tc_min_rows", "prefill_attn_fused_min_rows", "prefill_attn_fused_order", "prefill_attn_tiles", "prompt_pdl", "attn_stream", "prefill_group_tile" (rows per tile of the
- * products with one matrix per row group: 128, 256, 0 = by the rows per group), "block_attn_mma" (0 = the per-row attention kernel for every pass of a block model),
+ * products with one matrix per row group: 128, 256, 0 = by the rows per group), "block_row_one_cta" (a single residual row
+ * of a block model of up to this many columns is one CTA's work, a longer one a cluster's), "block_attn_mma" (0 = the per-row attention kernel for every pass of a block model),
  * "use_graph", "use_pdl", "attn_cluster", "loader_staged" (lcu_model_load: 1 = pinned double-buffered asynchronous copies, 0 = a file mapping and one
  * blocking pageable copy per tensor as the reference does).  Unknown keys are rejected. */
 int lcu_set_tuning(const char* key, int value);

@@ -54,7 +54,7 @@ __global__ void __launch_bounds__(512) block_embed_kernel(const embed_params<T> 
 // ------------------------------------------------------------------ hyper-connected residual + norm
 constexpr int HY_THREADS = 256;
 constexpr int HY_MIX = 5;       // inputs of a token-shifted mixer
-constexpr int HY_CLUSTER = 8;  // CTAs that share one row when there is only one
+constexpr int HY_CLUSTER = 8;  // CTAs that share one long row when there is only one
 
 // SM: room for the streams (p.streams <= SM); CL: CTAs per row; PRE: y is gathered and normed first
 template <typename T, int SM, int CL, bool PRE>
@@ -64,7 +64,7 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int i_row = blockIdx.x / CL, rank = blockIdx.x % CL;
   pdl_launch_dependents();
-  if (CL > 1) {  // a single row: what the columns' last step needs from the weights is on its way while the kernel before ends
+  if (gridDim.x == CL) {  // a single row: what the columns' last step needs from the weights is on its way while the kernel before ends
     const int first = min(p.width, rank * per), n = min(p.width, first + per) - first;
     if (p.router) {
       constexpr int LINE = 128 / sizeof(T);
@@ -240,14 +240,14 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
         reinterpret_cast<float*>(&back)[e] = to_f(o.e[e]);
       }
       *reinterpret_cast<pack*>(h + c) = o;
-      if (CL > 1 && p.router) *reinterpret_cast<float4*>(u_row + c - c0) = back;
+      if (p.router) *reinterpret_cast<float4*>(u_row + c - c0) = back;
     }
   } else for (int c = c0 + tid; c < c1; c += HY_THREADS) {
     const float u = u_row[c - c0];
     if (p.u_out) p.u_out[(size_t)i_row * W + c] = u;
     const T hv = from_f<T>(p.norm_w ? u * inv * (p.norm_base + p.norm_w[c]) : u);
     h[c] = hv;
-    if (CL > 1 && p.router) u_row[c - c0] = to_f(hv);
+    if (p.router) u_row[c - c0] = to_f(hv);
     if (p.mix) {
       const float hf = to_f(hv), d = (start ? 0.f : to_f(p.prev[c])) - hf;
       float mu[HY_MIX];
@@ -258,7 +258,7 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
       p.prev[c] = hv;
     }
   }
-  if (CL > 1 && p.router) {  // z = router . h: this CTA's columns of every expert, then the sum over the CTAs in rank 0
+  if (p.router) {  // z = router . h: this CTA's columns of every expert, then the sum over the CTAs in rank 0
     __syncthreads();
     float* z = u_row + per;
     for (int e = warp; e < p.experts; e += HY_THREADS / 32) {
@@ -278,17 +278,20 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_rows_kernel(const hyper_para
       a = warp_sum(a);
       if (lane == 0) z[e] = a;
     }
-    cluster_sync();
+    if (CL > 1) cluster_sync();
+    else __syncthreads();
     if (rank == 0) {
-      for (int e = tid; e < p.experts; e += HY_THREADS) {
-        float a = 0.f;
+      if (CL > 1) {
+        for (int e = tid; e < p.experts; e += HY_THREADS) {
+          float a = 0.f;
 #pragma unroll
-        for (int r = 0; r < CL; ++r) a += ld_dsmem_f32(mapa(smem_u32(z + e), r));
-        z[p.experts + e] = a;
+          for (int r = 0; r < CL; ++r) a += ld_dsmem_f32(mapa(smem_u32(z + e), r));
+          z[p.experts + e] = a;
+        }
+        __syncthreads();
       }
-      __syncthreads();
       if (warp == 0)
-        pick_largest(z + p.experts, p.experts, p.top, [&](int k, int e, float v) {
+        pick_largest(CL > 1 ? z + p.experts : z, p.experts, p.top, [&](int k, int e, float v) {
           p.pick[k] = e;
           p.pick_weight[k] = sigmoid_f(v);
         });
@@ -596,6 +599,11 @@ int launch_block_embed(const embed_params<T>& p, cudaStream_t stream) {
   return LCU_OK;
 }
 
+int& hyper_row_one_cta() {
+  static int width = 2048;
+  return width;
+}
+
 template <typename T>
 int launch_hyper_rows(const hyper_params<T>& p, int n_rows, cudaStream_t stream) {
   if (n_rows < 1) return LCU_OK;
@@ -603,9 +611,11 @@ int launch_hyper_rows(const hyper_params<T>& p, int n_rows, cudaStream_t stream)
   LCU_REQUIRE(p.mix == nullptr || (n_rows == 1 && p.n_mix == HY_MIX), "hyper_rows: the token shift is fused for a single row of %d inputs", HY_MIX);
   LCU_REQUIRE(p.router == nullptr || n_rows == 1, "hyper_rows: experts are picked for a single row");
   const bool pre = p.y && (p.post_w || p.y_rows);
+  const int most = hyper_row_one_cta();  // (measured: 7 % of a step at 1024 columns, lost again where a CTA has four vectors per thread to load twice)
+  const bool spread = n_rows == 1 && (p.width > most || p.width * p.streams > 2 * most);
 #define LCU_HYPER(SM)                                                                                                                        \
-  if (pre) return n_rows == 1 ? launch_hyper_one<T, SM, HY_CLUSTER, true>(p, n_rows, stream) : launch_hyper_one<T, SM, 1, true>(p, n_rows, stream); \
-  return n_rows == 1 ? launch_hyper_one<T, SM, HY_CLUSTER, false>(p, n_rows, stream) : launch_hyper_one<T, SM, 1, false>(p, n_rows, stream)
+  if (pre) return spread ? launch_hyper_one<T, SM, HY_CLUSTER, true>(p, n_rows, stream) : launch_hyper_one<T, SM, 1, true>(p, n_rows, stream); \
+  return spread ? launch_hyper_one<T, SM, HY_CLUSTER, false>(p, n_rows, stream) : launch_hyper_one<T, SM, 1, false>(p, n_rows, stream)
   if (p.streams == 1) { LCU_HYPER(1); }
   if (p.streams == 2) { LCU_HYPER(2); }
   if (p.streams <= 4) { LCU_HYPER(4); }

@@ -1,6 +1,6 @@
-// Kernels of the block models beside the matrix products: embedding with bigrams, hyper-connected residual rows with the
-// following norm, window-and-blocks attention, linear recurrences (retention, wkv), token shift, head normalisation and
-// gates.  T is the activation / cache / weight type of the model: __nv_bfloat16 or float.  Norms, residual streams,
+// Kernels of the block models beside the matrix products: embedding with bigrams, hyper-connected or normed residual rows with
+// the following norm, window-and-blocks attention, latent attention, linear recurrences (retention, wkv), token shift, head
+// normalisation and gates, routing of rows to experts.  T is the activation / cache / weight type of the model: __nv_bfloat16 or float.  Norms, residual streams,
 // positions, scores, softmax, decays, recurrent state and everything that enters a recurrence beside the projections are
 // binary32 in both.
 #pragma once
@@ -69,6 +69,7 @@ struct hyper_params {
   int* pick;             // [top]
   float* pick_weight;    // [top]
 };
+int& hyper_row_one_cta();  // a single row of up to this many columns (all streams: twice as many) is one CTA's, a longer one a cluster's
 template <typename T>
 int launch_hyper_rows(const hyper_params<T>& p, int n_rows, cudaStream_t stream);
 

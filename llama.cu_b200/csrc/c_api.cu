@@ -123,6 +123,7 @@ int lcu_set_tuning(const char* key, int value) {
   else if (k == "prefill_gate_fused") gemm_tc_gate_mode() = value;
   else if (k == "prompt_pdl") prompt_pdl() = value;
   else if (k == "prefill_group_tile") gemm_tc_group_mode() = value;
+  else if (k == "block_row_one_cta") hyper_row_one_cta() = value;
   else if (k == "block_attn_mma") window_mma_mode() = value;
   else if (k == "tp_debug") tp_set_debug(value);
   else if (k == "loader_staged") set_loader_staged(value);

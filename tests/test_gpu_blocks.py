@@ -161,12 +161,12 @@ def test_passes_longer_than_the_row_buffers(run):
         check(r.feed(t, WHOLE), want, dtype, factor=2.0 if dtype == "bfloat16" else 1.0)  # (a narrow model averages little out)
 
 
-@pytest.mark.parametrize("keys", [{"block_attn_mma": 0}, {"prefill_gate_fused": 256}, {"prefill_gate_fused": 512}, {"prefill_tc_sk": 256},
+@pytest.mark.parametrize("keys", [{"block_attn_mma": 0}, {"block_row_one_cta": 0}, {"prefill_gate_fused": 256}, {"prefill_gate_fused": 512}, {"prefill_tc_sk": 256},
                                   {"prefill_tc_pair": 128}, {"use_graph": 0, "use_pdl": 0}])
 def test_kernel_choices_agree(lcu, run, keys):
     """Other kernels for the same products and attention: balanced and two-SM products, the gate in the product's epilogue,
     the per-row attention, steps without a graph."""
-    defaults = {"block_attn_mma": 1, "prefill_gate_fused": -1, "prefill_tc_sk": -1, "prefill_tc_pair": -1, "use_graph": 1, "use_pdl": 1}
+    defaults = {"block_attn_mma": 1, "block_row_one_cta": 2048, "prefill_gate_fused": -1, "prefill_tc_sk": -1, "prefill_tc_pair": -1, "use_graph": 1, "use_pdl": 1}
     cfg, W = B.case(seed=14, layers=("parallel", "wkv"), width=256, ff=512,
                     mixer=dict(heads=4, kv_heads=2, dim=64, vdim=64, window=48, pool=16, rheads=2, rdim=64, rvdim=64, rot_dims=64), wkv=dict(heads=4, dim=64))
     t = B.tokens(cfg, 300, 4)

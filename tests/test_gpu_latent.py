@@ -208,11 +208,11 @@ def test_passes_longer_than_the_row_buffers(run):  # noqa: F811
 
 @pytest.mark.parametrize("width", [256, 384])
 @pytest.mark.parametrize("keys", [{}, {"prefill_group_tile": 128}, {"prefill_group_tile": 256}, {"block_attn_mma": 0}, {"use_graph": 0, "use_pdl": 0},
-                                  {"prompt_pdl": 0}])
+                                  {"prompt_pdl": 0}, {"block_row_one_cta": 0}])
 def test_kernel_choices_agree(lcu, run, keys, width):  # noqa: F811
     """Other kernels for the same products and attention: 128- and 256-row tiles of the experts' products, the per-row
-    attention, steps without a graph, launches one after the other."""
-    defaults = {"prefill_group_tile": 0, "block_attn_mma": 1, "use_graph": 1, "use_pdl": 1, "prompt_pdl": 1}
+    attention, steps without a graph, launches one after the other, a single row on a cluster."""
+    defaults = {"prefill_group_tile": 0, "block_attn_mma": 1, "use_graph": 1, "use_pdl": 1, "prompt_pdl": 1, "block_row_one_cta": 2048}
     cfg, W = B.latent_case(seed=14, layers=2, width=width, experts=3, top=2, ff=320, mixer=dict(heads=4, dim=64, rot_dim=32, vdim=64, kv_rank=128, window=48))
     t = B.tokens(cfg, 600, 4)
     want = P.forward(t, cfg, W)
